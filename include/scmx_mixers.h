@@ -1,0 +1,88 @@
+/* scmx_mixers.h — C ABI of libscmx_mixers.so: sequence mixers and bfloat16 / float32 matrix products of the hybrid decoder
+ * models (selective scan, retention, differential attention) on NVIDIA B200 (sm_100a).
+ *
+ * Conventions are those of scmx.h: device pointers only, nothing is allocated, work is enqueued on `stream`, 0 on success,
+ * shapes are validated on the host.  Additional ones:
+ *   - `dt` names the storage type of the activations, weights or cache concerned: 0 = bfloat16, 1 = float32.  Norms, scores,
+ *     recurrences and the residual stream are float32 in both cases.
+ *   - "ld" arguments are row pitches in elements.  Small per-channel vectors (norm weights, biases, decays) are float32.
+ *   - A position on the device (`pos_dev`, int32, may be NULL) replaces the host-side position, so that a captured decode step
+ *     can be replayed while the sequence grows.
+ * The functions have no counterpart in the reference project.
+ */
+#ifndef SCMX_MIXERS_H_
+#define SCMX_MIXERS_H_
+
+#include "scmx.h"
+
+#ifdef __cplusplus
+extern "C" {
+#endif
+
+/* x[t] = table[tokens[t]] (float32) and the same row in storage type as h (NULL: not wanted). */
+int scmx_embed(const int64_t* tokens, const void* table, int dt, int64_t V, int64_t T, int W, float* x, void* h, void* stream);
+
+/* r = x + w * y / rms(y).  n = 0: x_out = r.  n > 0: x_out = sum_{j < n-1} dwa[j] xs[j] + dwa[n-1] r, and with keep xs[n-1] = r
+ * (xs: [n][T, W] results xs_stride elements apart).  h_out: x_out in storage type dt, or NULL.  x_out may be x. */
+int scmx_res_norm(const float* y, int64_t ldy, const float* x, const float* w, float eps, int64_t T, int W, float* xs, int64_t xs_stride,
+                  const float* dwa, int n, int keep, float* x_out, void* h_out, int dt, void* stream);
+
+/* out[m] = w * x[rows[m]] / rms (rows NULL: m itself). */
+int scmx_norm_rows(const float* x, const int64_t* rows, const float* w, float eps, int64_t M, int W, void* out, int dt, void* stream);
+
+/* Causal depthwise convolution + SiLU: w [C, taps] (last column: the current token), b [C]; tail [C, taps-1] holds the inputs
+ * before this portion, oldest first, and is advanced. */
+int scmx_conv_silu(const void* x, int64_t ldx, int dt, int64_t T, int C, int taps, const float* w, const float* b, float* tail, void* out,
+                   int64_t ldo, void* stream);
+
+/* out[t, h] = o[t, h] / rms(o[t, h]) * silu(g[t, h]), dv values per head. */
+int scmx_head_norm_gate(const float* o, const void* g, int64_t ldg, int dt, int64_t T, int H, int dv, float eps, void* out, void* stream);
+
+/* In place on n float32 values: softplus(p) z^2 + z/2 above zero, (1/2 + softplus(q)) (e^z - 1 - z) + z/2 below. */
+int scmx_xielu(float* x, int64_t n, float a_pos, float a_neg, void* stream);
+
+/* Selective scan over n tokens: step = softplus(dtp + dt_bias), S <- 2^(step A2) S + step x B, y = (S C + D x) silu(z).
+ * A2 = -exp(A_log) log2(e) [C, N]; bc holds B at column 0 and C at column N; state [C, N] is carried. */
+int scmx_selective_scan(const void* x, int64_t ldx, const float* dtp, int64_t ldt, const void* bc, int64_t ldbc, const void* z, int64_t ldz,
+                        int dt, int64_t n, int C, int N, const float* dt_bias, const float* A2, const float* D, float* state, void* y,
+                        int64_t ldy, void* stream);
+/* One token of it; dbc = [R step inputs, B, C], the step projection w_dt [C, ldw] (type dt) is applied here. */
+int scmx_scan_step(const float* x, const float* z, const float* dbc, const void* w_dt, int64_t ldw, int dt, int C, int N, int R,
+                   const float* dt_bias, const float* A2, const float* D, float* state, float* y, void* stream);
+
+/* Retention over n tokens, S <- decay_h S + k v^T, o = S^T q (o float32 [n, H, dv]); state [H, d, dv] is carried.  q and k are
+ * rotated on their first `dims` elements by the rows of cs [n, dims] (cos, then sin), k is multiplied by kscale. */
+int scmx_retention(const void* q, int64_t ldq, const void* k, int64_t ldk, const void* v, int64_t ldv, int dt, int64_t n, int H, int d, int dv,
+                   const float* cs, int dims, float kscale, const float* decay, float* state, float* o, void* stream);
+/* One token of it with head norm and gate: y = o / rms(o) silu(g).  cs is the whole table; its row is the position. */
+int scmx_retention_step(const float* q, const float* k, const float* v, const float* g, int H, int d, int dv, const float* cs, int64_t cs_rows,
+                        int dims, int64_t pos, const int32_t* pos_dev, float kscale, const float* decay, float eps, float* state, float* y,
+                        void* stream);
+
+/* RMS norm of q (2 H vectors of d) and k (2 G vectors) with weights qw, kw; q -> q_out [2 H, n, d], k and v appended to the caches
+ * [2 G, cap, d] and [G, cap, dv] at row pos. */
+int scmx_qk_norm_append(const void* q, int64_t ldq, const void* k, int64_t ldk, const void* v, int64_t ldv, int in_dt, int cache_dt, int q_dt,
+                        int64_t n, int H, int G, int d, int dv, const float* qw, const float* kw, float eps, int64_t pos,
+                        const int32_t* pos_dev, void* q_out, void* k_cache, void* v_cache, int64_t cap, void* stream);
+/* Differential attention of n rows at positions pos .. pos+n-1 over the cache: per head o = a1 - lambda a2, o / rms(o) (1 - diff). */
+int scmx_diff_attn(const void* q, const void* k_cache, const void* v_cache, int dt, int64_t n, int64_t pos, int64_t cap, int H, int G, int d,
+                   int dv, float scale, float lambda, float diff, float eps, void* o, void* stream);
+/* One row of it; part f32 [G, nsplit, 2 H / G, dv + 2], counters int32 [G] (zero before the first call, left at zero), nsplit <= 32. */
+int scmx_diff_decode(const float* q, const void* k_cache, const void* v_cache, int dt, int64_t n_pos, const int32_t* pos_dev, int64_t cap,
+                     int H, int G, int d, int dv, float scale, float lambda, float diff, float eps, int nsplit, float* part,
+                     int32_t* counters, float* o, void* stream);
+
+/* out [M, N] = A [M, K] . W [N, K]^T, bfloat16 operands, float32 accumulation; act 1: xIELU with a_pos = softplus(p) and
+ * a_neg = 1/2 + softplus(q).  The pitches are multiples of 8; the output pitch covers N rounded up to 16 bytes (the padding is
+ * written).  tile: 0 = choose, 64 / 128 = one CTA per 128 x tile, 256 = CTA pairs.  status: int32[4]. */
+int scmx_gemm_bf16(const void* A, int64_t lda, const void* W, int64_t ldw, int64_t M, int64_t N, int64_t K, int act, float a_pos, float a_neg,
+                   void* out, int out_f32, int64_t ldo, int tile, int32_t* status, void* stream);
+/* out [N] = W [N, K] x.  epi 0: plain; 1: xIELU; 2: the first C rows pass the causal convolution + SiLU of scmx_conv_silu.
+ * Rows of W are zero padded to a multiple of 8 columns. */
+int scmx_gemv_x(const void* W, int64_t ldw, int dt, const float* x, int64_t N, int64_t K, int epi, float a_pos, float a_neg,
+                const float* conv_w, const float* conv_b, float* tail, int C, int taps, float* out, void* stream);
+
+#ifdef __cplusplus
+}
+#endif
+#endif

@@ -1,6 +1,7 @@
-"""ctypes binding of libscmx.so, the C-ABI library that holds every CUDA kernel of this package.
+"""ctypes binding of libscmx.so (the W4A8 path) and libscmx_mixers.so (sequence mixers of the hybrid decoders), the C-ABI
+libraries that hold every CUDA kernel of this package.
 
-There is no CPU fallback: if the library is missing, or a call fails, an exception is raised.
+There is no CPU fallback: if a library is missing, or a call fails, an exception is raised.
 """
 import ctypes
 import os
@@ -9,6 +10,7 @@ import torch
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "libscmx.so")
+MIXERS_PATH = os.path.join(_HERE, "libscmx_mixers.so")
 
 c_i64, c_int, c_float, c_vp = ctypes.c_int64, ctypes.c_int, ctypes.c_float, ctypes.c_void_p
 
@@ -101,25 +103,62 @@ SIGNATURES = {
     "scmx_gemv": [c_vp, c_vp, c_vp, c_vp, c_vp, c_i64, c_i64, _FMT_P, c_int, c_vp, c_vp, c_int, c_int, c_int, c_vp,
                   c_int, c_vp],
 }
+# the same for include/scmx_mixers.h
+MIXER_SIGNATURES = {
+    "scmx_embed": [c_vp, c_vp, c_int, c_i64, c_i64, c_int, c_vp, c_vp, c_vp],
+    "scmx_res_norm": [c_vp, c_i64, c_vp, c_vp, c_float, c_i64, c_int, c_vp, c_i64, c_vp, c_int, c_int, c_vp, c_vp, c_int, c_vp],
+    "scmx_norm_rows": [c_vp, c_vp, c_vp, c_float, c_i64, c_int, c_vp, c_int, c_vp],
+    "scmx_conv_silu": [c_vp, c_i64, c_int, c_i64, c_int, c_int, c_vp, c_vp, c_vp, c_vp, c_i64, c_vp],
+    "scmx_head_norm_gate": [c_vp, c_vp, c_i64, c_int, c_i64, c_int, c_int, c_float, c_vp, c_vp],
+    "scmx_xielu": [c_vp, c_i64, c_float, c_float, c_vp],
+    "scmx_selective_scan": [c_vp, c_i64, c_vp, c_i64, c_vp, c_i64, c_vp, c_i64, c_int, c_i64, c_int, c_int, c_vp, c_vp, c_vp, c_vp, c_vp,
+                            c_i64, c_vp],
+    "scmx_scan_step": [c_vp, c_vp, c_vp, c_vp, c_i64, c_int, c_int, c_int, c_int, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp],
+    "scmx_retention": [c_vp, c_i64, c_vp, c_i64, c_vp, c_i64, c_int, c_i64, c_int, c_int, c_int, c_vp, c_int, c_float, c_vp, c_vp, c_vp, c_vp],
+    "scmx_retention_step": [c_vp, c_vp, c_vp, c_vp, c_int, c_int, c_int, c_vp, c_i64, c_int, c_i64, c_vp, c_float, c_vp, c_float, c_vp,
+                            c_vp, c_vp],
+    "scmx_qk_norm_append": [c_vp, c_i64, c_vp, c_i64, c_vp, c_i64, c_int, c_int, c_int, c_i64, c_int, c_int, c_int, c_int, c_vp, c_vp,
+                            c_float, c_i64, c_vp, c_vp, c_vp, c_vp, c_i64, c_vp],
+    "scmx_diff_attn": [c_vp, c_vp, c_vp, c_int, c_i64, c_i64, c_i64, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_float, c_vp,
+                       c_vp],
+    "scmx_diff_decode": [c_vp, c_vp, c_vp, c_int, c_i64, c_vp, c_i64, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_float, c_int,
+                         c_vp, c_vp, c_vp, c_vp],
+    "scmx_gemm_bf16": [c_vp, c_i64, c_vp, c_i64, c_i64, c_i64, c_i64, c_int, c_float, c_float, c_vp, c_int, c_i64, c_int, c_vp, c_vp],
+    "scmx_gemv_x": [c_vp, c_i64, c_int, c_vp, c_i64, c_i64, c_int, c_float, c_float, c_vp, c_vp, c_vp, c_int, c_int, c_vp, c_vp],
+    "scmx_last_error_string": [],
+}
 _RESTYPE = {"scmx_last_error_string": ctypes.c_char_p}
 
 _lib = None
+_mixers = None
+
+
+def _load(path, signatures):
+    if not os.path.exists(path):
+        raise ImportError(f"{path} is missing: build it with `python {os.path.join(_HERE, 'build.py')}` "
+                          "(nvcc, sm_100a). This package has no fallback path.")
+    h = ctypes.CDLL(path)
+    for name, args in signatures.items():
+        fn = getattr(h, name)
+        fn.argtypes = args
+        fn.restype = _RESTYPE.get(name, c_int)
+    return h
 
 
 def lib():
     """The loaded library; raises ImportError with build instructions when it has not been compiled."""
     global _lib
     if _lib is None:
-        if not os.path.exists(LIB_PATH):
-            raise ImportError(f"{LIB_PATH} is missing: build it with `python {os.path.join(_HERE, 'build.py')}` "
-                              "(nvcc, sm_100a). This package has no fallback path.")
-        h = ctypes.CDLL(LIB_PATH)
-        for name, args in SIGNATURES.items():
-            fn = getattr(h, name)
-            fn.argtypes = args
-            fn.restype = _RESTYPE.get(name, c_int)
-        _lib = h
+        _lib = _load(LIB_PATH, SIGNATURES)
     return _lib
+
+
+def mixers():
+    """The library of the sequence mixers, loaded on first use."""
+    global _mixers
+    if _mixers is None:
+        _mixers = _load(MIXERS_PATH, MIXER_SIGNATURES)
+    return _mixers
 
 
 def check(rc):
@@ -129,6 +168,13 @@ def check(rc):
 
 def call(name, *args):
     check(getattr(lib(), name)(*args))
+
+
+def mcall(name, *args):
+    """The same for an entry point of the mixers library."""
+    rc = getattr(mixers(), name)(*args)
+    if rc != 0:
+        raise ScmxError(f"libscmx_mixers error {rc}: {mixers().scmx_last_error_string().decode()}")
 
 
 def ptr(t):
@@ -159,9 +205,30 @@ def status_buffer():
     return _status[dev]
 
 
+_mixer_status = {}
+
+
+def mixer_status_buffer():
+    """The status word of the mixers library's matrix products (same codes)."""
+    dev = torch.cuda.current_device()
+    if dev not in _mixer_status:
+        _mixer_status[dev] = torch.zeros(4, dtype=torch.int32, device=f"cuda:{dev}")
+    return _mixer_status[dev]
+
+
+def check_mixer_status():
+    """check_status for kernels of the mixers library alone (libscmx.so need not be built)."""
+    _raise_status(mixer_status_buffer())
+
+
 def check_status():
     """Synchronises and raises if any kernel since the last check gave up on a wait. Call outside timed regions."""
-    st = status_buffer()
+    _raise_status(status_buffer())
+    if torch.cuda.current_device() in _mixer_status:
+        check_mixer_status()
+
+
+def _raise_status(st):
     v = st.cpu().tolist()
     if v[0] != 0:
         st.zero_()

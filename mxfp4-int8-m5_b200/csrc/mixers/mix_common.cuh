@@ -1,0 +1,87 @@
+// Shared helpers of the sequence-mixer kernels: activation storage types (bfloat16 bits or float), float reductions,
+// activation functions in 32-bit, and the rotate-half table.
+#pragma once
+#include "../scmx_common.cuh"
+#include "../../../include/scmx_mixers.h"
+
+namespace scmx {
+
+typedef uint16_t bf16_t;      // storage type of a bfloat16 value
+
+__device__ __forceinline__ float ldf(const bf16_t* p) { return bf16_to_f32(*p); }
+__device__ __forceinline__ float ldf(const float* p) { return *p; }
+__device__ __forceinline__ void stf(bf16_t* p, float v) { *p = f32_to_bf16(v); }
+__device__ __forceinline__ void stf(float* p, float v) { *p = v; }
+
+// Eight consecutive values (16-byte aligned for bf16, 16-byte aligned halves for float).
+__device__ __forceinline__ void ld8(const bf16_t* p, float (&v)[8]) {
+    const uint4 w = *reinterpret_cast<const uint4*>(p);
+    const uint32_t u[4] = {w.x, w.y, w.z, w.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        v[2 * i] = bf16_lo(u[i]);
+        v[2 * i + 1] = bf16_hi(u[i]);
+    }
+}
+__device__ __forceinline__ void ld8(const float* p, float (&v)[8]) {
+    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+    v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+// Four consecutive values.
+__device__ __forceinline__ void st4(bf16_t* p, float a, float b, float c, float d) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(a, b), pack_bf16x2(c, d));
+}
+__device__ __forceinline__ void st4(float* p, float a, float b, float c, float d) {
+    *reinterpret_cast<float4*>(p) = make_float4(a, b, c, d);
+}
+__device__ __forceinline__ float4 ld4(const bf16_t* p) {
+    const uint2 w = *reinterpret_cast<const uint2*>(p);
+    return make_float4(bf16_lo(w.x), bf16_hi(w.x), bf16_lo(w.y), bf16_hi(w.y));
+}
+__device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+
+__device__ __forceinline__ float warp_sumf(float v) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+}
+// Block-wide sum; `red` holds 33 floats; every thread gets the result.
+__device__ __forceinline__ float block_sumf(float v, float* red) {
+    const int lane = threadIdx.x & 31, w = threadIdx.x >> 5, nw = blockDim.x >> 5;
+    v = warp_sumf(v);
+    __syncthreads();
+    if (lane == 0) red[w] = v;
+    __syncthreads();
+    if (w == 0) {
+        const float t = warp_sumf(lane < nw ? red[lane] : 0.0f);
+        if (lane == 0) red[32] = t;
+    }
+    __syncthreads();
+    return red[32];
+}
+
+__device__ __forceinline__ float rms_inv_f32(float sumsq, int n, float eps) { return 1.0f / sqrtf(sumsq / (float)n + eps); }
+__device__ __forceinline__ float silu_f32(float z) { return z / (1.0f + expf(-z)); }
+// log(1 + e^z) without overflow.
+__device__ __forceinline__ float softplus_f32(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
+// xIELU with a_pos = softplus(p) and a_neg = 1/2 + softplus(q): quadratic above zero, exponential below, slope 1/2 at zero.
+__device__ __forceinline__ float xielu_f32(float z, float a_pos, float a_neg) {
+    const float t = z > 0.0f ? a_pos * z * z : a_neg * (expm1f(z) - z);
+    return t + 0.5f * z;
+}
+
+// Element i of a head vector of size d after the rotate-half rotation of its first `dims` elements: i < dims/2 pairs with
+// i + dims/2.  cs: the position's table row, cos (dims/2) then sin (dims/2).
+template <typename T>
+__device__ __forceinline__ float rotated(const T* v, int i, int dims, const float* cs) {
+    const float self = ldf(v + i);
+    if (i >= dims) return self;
+    const int half = dims >> 1;
+    if (i < half) return self * cs[i] - ldf(v + i + half) * cs[half + i];
+    return self * cs[i - half] + ldf(v + i - half) * cs[i];
+}
+
+#define SCMX_DT_OK(who, dt) SCMX_REQUIRE((dt) == 0 || (dt) == 1, SCMX_EINVAL, "%s: dtype %d (0 = bfloat16, 1 = float)", who, dt)
+
+}  // namespace scmx

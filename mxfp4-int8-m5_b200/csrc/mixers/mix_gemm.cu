@@ -1,0 +1,347 @@
+// bfloat16 GEMM with float32 accumulation, out = A [M, K] . W [N, K]^T, on tcgen05.mma kind::f16.  Same structure as the INT8
+// GEMM (TMA producer warp, one MMA-issuing thread, 8 epilogue warps, two accumulators in tensor memory, persistent tiles): a K
+// block is 128 bytes = 64 values, so the stages, swizzle and descriptors are the INT8 kernel's.  Large shapes run on CTA pairs
+// (256 x 256 tiles), others on single CTAs (128 x BN tiles).
+// Epilogue: float32 or bfloat16 output, optionally through xIELU.  Rows of the output are padded to a multiple of 16 bytes.
+#include "../scmx_gemm_core.cuh"
+#include "mix_common.cuh"
+
+namespace scmx {
+
+struct BgArgs {
+    int M, N, K;
+    int out_f32;                 // 1: float output, 0: bfloat16
+    int act;                     // 0: none, 1: xIELU
+    float a_pos, a_neg;          // xIELU: softplus(p), 1/2 + softplus(q)
+    void* out;
+    int64_t ldo;                 // elements
+    int32_t* status;
+    uint64_t wait_ns;
+};
+
+// D[tmem] (+)= A[smem] * B[smem]^T, bfloat16 operands, float32 accumulate.
+__device__ __forceinline__ void umma_bf16(uint32_t d_tmem, uint64_t adesc, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
+    asm volatile(
+        "{\n\t.reg .pred p;\n\t"
+        "setp.ne.b32 p, %4, 0;\n\t"
+        "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
+        ::"r"(d_tmem), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate)
+        : "memory");
+}
+__device__ __forceinline__ void umma_bf16_pair(uint32_t d_tmem, uint64_t adesc, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
+    asm volatile(
+        "{\n\t.reg .pred p;\n\t"
+        "setp.ne.b32 p, %4, 0;\n\t"
+        "tcgen05.mma.cta_group::2.kind::f16 [%0], %1, %2, %3, p;\n\t}"
+        ::"r"(d_tmem), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate)
+        : "memory");
+}
+// Instruction descriptor, kind::f16: D = F32 (1 at [4,6)), A and B bfloat16 (1 at [7,10) and [10,13)), both K-major,
+// N >> 3 at [17,23), M >> 4 at [24,29).
+__host__ __device__ constexpr uint32_t umma_idesc_bf16(int m, int n) {
+    return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(m >> 4) << 24);
+}
+
+// Waits for this thread's tensor-memory loads; the registers pass through, so that nothing that uses them moves above the wait.
+__device__ __forceinline__ void tmem_ld_fence(uint32_t (&r)[32]) {
+    asm volatile("tcgen05.wait::ld.sync.aligned;"
+                 : "+r"(r[0]), "+r"(r[1]), "+r"(r[2]), "+r"(r[3]), "+r"(r[4]), "+r"(r[5]), "+r"(r[6]), "+r"(r[7]), "+r"(r[8]),
+                   "+r"(r[9]), "+r"(r[10]), "+r"(r[11]), "+r"(r[12]), "+r"(r[13]), "+r"(r[14]), "+r"(r[15]), "+r"(r[16]),
+                   "+r"(r[17]), "+r"(r[18]), "+r"(r[19]), "+r"(r[20]), "+r"(r[21]), "+r"(r[22]), "+r"(r[23]), "+r"(r[24]),
+                   "+r"(r[25]), "+r"(r[26]), "+r"(r[27]), "+r"(r[28]), "+r"(r[29]), "+r"(r[30]), "+r"(r[31])
+                 :: "memory");
+}
+
+// Staged 32 rows x 128 bytes -> global memory, full lines, 4 rows per instruction; `valid` bytes of the unit (a multiple of 16).
+__device__ __forceinline__ void bg_drain(const BgArgs& a, const uint8_t* stg, int lane, int row0, size_t row_bytes, size_t col_byte0, int valid) {
+    const int piece = lane & 7, rsub = lane >> 3;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        const int rl = 4 * i + rsub, row = row0 + rl;
+        const uint4 v = *reinterpret_cast<const uint4*>(stg + rl * EPI_PITCH + piece * 16);
+        if (row < a.M && piece * 16 < valid)
+            *reinterpret_cast<uint4*>(static_cast<uint8_t*>(a.out) + (size_t)row * row_bytes + col_byte0 + piece * 16) = v;
+    }
+}
+
+// One warp's 32 rows x BN/2 accumulator columns (see epilogue_warp of the INT8 kernel for the staging layout).
+template <int BN>
+__device__ __forceinline__ void bg_epilogue(const BgArgs& a, uint32_t taddr, int row0, int n0, uint8_t* stg, int lane) {
+    constexpr int CHUNKS = BN / 64;           // 32-column chunks
+    uint8_t* my = stg + lane * EPI_PITCH;
+    const int esz = a.out_f32 ? 4 : 2;
+    const size_t row_bytes = (size_t)a.ldo * esz;
+    const int npad = a.out_f32 ? (a.N + 3) & ~3 : (a.N + 7) & ~7;
+    uint32_t r[2][32];
+    tmem_ld32(taddr, r[0]);
+    tmem_ld_fence(r[0]);
+#pragma unroll
+    for (int c = 0; c < CHUNKS; ++c) {
+        uint32_t(&v)[32] = r[c & 1];
+        if (c + 1 < CHUNKS) tmem_ld32(taddr + (c + 1) * 32, r[(c + 1) & 1]);
+        if (a.act == 1) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) v[j] = __float_as_uint(xielu_f32(__uint_as_float(v[j]), a.a_pos, a.a_neg));
+        }
+        if (a.out_f32) {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) reinterpret_cast<uint4*>(my)[j] = make_uint4(v[4 * j], v[4 * j + 1], v[4 * j + 2], v[4 * j + 3]);
+            __syncwarp();
+            const int col = n0 + c * 32;
+            bg_drain(a, stg, lane, row0, row_bytes, (size_t)col * 4, min(128, (npad - col) * 4));
+            __syncwarp();
+        } else {
+            uint4* o = reinterpret_cast<uint4*>(my + 64 * (c & 1));
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                uint32_t pk[4];
+#pragma unroll
+                for (int i = 0; i < 4; ++i) pk[i] = pack_bf16x2(__uint_as_float(v[8 * j + 2 * i]), __uint_as_float(v[8 * j + 2 * i + 1]));
+                o[j] = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+            }
+            if ((c & 1) || c + 1 == CHUNKS) {
+                __syncwarp();
+                const int col = n0 + (c & ~1) * 32;
+                bg_drain(a, stg, lane, row0, row_bytes, (size_t)col * 2, min((c & 1) ? 128 : 64, (npad - col) * 2));
+                __syncwarp();
+            }
+        }
+        if (c + 1 < CHUNKS) tmem_ld_fence(r[(c + 1) & 1]);
+    }
+}
+
+template <int BN_, int STAGES_, bool PAIR>
+struct BgSmem {
+    static constexpr int BN = BN_, STAGES = STAGES_;
+    static constexpr int A_BYTES = BM * BK;
+    static constexpr int B_BYTES = (PAIR ? BN / 2 : BN) * BK;
+    static constexpr int STAGE_BYTES = A_BYTES + B_BYTES;
+    static constexpr int BAR_OFF = STAGES * STAGE_BYTES;
+    static constexpr int MISC_OFF = BAR_OFF + 8 * (2 * STAGES + 4);
+    static constexpr int EPI_OFF = (MISC_OFF + 16 + 127) & ~127;
+    static constexpr int TOTAL = EPI_OFF + EPI_STAGE_BYTES + 1024;
+};
+
+// PAIR = false: one CTA per 128 x BN tile.  PAIR = true: launched as clusters of 2, 256 x BN tile, each CTA loads its 128 rows of
+// A and its BN/2 weight rows (plain TMA loads), the leader issues the MMAs; barriers as in gemm_i8_pair_kernel.
+template <int BN, int STAGES, bool PAIR>
+__device__ __forceinline__ void gemm_bf16_body(const CUtensorMap& tmA, const CUtensorMap& tmB, const BgArgs& a) {
+    using L = BgSmem<BN, STAGES, PAIR>;
+    extern __shared__ uint8_t smem_raw[];
+    uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);
+    const uint32_t sbase = smem_u32(smem);
+    const uint32_t bar_full = sbase + L::BAR_OFF, bar_empty = bar_full + 8 * STAGES;
+    const uint32_t bar_tfull = bar_empty + 8 * STAGES, bar_tempty = bar_tfull + 16;
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + L::MISC_OFF);
+    volatile int* abort_flag = reinterpret_cast<volatile int*>(smem + L::MISC_OFF + 4);
+    constexpr uint32_t TMEM_COLS = 2 * BN;      // 128, 256 or 512
+
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const uint32_t rank = PAIR ? cluster_ctarank() : 0;
+    const bool leader = rank == 0;
+
+    if (threadIdx.x == 0) {
+        for (int s = 0; s < STAGES; ++s) {
+            mbar_init(bar_full + 8 * s, 1);
+            mbar_init(bar_empty + 8 * s, 1);
+        }
+        for (int i = 0; i < 2; ++i) {
+            mbar_init(bar_tfull + 8 * i, 1);
+            mbar_init(bar_tempty + 8 * i, PAIR ? 2 * EPI_WARPS : EPI_WARPS);
+        }
+        *abort_flag = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+    }
+    if (warp == 1) {
+        if (PAIR) {
+            tmem_alloc2(smem_u32(tmem_slot), TMEM_COLS);
+            tmem_relinquish2();
+        } else {
+            tmem_alloc(smem_u32(tmem_slot), TMEM_COLS);
+            tmem_relinquish();
+        }
+    }
+    pdl_launch_dependents();
+    tc_fence_before();
+    __syncthreads();
+    if (PAIR) cluster_sync_all();
+    tc_fence_after();
+    const uint32_t tmem_base = *tmem_slot;
+    pdl_wait();
+
+    const uint32_t full_leader = PAIR ? mapa_u32(bar_full, 0) : bar_full;
+    const uint32_t tempty_leader = PAIR ? mapa_u32(bar_tempty, 0) : bar_tempty;
+    constexpr int TM_ROWS = PAIR ? 2 * BM : BM;
+    const int worker = PAIR ? blockIdx.x >> 1 : blockIdx.x, nworkers = PAIR ? gridDim.x >> 1 : gridDim.x;
+    const int tiles_m = (a.M + TM_ROWS - 1) / TM_ROWS, tiles_n = (a.N + BN - 1) / BN;
+    const int total = tiles_m * tiles_n;
+    const int num_kb = (2 * a.K + BK - 1) / BK;
+    int fail = 0;
+
+    if (warp == 0) {
+        if (lane == 0) {
+            int stage = 0;
+            uint32_t phase = 0;
+            for (int t = worker; t < total && fail == 0; t += nworkers) {
+                const int nt = t / tiles_m, mt = t - nt * tiles_m;
+                const int row0 = mt * TM_ROWS + (int)rank * BM, brow = nt * BN + (PAIR ? (int)rank * (BN / 2) : 0);
+                for (int kb = 0; kb < num_kb; ++kb) {
+                    if (int w = mbar_wait(bar_empty + 8 * stage, phase ^ 1, abort_flag, a.wait_ns)) { fail = w == 1 ? 1 : -1; break; }
+                    const uint32_t sa = sbase + stage * L::STAGE_BYTES, sb = sa + L::A_BYTES;
+                    if (PAIR) {
+                        if (leader) mbar_expect_tx(bar_full + 8 * stage, 2 * L::STAGE_BYTES);
+                        tma_load_2d_pair(sa, &tmA, kb * BK, row0, full_leader + 8 * stage);
+                        tma_load_2d_pair(sb, &tmB, kb * BK, brow, full_leader + 8 * stage);
+                    } else {
+                        mbar_expect_tx(bar_full + 8 * stage, L::STAGE_BYTES);
+                        tma_load_2d(sa, &tmA, kb * BK, row0, bar_full + 8 * stage);
+                        tma_load_2d(sb, &tmB, kb * BK, brow, bar_full + 8 * stage);
+                    }
+                    if (++stage == STAGES) { stage = 0; phase ^= 1; }
+                }
+            }
+        }
+    } else if (warp == 1) {
+        if (lane == 0 && leader) {
+            constexpr uint32_t idesc = umma_idesc_bf16(TM_ROWS, BN);
+            int stage = 0;
+            uint32_t phase = 0, acc = 0, acc_phase = 0;
+            for (int t = worker; t < total && fail == 0; t += nworkers) {
+                const int w0 = PAIR ? mbar_wait_cluster(bar_tempty + 8 * acc, acc_phase ^ 1, abort_flag, a.wait_ns)
+                                    : mbar_wait(bar_tempty + 8 * acc, acc_phase ^ 1, abort_flag, a.wait_ns);
+                if (w0) { fail = w0 == 1 ? 2 : -1; break; }
+                tc_fence_after();
+                const uint32_t d_tmem = tmem_base + acc * BN;
+                for (int kb = 0; kb < num_kb; ++kb) {
+                    if (int w = mbar_wait(bar_full + 8 * stage, phase, abort_flag, a.wait_ns)) { fail = w == 1 ? 3 : -1; break; }
+                    tc_fence_after();
+                    const uint32_t sa = sbase + stage * L::STAGE_BYTES, sb = sa + L::A_BYTES;
+                    const uint64_t da = umma_desc(sa), db = umma_desc(sb);
+#pragma unroll
+                    for (int k = 0; k < BK / UMMA_K; ++k) {       // 16 values = 32 bytes of K per instruction
+                        const uint64_t o = (uint64_t)(k * (UMMA_K >> 4));
+                        if (PAIR) umma_bf16_pair(d_tmem, da + o, db + o, idesc, (kb | k) != 0 ? 1u : 0u);
+                        else umma_bf16(d_tmem, da + o, db + o, idesc, (kb | k) != 0 ? 1u : 0u);
+                    }
+                    if (PAIR) umma_commit_pair(bar_empty + 8 * stage);
+                    else umma_commit(bar_empty + 8 * stage);
+                    if (++stage == STAGES) { stage = 0; phase ^= 1; }
+                }
+                if (fail) break;
+                if (PAIR) umma_commit_pair(bar_tfull + 8 * acc);
+                else umma_commit(bar_tfull + 8 * acc);
+                acc ^= 1;
+                if (acc == 0) acc_phase ^= 1;
+            }
+        }
+    } else {
+        const int q = warp & 3, chalf = (warp - 2) >> 2;
+        uint32_t acc = 0, acc_phase = 0;
+        for (int t = worker; t < total && fail == 0; t += nworkers) {
+            const int nt = t / tiles_m, mt = t - nt * tiles_m;
+            const int n0 = nt * BN + chalf * (BN / 2), wrow0 = mt * TM_ROWS + (int)rank * BM + 32 * q;
+            if (int w = mbar_wait(bar_tfull + 8 * acc, acc_phase, abort_flag, a.wait_ns)) fail = w == 1 ? 4 : -1;
+            epilogue_bar();         // the epilogue threads agree on giving up before anyone touches TMEM
+            if (*abort_flag) { if (!fail) fail = -1; break; }
+            tc_fence_after();
+            bg_epilogue<BN>(a, tmem_base + acc * BN + chalf * (BN / 2) + ((uint32_t)(32 * q) << 16), wrow0, n0,
+                            smem + L::EPI_OFF + (warp - 2) * EPI_STAGE_WARP, lane);
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) {
+                if (!PAIR || leader) mbar_arrive(bar_tempty + 8 * acc);
+                else mbar_arrive_cluster(tempty_leader + 8 * acc);
+            }
+            acc ^= 1;
+            if (acc == 0) acc_phase ^= 1;
+        }
+    }
+
+    if (fail > 0) {
+        if (atomicCAS(a.status, 0, fail) == 0) {
+            a.status[1] = blockIdx.x;
+            a.status[2] = threadIdx.x;
+        }
+    }
+    __syncwarp();
+    tc_fence_before();
+    __syncthreads();
+    if (*abort_flag) {
+        const uint64_t t0 = globaltimer_ns();
+        while (globaltimer_ns() - t0 < 200000ull) __nanosleep(1000);   // 0.2 ms for outstanding TMA writes
+        __syncthreads();
+    }
+    if (PAIR) cluster_sync_all();
+    tc_fence_after();
+    if (warp == 1) {
+        if (PAIR) tmem_dealloc2(tmem_base, TMEM_COLS);
+        else tmem_dealloc(tmem_base, TMEM_COLS);
+    }
+}
+
+template <int BN, int STAGES>
+__global__ void __launch_bounds__(CTA_THREADS, 1) gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA,
+                                                            const __grid_constant__ CUtensorMap tmB, const BgArgs a) {
+    gemm_bf16_body<BN, STAGES, false>(tmA, tmB, a);
+}
+template <int BN, int STAGES>
+__global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(CTA_THREADS, 1)
+    gemm_bf16_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB, const BgArgs a) {
+    gemm_bf16_body<BN, STAGES, true>(tmA, tmB, a);
+}
+
+template <int BN, int STAGES, bool PAIR>
+static int launch_bg(const void* A, int64_t lda, const void* W, int64_t ldw, const BgArgs& a, cudaStream_t st) {
+    using L = BgSmem<BN, STAGES, PAIR>;
+    static bool configured[64] = {};
+    const int dev = current_device();
+    SCMX_REQUIRE(dev >= 0, SCMX_ECUDA, "no current CUDA device (ordinal 0..63)");
+    auto kernel = PAIR ? gemm_bf16_pair_kernel<BN, STAGES> : gemm_bf16_kernel<BN, STAGES>;
+    if (!configured[dev]) {
+        SCMX_CUDA_OK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL));
+        configured[dev] = true;
+    }
+    CUtensorMap tmA, tmB;
+    int rc = make_map_u8(&tmA, A, a.M, 2 * (int64_t)a.K, BK, BM, 128, 2 * lda);
+    if (rc) return rc;
+    rc = make_map_u8(&tmB, W, a.N, 2 * (int64_t)a.K, BK, PAIR ? BN / 2 : BN, 128, 2 * ldw);
+    if (rc) return rc;
+    constexpr int rows = PAIR ? 2 * BM : BM;
+    const int64_t tiles = ((a.M + rows - 1) / rows) * (int64_t)((a.N + BN - 1) / BN);
+    int workers = PAIR ? sm_count() / 2 : sm_count();
+    if (tiles < workers) workers = (int)tiles;
+    SCMX_PDL_OK("gemm_bf16", launch_pdl(kernel, dim3(PAIR ? 2 * workers : workers), dim3(CTA_THREADS), (size_t)L::TOTAL, st, tmA, tmB, a));
+    return SCMX_OK;
+}
+
+}  // namespace scmx
+
+using namespace scmx;
+
+extern "C" int scmx_gemm_bf16(const void* A, int64_t lda, const void* W, int64_t ldw, int64_t M, int64_t N, int64_t K, int act, float a_pos,
+                              float a_neg, void* out, int out_f32, int64_t ldo, int tile, int32_t* status, void* stream) {
+    SCMX_REQUIRE(A && W && out && status, SCMX_EINVAL, "gemm_bf16: null buffer");
+    SCMX_REQUIRE(M >= 0 && N > 0 && K > 0 && M < (1ll << 30) && N < (1ll << 30) && K < (1ll << 29), SCMX_EINVAL, "gemm_bf16: M=%lld N=%lld K=%lld",
+                 (long long)M, (long long)N, (long long)K);
+    SCMX_REQUIRE(lda % 8 == 0 && ldw % 8 == 0 && lda >= K && ldw >= K, SCMX_EINVAL,
+                 "gemm_bf16: the row pitches %lld, %lld must be multiples of 8 that hold K=%lld", (long long)lda, (long long)ldw, (long long)K);
+    const int q = out_f32 ? 4 : 8;
+    SCMX_REQUIRE(ldo % q == 0 && ldo >= (N + q - 1) / q * q, SCMX_EINVAL, "gemm_bf16: output pitch %lld for %lld columns", (long long)ldo, (long long)N);
+    SCMX_REQUIRE(((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0 && ((uintptr_t)out & 15) == 0, SCMX_EINVAL, "gemm_bf16: pointer not 16-byte aligned");
+    SCMX_REQUIRE(act == 0 || act == 1, SCMX_EINVAL, "gemm_bf16: act=%d", act);
+    SCMX_REQUIRE(tile == 0 || tile == 64 || tile == 128 || tile == 256, SCMX_EINVAL, "gemm_bf16: tile=%d", tile);
+    if (M == 0) return SCMX_OK;
+    BgArgs a;
+    a.M = (int)M; a.N = (int)N; a.K = (int)K; a.out_f32 = out_f32 ? 1 : 0; a.act = act; a.a_pos = a_pos; a.a_neg = a_neg;
+    a.out = out; a.ldo = ldo; a.status = status; a.wait_ns = g_wait_limit_ns;
+    const cudaStream_t st = (cudaStream_t)stream;
+    if (tile == 0) {
+        const int64_t m = (M + 127) / 128;
+        if (M > 128 && N >= 256 && ((M + 255) / 256) * ((N + 255) / 256) * 2 >= sm_count() / 2) tile = 256;
+        else tile = m * ((N + 127) / 128) >= sm_count() / 2 ? 128 : 64;
+    }
+    if (tile == 256) return launch_bg<256, 5, true>(A, lda, W, ldw, a, st);
+    if (tile == 128) return launch_bg<128, 5, false>(A, lda, W, ldw, a, st);
+    return launch_bg<64, 7, false>(A, lda, W, ldw, a, st);
+}

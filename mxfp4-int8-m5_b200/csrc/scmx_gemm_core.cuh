@@ -377,9 +377,10 @@ __device__ __forceinline__ void umma_commit_pair(uint32_t bar) {
                  ::"r"(bar), "h"(mask) : "memory");
 }
 
-// ---- host-side helpers defined in scmx_gemm.cu -------------------------------------------------------------------------------
+// ---- host-side helpers (scmx_gemm.cu, scmx_tma.cu) -------------------------------------------------------------------------------
 int silu_lut_ptr(cudaStream_t st, const uint16_t** out);
-int make_map_u8(CUtensorMap* map, const void* ptr, int64_t rows, int64_t row_bytes, int box_bytes, int box_rows, int swizzle_bytes);
+int make_map_u8(CUtensorMap* map, const void* ptr, int64_t rows, int64_t row_bytes, int box_bytes, int box_rows, int swizzle_bytes,
+                int64_t pitch = 0);
 int check_common(const char* who, int64_t N, int64_t K, int epi, const float* xscale, const float* wscale, const void* out,
                  const int32_t* status);
 

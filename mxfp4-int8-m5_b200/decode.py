@@ -14,7 +14,10 @@ signature.
 persistent=True (DecodeQwen3) runs all layers of a step as ONE cooperative kernel (scmx_decode_step_dense): the phases of a
 layer are separated by grid-wide barriers instead of kernel boundaries, each CTA re-quantizes the activations it needs in
 shared memory, and weight loads are issued ahead of the barriers.  Same bits as the chain of kernels; used where its limits
-hold (head size 128, widths multiples of 1024 up to 6144) and attention="kernel"."""
+hold (head size 128, widths multiples of 1024 up to 6144) and attention="kernel".
+
+DecodeHybrid is the same for hybrid decoders (fused_hybrid.FusedHybrid): GEMVs on bfloat16 or float32 weights with the mixers'
+one-token kernels between them, float32 activations."""
 import ctypes
 
 import numpy as np
@@ -23,6 +26,7 @@ import torch
 from . import _lib
 from . import sc_decode as G
 from . import sc_kernels as S
+from . import sc_mixers as X
 from . import sc_moe as M_
 
 
@@ -44,6 +48,11 @@ class _Decoder:
         self._graph = None
         self._mk = None                                       # persistent-kernel state, built per cache
 
+    @property
+    def replayable(self):
+        """Whether a step reads its position on the device, so that one captured graph serves every position."""
+        return self.attn is not None
+
     def _attend(self, at, c, q, k, v, pos_dev):
         if self.attn is not None:
             return self.attn(q, c, at.scale, n_pos=None if pos_dev is not None else c.offset + 1, pos_dev=pos_dev)
@@ -62,7 +71,7 @@ class _Decoder:
     def generate(self, tok, cache, n):
         """Greedy decoding of n tokens after `tok` (int [1, 1]) from one captured CUDA graph replayed n times.
         Returns int64 [n]; the cache advances by n positions."""
-        assert self.attn is not None, "graph decoding needs attention='kernel'"
+        assert self.replayable, "graph decoding needs attention='kernel'"
         dev = tok.device
         if self._graph is None or self._graph[0] is not cache:
             offsets = [c.offset for c in cache]
@@ -74,7 +83,10 @@ class _Decoder:
             s = torch.cuda.Stream(device=dev)
             s.wait_stream(torch.cuda.current_stream())
             with torch.cuda.stream(s):
+                kept = [(t, t.clone()) for c in cache for t in c.carried()]
                 self._step(tok_buf, cache, pos)                # warm-up outside the capture (lazy initialisations)
+                for t, old in kept:                            # recurrent states must not see the warm-up token
+                    t.copy_(old)
                 torch.cuda.synchronize()
                 g = torch.cuda.CUDAGraph()
                 with torch.cuda.graph(g, stream=s):
@@ -87,7 +99,7 @@ class _Decoder:
             self._graph = (cache, g, tok_buf, pos, logits)
         _, g, tok_buf, pos, _ = self._graph
         start = cache[0].offset
-        assert start + n <= cache[0].k.shape[1], "KV cache capacity exceeded"
+        assert start + n <= cache[0].capacity, "KV cache capacity exceeded"
         tok_buf.copy_(tok.reshape(1, 1))
         pos.fill_(start)
         out = torch.empty(n, dtype=torch.long, device=dev)
@@ -214,3 +226,59 @@ class DecodeOlmoe(_Decoder):
             h = M_.moe_combine(yd, self.pos, scores, h, pn, eps, 1, quant=False)[0]
         xn = S.rmsnorm_quant_n(h, self.model.model.norm.weight, eps, 1)[2]
         return self.head(xn[None])
+
+
+class DecodeHybrid(_Decoder):
+    """Built from a FusedHybrid.  Activations of a step are float32 vectors in buffers that live with the decoder."""
+    replayable = True
+
+    def __init__(self, fused):
+        self.f, self.model, self.args, self._graph = fused, fused.model, fused.args, None
+        dev, a = fused.model.device, self.args
+        f32 = lambda *s: torch.empty(s, dtype=torch.float32, device=dev)    # noqa: E731
+        self.xs = f32(len(a.layers) + 1, 1, a.hidden_size)      # the embedding's and every layer's result, for the depth average
+        self.x = f32(1, a.hidden_size)
+        self.bufs = []
+        for ly in fused.layers:
+            b = {"y": f32(1, a.hidden_size)}
+            if ly.type == "mamba1":
+                b.update(xz=f32(2 * ly.C), dbc=f32(ly.w_x.N), s=f32(ly.C))
+            else:
+                b.update(qkv=f32(ly.w_in.N), o=f32(ly.w_o.K))
+            if ly.type == "attention":
+                b["attn"] = X.DiffDecodeAttention(ly.H, ly.G, ly.d, ly.dv, dev)
+            if ly.w_up is not None:
+                b["u"] = f32(ly.w_up.N)
+            self.bufs.append(b)
+
+    def _mix(self, ly, b, x, c, pos_dev):
+        if ly.type == "mamba1":
+            xz = ly.w_in.vec(x, conv=(ly.conv_w, ly.conv_b, c.tail), out=b["xz"])
+            dbc = ly.w_x.vec(xz[:ly.C], out=b["dbc"])
+            o = X.scan_step(xz, xz[ly.C:], dbc, ly.w_dt, ly.dt_b, ly.A2, ly.D, c.ssm, b["s"])
+        elif ly.type == "retention":
+            q, k, v, g = ly.w_in.vec(x, out=b["qkv"]).split(ly.sizes)
+            o = X.retention_step(q, k, v, g, self.f.table(ly), ly.dims, ly.kscale, ly.decay, self.f.eps, c.kv, b["o"], c.offset, pos_dev)
+        else:
+            q, k, v = ly.w_in.vec(x, out=b["qkv"])[None].split(ly.sizes, 1)
+            q = X.qk_norm_append(q, k, v, ly.H, ly.G, ly.q_norm, ly.k_norm, self.f.eps, c, torch.float32, pos_dev)
+            o = b["attn"](q, c, ly.scale, ly.lam, ly.diff, self.f.eps, b["o"], n_pos=c.offset + 1, pos_dev=pos_dev)
+        return ly.w_o.vec(o, out=b["y"].view(-1))
+
+    def _step(self, tok, cache, pos_dev):
+        f = self.f
+        f.ensure_positions(cache[0].capacity)
+        assert pos_dev is not None or cache[0].offset < cache[0].capacity, "KV cache capacity exceeded"
+        X.embed(tok.view(-1), f.embed, self.xs[0])
+        x = self.xs[0]
+        for i, (ly, b, c) in enumerate(zip(f.layers, self.bufs, cache)):
+            self._mix(ly, b, x[0], c, pos_dev)
+            y = b["y"]
+            if ly.w_up is not None:
+                X.res_norm(y, x, ly.norm1, f.eps, self.x)
+                x = self.x
+                ly.w_down.vec(ly.w_up.vec(x[0], act=ly.act, out=b["u"]), out=y.view(-1))
+            X.res_norm(y, x, ly.norm2 if ly.w_up is not None else ly.norm1, f.eps, self.x,
+                       average=(self.xs, ly.dwa, i + 1 < len(f.layers)))
+            x = self.x
+        return f.head.vec(X.norm_rows(x, f.final_norm, f.eps, torch.float32)[0])[None, None]

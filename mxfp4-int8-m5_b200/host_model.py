@@ -64,12 +64,21 @@ def rope(x, inv_freq, offset=0):
 
 
 class KVCache:
-    """Keys and values of one layer in preallocated [heads, capacity, d] tensors; `offset` positions are filled."""
+    """Keys and values of one layer in preallocated [heads, capacity, d] tensors; `offset` positions are filled.  Values may have
+    their own head count and size."""
 
-    def __init__(self, heads, d, capacity, device="cuda", dtype=torch.bfloat16):
+    def __init__(self, heads, d, capacity, device="cuda", dtype=torch.bfloat16, v_heads=None, v_d=None):
         self.k = torch.empty((heads, capacity, d), dtype=dtype, device=device)
-        self.v = torch.empty_like(self.k)
+        self.v = torch.empty((v_heads or heads, capacity, v_d or d), dtype=dtype, device=device)
+        self.offset, self.capacity = 0, capacity
+
+    def reset(self):
+        """Forget the sequence; rows past `offset` are never read."""
         self.offset = 0
+
+    def carried(self):
+        """Tensors that a step changes in place and whose old content it reads (none: a row is only overwritten)."""
+        return []
 
     def update_and_fetch(self, k, v):
         L = k.shape[-2]
@@ -78,6 +87,29 @@ class KVCache:
         self.v[:, self.offset:self.offset + L] = v.reshape(self.k.shape[0], L, -1)
         self.offset += L
         return self.k[:, :self.offset], self.v[:, :self.offset]
+
+
+class StateCache:
+    """Recurrent state of one layer: float32 tensors of fixed size that every token updates in place, zero at the start of a
+    sequence.  `offset` and `capacity` count positions as in KVCache, so that both kinds sit in one list."""
+
+    def __init__(self, shapes, capacity, device="cuda"):
+        self.state = {n: torch.zeros(s, dtype=torch.float32, device=device) for n, s in shapes.items()}
+        self.offset, self.capacity = 0, capacity
+
+    def __getattr__(self, name):
+        try:
+            return self.__dict__["state"][name]
+        except KeyError:
+            raise AttributeError(name) from None
+
+    def reset(self):
+        self.offset = 0
+        for t in self.state.values():
+            t.zero_()
+
+    def carried(self):
+        return list(self.state.values())
 
 
 def sdpa(q, k, v, scale, causal):
@@ -252,7 +284,125 @@ class CausalLM(torch.nn.Module):
         return self
 
 
+# ---- hybrid decoders: every layer names its own mixer -------------------------------------------------------------------------
+
+@dataclass
+class LayerArgs:
+    """One entry of a hybrid model's layer list: the mixer's type and sizes, and its feed-forward (None: no second sublayer)."""
+    type: str
+    mixer: dict
+    mlp: dict = None
+
+
+@dataclass
+class HybridArgs:
+    vocab_size: int
+    hidden_size: int
+    rms_norm_eps: float
+    layers: list
+    model_type: str = "sebesun"
+
+    @classmethod
+    def from_config(cls, cfg):
+        """cfg: the dictionary of a config.json with 'vocab', 'width', 'norm' and 'layers'."""
+        layers = [LayerArgs(e["type"], dict(e["mixer"]), dict(e["mlp"]) if e.get("mlp") else None) for e in cfg["layers"]]
+        for i, e in enumerate(layers):
+            if e.type not in MIXERS:
+                raise ValueError(f"layer {i}: mixer {e.type!r} is not one of {sorted(MIXERS)}")
+            if e.mlp is not None and e.mlp.get("kind") != "dense":
+                raise ValueError(f"layer {i}: feed-forward kind {e.mlp.get('kind')!r} (only 'dense')")
+            m = e.mixer
+            if e.type == "attention" and m["heads"] % m["kv_heads"]:
+                raise ValueError(f"layer {i}: {m['heads']} heads over {m['kv_heads']} key/value heads")
+            if e.type == "retention" and len(m["decay"]) != m["heads"]:
+                raise ValueError(f"layer {i}: {len(m['decay'])} decays for {m['heads']} heads")
+        return cls(cfg["vocab"], cfg["width"], float(cfg["norm"]["eps"]), layers, cfg["architecture"].lower())
+
+
+def _mamba1_tensors(m, D):
+    inner, r, n = m["inner"], m["dt_rank"], m["state"]
+    return {"in": (2 * inner, D), "conv": (inner, m["conv"]), "conv.b": (inner,), "x": (r + 2 * n, inner), "dt": (inner, r), "dt.b": (inner,),
+            "A_log": (inner, n), "D": (inner,), "o": (D, inner)}
+
+
+def _retention_tensors(m, D):
+    h, d, dv = m["heads"], m["dim"], m["vdim"]
+    return {"q": (h * d, D), "k": (h * d, D), "v": (h * dv, D), "g": (h * dv, D), "o": (D, h * dv)}
+
+
+def _diff_attention_tensors(m, D):
+    h, g, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    return {"q": (2 * h * d, D), "k": (2 * g * d, D), "v": (g * dv, D), "q.norm": (d,), "k.norm": (d,), "lq1": (d,), "lk1": (d,), "lq2": (d,),
+            "lk2": (d,), "o": (D, h * dv)}
+
+
+# mixer type -> (tensor shapes, cache of one layer)
+MIXERS = {
+    "mamba1": (_mamba1_tensors, lambda m, cap, dev, dt: StateCache(
+        {"tail": (m["inner"], m["conv"] - 1), "ssm": (m["inner"], m["state"])}, cap, dev)),
+    "retention": (_retention_tensors, lambda m, cap, dev, dt: StateCache({"kv": (m["heads"], m["dim"], m["vdim"])}, cap, dev)),
+    "attention": (_diff_attention_tensors, lambda m, cap, dev, dt: KVCache(
+        2 * m["kv_heads"], m["dim"], cap, dev, dt, m["kv_heads"], m["vdim"])),
+}
+
+
+class HybridLM:
+    """Weights of a decoder whose layers mix selective scans, retention and differential attention: {tensor name: tensor} in the
+    checkpoint's names, on one device, bfloat16 (the serving type) or float32."""
+
+    def __init__(self, args, device="cuda", dtype=torch.bfloat16):
+        assert dtype in (torch.bfloat16, torch.float32)
+        self.args, self.device, self.dtype, self.w = args, torch.device(device), dtype, {}
+
+    def shapes(self):
+        a = self.args
+        D = a.hidden_size
+        out = {"embed": (a.vocab_size, D), "final.norm": (D,), "head": (a.vocab_size, D)}
+        for i, e in enumerate(a.layers):
+            out.update({f"l{i}.mix.{n}": s for n, s in MIXERS[e.type][0](e.mixer, D).items()})
+            out.update({f"l{i}.norm1": (D,), f"l{i}.dwa": (i + 2,)})
+            if e.mlp is not None:
+                ff = e.mlp["ff"]
+                out.update({f"l{i}.norm2": (D,), f"l{i}.mlp.up": (ff, D), f"l{i}.mlp.down": (D, ff), f"l{i}.mlp.act": (2,)})
+        return out
+
+    def load_state_dict(self, sd):
+        """sd: {name: tensor} with exactly the model's tensors."""
+        shapes = self.shapes()
+        missing, extra = sorted(set(shapes) - set(sd)), sorted(set(sd) - set(shapes))
+        if missing or extra:
+            raise ValueError(f"checkpoint tensors: missing {missing[:5]}, unexpected {extra[:5]}")
+        for n, s in shapes.items():
+            if tuple(sd[n].shape) != tuple(s):
+                raise ValueError(f"{n}: shape {tuple(sd[n].shape)}, expected {tuple(s)}")
+            self.w[n] = sd[n].to(self.device, self.dtype).contiguous()
+        return self
+
+    @torch.no_grad()
+    def init_random(self, seed=0):
+        """Seeded synthetic weights of the architecture."""
+        g = torch.Generator(device=self.device).manual_seed(seed)
+        for n, s in self.shapes().items():
+            r = torch.randn(s, generator=g, device=self.device, dtype=torch.float32)
+            leaf = n.split(".", 1)[-1]
+            if leaf in ("norm1", "norm2", "norm") or leaf.endswith((".norm", "mix.D")):
+                r = 1.0 + 0.1 * r
+            elif leaf == "dwa":
+                r = 0.05 * r
+                r[-1] += 1.0
+            elif leaf.endswith("dt.b"):
+                r -= 2.0
+            elif len(s) == 2 and leaf not in ("mix.A_log", "mix.conv"):
+                r /= s[1] ** 0.5
+            else:
+                r *= 0.3
+            self.w[n] = r.to(self.dtype)
+        return self
+
+
 def make_prompt_cache(model, capacity, device=None):
     a = model.args
+    if isinstance(model, HybridLM):
+        return [MIXERS[e.type][1](e.mixer, capacity, device or model.device, model.dtype) for e in a.layers]
     device = device or model.model.embed_tokens.weight.device
     return [KVCache(a.num_key_value_heads, a.head_dim, capacity, device) for _ in model.model.layers]

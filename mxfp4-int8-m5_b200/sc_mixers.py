@@ -1,0 +1,209 @@
+"""Torch-level calls of the sequence-mixer kernels (include/scmx_mixers.h): matrix products for bfloat16 and float32 weights,
+row kernels, selective scan, retention, differential attention.  Every function takes CUDA tensors and launches on torch's
+current stream; there is no CPU path.  Activations are bfloat16 or float32 (the weights' type); the residual stream, norms,
+scores and recurrent states are float32."""
+import torch
+
+from . import _lib
+
+LOG2E = 1.4426950408889634
+
+
+def _dt(t):
+    if t.dtype == torch.bfloat16:
+        return 0
+    assert t.dtype == torch.float32, t.dtype
+    return 1
+
+
+def _ld(t):
+    """Row pitch of a 2-D activation (unit column stride)."""
+    assert t.dim() == 2 and (t.stride(1) == 1 or t.shape[1] == 1)
+    return t.stride(0) if t.shape[0] > 1 else max(t.stride(0), t.shape[1])
+
+
+def _round8(n):
+    return (n + 7) // 8 * 8
+
+
+def empty_rows(m, n, dtype, device):
+    """[m, n] whose rows start 16-byte aligned."""
+    return torch.empty((m, _round8(n)), dtype=dtype, device=device)[:, :n]
+
+
+class XIELU:
+    """The two constants of an xIELU activation from its parameters (p, q): softplus(p) and 1/2 + softplus(q)."""
+
+    def __init__(self, act):
+        p, q = (torch.nn.functional.softplus(act.detach().double().cpu())).tolist()
+        self.a_pos, self.a_neg = p, 0.5 + q
+
+
+class Linear:
+    """y = W x without bias.  W [N, K] bfloat16 (tcgen05 GEMM / GEMV kernels) or float32 (GEMV kernel for one row, the library's
+    float32 product without reduced-precision modes otherwise)."""
+
+    def __init__(self, w):
+        self.N, self.K = w.shape
+        ld = _round8(self.K)
+        if ld == self.K:
+            self.w = w.contiguous()
+        else:
+            self.w = torch.zeros((self.N, ld), dtype=w.dtype, device=w.device)
+            self.w[:, :self.K] = w
+        self.dt = _dt(w)
+
+    def __call__(self, x, out_dtype=None, act=None, tile=0):
+        """x [M, K] -> [M, N] in out_dtype (default: the weights' type)."""
+        out_dtype = out_dtype or self.w.dtype
+        M = x.shape[0]
+        assert x.shape[1] == self.K and x.dtype == self.w.dtype and x.is_cuda
+        if self.dt == 1:
+            with _full_float32():
+                y = x @ self.w[:, :self.K].T
+            if act is not None:
+                _lib.mcall("scmx_xielu", _lib.ptr(y), y.numel(), act.a_pos, act.a_neg, _lib.stream())
+            return y
+        if _ld(x) % 8 or x.data_ptr() % 16:
+            x = empty_rows(M, self.K, x.dtype, x.device).copy_(x)
+        y = empty_rows(M, self.N, out_dtype, x.device)
+        _lib.mcall("scmx_gemm_bf16", _lib.ptr(x), _ld(x), _lib.ptr(self.w), self.w.shape[1], M, self.N, self.K, int(act is not None),
+                   act.a_pos if act else 0.0, act.a_neg if act else 0.0, _lib.ptr(y), int(out_dtype == torch.float32), _round8(self.N), tile,
+                   _lib.ptr(_lib.mixer_status_buffer()), _lib.stream())
+        return y
+
+    def vec(self, x, act=None, conv=None, out=None):
+        """One float32 row [K] -> float32 [N]; conv = (weights [C, taps], bias [C], tail) for the convolution epilogue."""
+        assert x.dtype == torch.float32 and x.numel() == self.K and x.is_contiguous()
+        out = torch.empty(self.N, dtype=torch.float32, device=x.device) if out is None else out
+        epi = 2 if conv is not None else int(act is not None)
+        cw, cb, tail = conv if conv is not None else (None, None, None)
+        _lib.mcall("scmx_gemv_x", _lib.ptr(self.w), self.w.shape[1], self.dt, _lib.ptr(x), self.N, self.K, epi, act.a_pos if act else 0.0,
+                   act.a_neg if act else 0.0, _lib.ptr(cw), _lib.ptr(cb), _lib.ptr(tail), 0 if cw is None else cw.shape[0],
+                   0 if cw is None else cw.shape[1], _lib.ptr(out), _lib.stream())
+        return out
+
+
+class _full_float32:
+    """No TF32 in the float32 products, whatever the process-wide setting."""
+
+    def __enter__(self):
+        self.old = torch.backends.cuda.matmul.allow_tf32
+        torch.backends.cuda.matmul.allow_tf32 = False
+
+    def __exit__(self, *a):
+        torch.backends.cuda.matmul.allow_tf32 = self.old
+
+
+def embed(tokens, table, x, h=None):
+    """x [T, W] float32 <- table rows; h: the same in the table's type."""
+    _lib.require_cuda(tokens, table, x, h)
+    _lib.mcall("scmx_embed", _lib.ptr(tokens), _lib.ptr(table), _dt(table), table.shape[0], tokens.numel(), table.shape[1], _lib.ptr(x),
+               _lib.ptr(h), _lib.stream())
+
+
+def res_norm(y, x, w, eps, x_out, h_out=None, average=None):
+    """x_out = x + w * y / rms(y), or with average = (xs [n, T, W], weights [n], keep) the weighted sum of xs[: n - 1] and that
+    value (stored at xs[n - 1] when keep)."""
+    T, W = x.shape
+    xs, dwa, keep = average if average is not None else (None, None, False)
+    n = 0 if dwa is None else dwa.numel()
+    _lib.mcall("scmx_res_norm", _lib.ptr(y), _ld(y), _lib.ptr(x), _lib.ptr(w), eps, T, W, _lib.ptr(xs), 0 if xs is None else xs.stride(0),
+               _lib.ptr(dwa), n, int(keep), _lib.ptr(x_out), _lib.ptr(h_out), 1 if h_out is None else _dt(h_out), _lib.stream())
+
+
+def norm_rows(x, w, eps, dtype, rows=None):
+    M = x.shape[0] if rows is None else rows.numel()
+    out = torch.empty((M, x.shape[1]), dtype=dtype, device=x.device)
+    _lib.mcall("scmx_norm_rows", _lib.ptr(x), _lib.ptr(rows), _lib.ptr(w), eps, M, x.shape[1], _lib.ptr(out), _dt(out), _lib.stream())
+    return out
+
+
+def conv_silu(x, w, b, tail):
+    """x [T, C] (row pitch free) -> silu(causal convolution); tail is advanced."""
+    T, C = x.shape
+    out = empty_rows(T, C, x.dtype, x.device)
+    _lib.mcall("scmx_conv_silu", _lib.ptr(x), _ld(x), _dt(x), T, C, w.shape[1], _lib.ptr(w), _lib.ptr(b), _lib.ptr(tail), _lib.ptr(out),
+               _ld(out), _lib.stream())
+    return out
+
+
+def selective_scan(x, dtp, bc, z, dt_bias, A2, D, state):
+    """x, z [T, C], dtp [T, C] float32, bc [T, 2 N] -> gated output [T, C]; state [C, N] is advanced."""
+    T, C = x.shape
+    y = empty_rows(T, C, x.dtype, x.device)
+    _lib.mcall("scmx_selective_scan", _lib.ptr(x), _ld(x), _lib.ptr(dtp), _ld(dtp), _lib.ptr(bc), _ld(bc), _lib.ptr(z), _ld(z), _dt(x), T, C,
+               A2.shape[1], _lib.ptr(dt_bias), _lib.ptr(A2), _lib.ptr(D), _lib.ptr(state), _lib.ptr(y), _ld(y), _lib.stream())
+    return y
+
+
+def scan_step(x, z, dbc, w_dt, dt_bias, A2, D, state, y):
+    C, N = A2.shape
+    _lib.mcall("scmx_scan_step", _lib.ptr(x), _lib.ptr(z), _lib.ptr(dbc), _lib.ptr(w_dt.w), w_dt.w.shape[1], w_dt.dt, C, N, w_dt.K,
+               _lib.ptr(dt_bias), _lib.ptr(A2), _lib.ptr(D), _lib.ptr(state), _lib.ptr(y), _lib.stream())
+    return y
+
+
+def rotary_table(base, dims, rows, device):
+    """float32 [rows, dims]: cos then sin of position * base^(-2i/dims), angles in float64."""
+    f = float(base) ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64, device=device) / max(dims, 1))
+    ang = torch.arange(rows, dtype=torch.float64, device=device)[:, None] * f[None, :]
+    return torch.cat([torch.cos(ang), torch.sin(ang)], 1).float().contiguous()
+
+
+def retention(q, k, v, cs, dims, kscale, decay, state):
+    """q, k [T, H d], v [T, H dv] -> o [T, H, dv] float32; cs: the table rows of this portion; state [H, d, dv] is advanced."""
+    T, (H, d, dv) = q.shape[0], state.shape
+    o = torch.empty((T, H, dv), dtype=torch.float32, device=q.device)
+    _lib.mcall("scmx_retention", _lib.ptr(q), _ld(q), _lib.ptr(k), _ld(k), _lib.ptr(v), _ld(v), _dt(q), T, H, d, dv, _lib.ptr(cs), dims, kscale,
+               _lib.ptr(decay), _lib.ptr(state), _lib.ptr(o), _lib.stream())
+    return o
+
+
+def head_norm_gate(o, g, eps):
+    T, H, dv = o.shape
+    out = torch.empty((T, H * dv), dtype=g.dtype, device=o.device)
+    _lib.mcall("scmx_head_norm_gate", _lib.ptr(o), _lib.ptr(g), _ld(g), _dt(g), T, H, dv, eps, _lib.ptr(out), _lib.stream())
+    return out
+
+
+def retention_step(q, k, v, g, table, dims, kscale, decay, eps, state, y, pos=0, pos_dev=None):
+    H, d, dv = state.shape
+    _lib.mcall("scmx_retention_step", _lib.ptr(q), _lib.ptr(k), _lib.ptr(v), _lib.ptr(g), H, d, dv, _lib.ptr(table), max(1, table.shape[0]), dims,
+               pos, _lib.ptr(pos_dev), kscale, _lib.ptr(decay), eps, _lib.ptr(state), _lib.ptr(y), _lib.stream())
+    return y
+
+
+def qk_norm_append(q, k, v, H, G, qw, kw, eps, cache, q_dtype, pos_dev=None):
+    """q [T, 2 H d], k [T, 2 G d], v [T, G dv]: normalized q [2 H, T, d]; normalized k and v go to rows cache.offset .. of the cache."""
+    T, d, dv, cap = q.shape[0], qw.numel(), cache.v.shape[2], cache.k.shape[1]
+    qo = torch.empty((2 * H, T, d), dtype=q_dtype, device=q.device)
+    _lib.mcall("scmx_qk_norm_append", _lib.ptr(q), _ld(q), _lib.ptr(k), _ld(k), _lib.ptr(v), _ld(v), _dt(q), _dt(cache.k), _dt(qo), T, H, G, d, dv,
+               _lib.ptr(qw), _lib.ptr(kw), eps, cache.offset, _lib.ptr(pos_dev), _lib.ptr(qo), _lib.ptr(cache.k), _lib.ptr(cache.v), cap,
+               _lib.stream())
+    return qo
+
+
+def diff_attention(q, cache, H, G, scale, lam, diff, eps):
+    """q [2 H, T, d] at positions cache.offset .. (their keys and values already in the cache) -> [T, H dv]."""
+    T, d, dv = q.shape[1], q.shape[2], cache.v.shape[2]
+    o = torch.empty((T, H * dv), dtype=q.dtype, device=q.device)
+    _lib.mcall("scmx_diff_attn", _lib.ptr(q), _lib.ptr(cache.k), _lib.ptr(cache.v), _dt(q), T, cache.offset, cache.k.shape[1], H, G, d, dv, scale,
+               lam, diff, eps, _lib.ptr(o), _lib.stream())
+    return o
+
+
+class DiffDecodeAttention:
+    """One query row of differential attention over the cache, with its scratch."""
+
+    def __init__(self, H, G, d, dv, device, n_sm=148):
+        self.H, self.G, self.d, self.dv = H, G, d, dv
+        self.nsplit = max(1, min(32, n_sm // G))
+        self.part = torch.empty((G, self.nsplit, 2 * (H // G), dv + 2), dtype=torch.float32, device=device)
+        self.counters = torch.zeros(G, dtype=torch.int32, device=device)
+
+    def __call__(self, q, cache, scale, lam, diff, eps, o, n_pos=None, pos_dev=None):
+        _lib.mcall("scmx_diff_decode", _lib.ptr(q), _lib.ptr(cache.k), _lib.ptr(cache.v), _dt(cache.k), int(n_pos or 0), _lib.ptr(pos_dev),
+                   cache.k.shape[1], self.H, self.G, self.d, self.dv, scale, lam, diff, eps, self.nsplit, _lib.ptr(self.part),
+                   _lib.ptr(self.counters), _lib.ptr(o), _lib.stream())
+        return o
