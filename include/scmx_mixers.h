@@ -51,9 +51,13 @@ int scmx_scan_step(const float* x, const float* z, const float* dbc, const void*
                    const float* dt_bias, const float* A2, const float* D, float* state, float* y, void* stream);
 
 /* Retention over n tokens, S <- decay_h S + k v^T, o = S^T q (o float32 [n, H, dv]); state [H, d, dv] is carried.  q and k are
- * rotated on their first `dims` elements by the rows of cs [n, dims] (cos, then sin), k is multiplied by kscale. */
+ * rotated on their first `dims` elements by the rows of cs [n, dims] (cos, then sin), k is multiplied by kscale.
+ * scratch NULL: token by token on the CUDA cores, any sizes.  Otherwise the chunk-parallel tensor-core form (bfloat16, positive
+ * decays) with scmx_retention_scratch bytes, 256-byte aligned; 0 bytes: the sizes have no such form.  status: int32[4]. */
+int64_t scmx_retention_scratch(int64_t n, int H, int d, int dv, int dims, int64_t ldv);
 int scmx_retention(const void* q, int64_t ldq, const void* k, int64_t ldk, const void* v, int64_t ldv, int dt, int64_t n, int H, int d, int dv,
-                   const float* cs, int dims, float kscale, const float* decay, float* state, float* o, void* stream);
+                   const float* cs, int dims, float kscale, const float* decay, float* state, float* o, void* scratch, int64_t scratch_bytes,
+                   int32_t* status, void* stream);
 /* One token of it with head norm and gate: y = o / rms(o) silu(g).  cs is the whole table; its row is the position. */
 int scmx_retention_step(const float* q, const float* k, const float* v, const float* g, int H, int d, int dv, const float* cs, int64_t cs_rows,
                         int dims, int64_t pos, const int32_t* pos_dev, float kscale, const float* decay, float eps, float* state, float* y,
@@ -64,9 +68,10 @@ int scmx_retention_step(const float* q, const float* k, const float* v, const fl
 int scmx_qk_norm_append(const void* q, int64_t ldq, const void* k, int64_t ldk, const void* v, int64_t ldv, int in_dt, int cache_dt, int q_dt,
                         int64_t n, int H, int G, int d, int dv, const float* qw, const float* kw, float eps, int64_t pos,
                         const int32_t* pos_dev, void* q_out, void* k_cache, void* v_cache, int64_t cap, void* stream);
-/* Differential attention of n rows at positions pos .. pos+n-1 over the cache: per head o = a1 - lambda a2, o / rms(o) (1 - diff). */
+/* Differential attention of n rows at positions pos .. pos+n-1 over the cache: per head o = a1 - lambda a2, o / rms(o) (1 - diff).
+ * form: 0 = choose, 1 = CUDA cores (any sizes), 2 = tensor cores (bfloat16, sizes up to 128, multiples of 8; status: int32[4]). */
 int scmx_diff_attn(const void* q, const void* k_cache, const void* v_cache, int dt, int64_t n, int64_t pos, int64_t cap, int H, int G, int d,
-                   int dv, float scale, float lambda, float diff, float eps, void* o, void* stream);
+                   int dv, float scale, float lambda, float diff, float eps, void* o, int form, int32_t* status, void* stream);
 /* One row of it; part f32 [G, nsplit, 2 H / G, dv + 2], counters int32 [G] (zero before the first call, left at zero), nsplit <= 32. */
 int scmx_diff_decode(const float* q, const void* k_cache, const void* v_cache, int dt, int64_t n_pos, const int32_t* pos_dev, int64_t cap,
                      int H, int G, int d, int dv, float scale, float lambda, float diff, float eps, int nsplit, float* part,

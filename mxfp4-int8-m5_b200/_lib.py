@@ -114,20 +114,22 @@ MIXER_SIGNATURES = {
     "scmx_selective_scan": [c_vp, c_i64, c_vp, c_i64, c_vp, c_i64, c_vp, c_i64, c_int, c_i64, c_int, c_int, c_vp, c_vp, c_vp, c_vp, c_vp,
                             c_i64, c_vp],
     "scmx_scan_step": [c_vp, c_vp, c_vp, c_vp, c_i64, c_int, c_int, c_int, c_int, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp],
-    "scmx_retention": [c_vp, c_i64, c_vp, c_i64, c_vp, c_i64, c_int, c_i64, c_int, c_int, c_int, c_vp, c_int, c_float, c_vp, c_vp, c_vp, c_vp],
+    "scmx_retention_scratch": [c_i64, c_int, c_int, c_int, c_int, c_i64],
+    "scmx_retention": [c_vp, c_i64, c_vp, c_i64, c_vp, c_i64, c_int, c_i64, c_int, c_int, c_int, c_vp, c_int, c_float, c_vp, c_vp, c_vp, c_vp,
+                       c_i64, c_vp, c_vp],
     "scmx_retention_step": [c_vp, c_vp, c_vp, c_vp, c_int, c_int, c_int, c_vp, c_i64, c_int, c_i64, c_vp, c_float, c_vp, c_float, c_vp,
                             c_vp, c_vp],
     "scmx_qk_norm_append": [c_vp, c_i64, c_vp, c_i64, c_vp, c_i64, c_int, c_int, c_int, c_i64, c_int, c_int, c_int, c_int, c_vp, c_vp,
                             c_float, c_i64, c_vp, c_vp, c_vp, c_vp, c_i64, c_vp],
     "scmx_diff_attn": [c_vp, c_vp, c_vp, c_int, c_i64, c_i64, c_i64, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_float, c_vp,
-                       c_vp],
+                       c_int, c_vp, c_vp],
     "scmx_diff_decode": [c_vp, c_vp, c_vp, c_int, c_i64, c_vp, c_i64, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_float, c_int,
                          c_vp, c_vp, c_vp, c_vp],
     "scmx_gemm_bf16": [c_vp, c_i64, c_vp, c_i64, c_i64, c_i64, c_i64, c_int, c_float, c_float, c_vp, c_int, c_i64, c_int, c_vp, c_vp],
     "scmx_gemv_x": [c_vp, c_i64, c_int, c_vp, c_i64, c_i64, c_int, c_float, c_float, c_vp, c_vp, c_vp, c_int, c_int, c_vp, c_vp],
     "scmx_last_error_string": [],
 }
-_RESTYPE = {"scmx_last_error_string": ctypes.c_char_p}
+_RESTYPE = {"scmx_last_error_string": ctypes.c_char_p, "scmx_retention_scratch": c_i64}
 
 _lib = None
 _mixers = None
@@ -235,7 +237,12 @@ def _raise_status(st):
         raise ScmxError(f"device-side wait ran out: {describe_status(v[0])} (CTA or rank {v[1]}, thread {v[2]})")
 
 
-_GEMM_ROLES = {6: "GEMM unpack warp waiting for a packed weight tile", 1: "GEMM producer waiting for a free stage", 2: "GEMM MMA warp waiting for a free accumulator",
+_GEMM_ROLES = {41: "retention chunk product waiting for operands", 42: "retention chunk kernel waiting for the product",
+               43: "retention producer waiting for a free stage", 44: "retention MMA thread waiting for operands or weights",
+               45: "retention warp waiting for scores or outputs",
+               31: "attention producer waiting for a free key tile", 32: "attention producer waiting for a free value tile",
+               33: "attention MMA thread waiting for operands", 34: "attention MMA thread waiting for softmax weights",
+               35: "attention softmax warp waiting for scores", 36: "attention softmax warp waiting for the last product", 6: "GEMM unpack warp waiting for a packed weight tile", 1: "GEMM producer waiting for a free stage", 2: "GEMM MMA warp waiting for a free accumulator",
                3: "GEMM MMA warp waiting for operands", 4: "GEMM epilogue waiting for an accumulator",
                5: "GEMM CTA pair waiting for its peer", 11: "streaming GEMV producer waiting for a free stage",
                12: "streaming GEMV consumer waiting for a tile", 20: "peer barrier waiting for another rank's flag"}

@@ -2,11 +2,16 @@
 // and scaled.  Keys are cached after their norm: K [2 G, cap, d] (map m of key/value head g at row 2 g + m), V [G, cap, dv].
 //
 // qk_norm_append_kernel   q / k RMS norm per head and map, K / V rows appended to the cache
-// diff_attn_kernel        prompt portions, any sizes and storage types, float32 arithmetic on the CUDA cores
+// diff_attn_kernel        prompt portions, any sizes and storage types, float32 arithmetic on the CUDA cores (bfloat16 with head
+//                         sizes up to 128: diff_attn_tc, tensor cores)
 // diff_decode_kernel      one query row: positions split over CTAs, the last CTA of a key/value head combines
 #include "mix_common.cuh"
 
 namespace scmx {
+
+bool diff_attn_tc_supported(int64_t n, int64_t pos, int d, int dv, float scale);
+int diff_attn_tc(const bf16_t* q, const bf16_t* kc, const bf16_t* vc, int64_t n, int64_t pos, int64_t cap, int H, int G, int d, int dv, float scale,
+                 float lambda, float diff, float eps, bf16_t* o, int32_t* status, cudaStream_t st);
 
 // ---- q / k norm + cache append ------------------------------------------------------------------------------------------
 template <typename TI, typename TC, typename TQ>
@@ -387,12 +392,18 @@ extern "C" int scmx_qk_norm_append(const void* q, int64_t ldq, const void* k, in
 }
 
 extern "C" int scmx_diff_attn(const void* q, const void* k_cache, const void* v_cache, int dt, int64_t n, int64_t pos, int64_t cap, int H, int G,
-                              int d, int dv, float scale, float lambda, float diff, float eps, void* o, void* stream) {
+                              int d, int dv, float scale, float lambda, float diff, float eps, void* o, int form, int32_t* status, void* stream) {
     SCMX_DT_OK("diff_attn", dt);
     SCMX_REQUIRE(q && k_cache && v_cache && o, SCMX_EINVAL, "diff_attn: null buffer");
     SCMX_REQUIRE(n >= 0 && pos >= 0 && pos + n <= cap && H > 0 && G > 0 && H % G == 0 && d > 0 && dv > 0, SCMX_EINVAL,
                  "diff_attn: %lld rows at %lld in a cache of %lld, heads %d / %d of %d / %d", (long long)n, (long long)pos, (long long)cap, H, G, d, dv);
+    SCMX_REQUIRE(form >= 0 && form <= 2, SCMX_EINVAL, "diff_attn: form=%d", form);
     if (n == 0) return SCMX_OK;
+    const bool tc = dt == 0 && status != nullptr && diff_attn_tc_supported(n, pos, d, dv, scale);
+    SCMX_REQUIRE(form != 2 || tc, SCMX_ELIMIT, "diff_attn: no tensor-core form for head sizes %d / %d", d, dv);
+    if (tc && form != 1)
+        return diff_attn_tc((const bf16_t*)q, (const bf16_t*)k_cache, (const bf16_t*)v_cache, n, pos, cap, H, G, d, dv, scale, lambda, diff, eps,
+                            (bf16_t*)o, status, (cudaStream_t)stream);
 #define FILL(T)                                                                                                           \
     DiffAttnArgs<T> a;                                                                                                     \
     a.q = (const T*)q; a.k = (const T*)k_cache; a.v = (const T*)v_cache; a.o = (T*)o; a.n = n; a.pos = pos; a.cap = cap;   \

@@ -3,8 +3,7 @@
 // block is 128 bytes = 64 values, so the stages, swizzle and descriptors are the INT8 kernel's.  Large shapes run on CTA pairs
 // (256 x 256 tiles), others on single CTAs (128 x BN tiles).
 // Epilogue: float32 or bfloat16 output, optionally through xIELU.  Rows of the output are padded to a multiple of 16 bytes.
-#include "../scmx_gemm_core.cuh"
-#include "mix_common.cuh"
+#include "mix_tc.cuh"
 
 namespace scmx {
 
@@ -18,39 +17,6 @@ struct BgArgs {
     int32_t* status;
     uint64_t wait_ns;
 };
-
-// D[tmem] (+)= A[smem] * B[smem]^T, bfloat16 operands, float32 accumulate.
-__device__ __forceinline__ void umma_bf16(uint32_t d_tmem, uint64_t adesc, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
-    asm volatile(
-        "{\n\t.reg .pred p;\n\t"
-        "setp.ne.b32 p, %4, 0;\n\t"
-        "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
-        ::"r"(d_tmem), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate)
-        : "memory");
-}
-__device__ __forceinline__ void umma_bf16_pair(uint32_t d_tmem, uint64_t adesc, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
-    asm volatile(
-        "{\n\t.reg .pred p;\n\t"
-        "setp.ne.b32 p, %4, 0;\n\t"
-        "tcgen05.mma.cta_group::2.kind::f16 [%0], %1, %2, %3, p;\n\t}"
-        ::"r"(d_tmem), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate)
-        : "memory");
-}
-// Instruction descriptor, kind::f16: D = F32 (1 at [4,6)), A and B bfloat16 (1 at [7,10) and [10,13)), both K-major,
-// N >> 3 at [17,23), M >> 4 at [24,29).
-__host__ __device__ constexpr uint32_t umma_idesc_bf16(int m, int n) {
-    return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(m >> 4) << 24);
-}
-
-// Waits for this thread's tensor-memory loads; the registers pass through, so that nothing that uses them moves above the wait.
-__device__ __forceinline__ void tmem_ld_fence(uint32_t (&r)[32]) {
-    asm volatile("tcgen05.wait::ld.sync.aligned;"
-                 : "+r"(r[0]), "+r"(r[1]), "+r"(r[2]), "+r"(r[3]), "+r"(r[4]), "+r"(r[5]), "+r"(r[6]), "+r"(r[7]), "+r"(r[8]),
-                   "+r"(r[9]), "+r"(r[10]), "+r"(r[11]), "+r"(r[12]), "+r"(r[13]), "+r"(r[14]), "+r"(r[15]), "+r"(r[16]),
-                   "+r"(r[17]), "+r"(r[18]), "+r"(r[19]), "+r"(r[20]), "+r"(r[21]), "+r"(r[22]), "+r"(r[23]), "+r"(r[24]),
-                   "+r"(r[25]), "+r"(r[26]), "+r"(r[27]), "+r"(r[28]), "+r"(r[29]), "+r"(r[30]), "+r"(r[31])
-                 :: "memory");
-}
 
 // Staged 32 rows x 128 bytes -> global memory, full lines, 4 rows per instruction; `valid` bytes of the unit (a multiple of 16).
 __device__ __forceinline__ void bg_drain(const BgArgs& a, const uint8_t* stg, int lane, int row0, size_t row_bytes, size_t col_byte0, int valid) {
@@ -297,7 +263,9 @@ static int launch_bg(const void* A, int64_t lda, const void* W, int64_t ldw, con
     static bool configured[64] = {};
     const int dev = current_device();
     SCMX_REQUIRE(dev >= 0, SCMX_ECUDA, "no current CUDA device (ordinal 0..63)");
-    auto kernel = PAIR ? gemm_bf16_pair_kernel<BN, STAGES> : gemm_bf16_kernel<BN, STAGES>;
+    void (*kernel)(CUtensorMap, CUtensorMap, BgArgs);
+    if constexpr (PAIR) kernel = gemm_bf16_pair_kernel<BN, STAGES>;
+    else kernel = gemm_bf16_kernel<BN, STAGES>;
     if (!configured[dev]) {
         SCMX_CUDA_OK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL));
         configured[dev] = true;

@@ -1,7 +1,7 @@
 // Retention: linear attention with a fixed decay per head.  S_t = decay S_(t-1) + k_t v_t^T, o_t = S_t^T q_t; q and k are rotated
 // (rotate-half, table of cosines and sines per position) and k is scaled when they are read, in float32.
 //
-// retention_scan_kernel   any sizes, any storage type: token by token, float32
+// retention_scan_kernel   any sizes, any storage type: token by token, float32 (bfloat16 prompts: retention_tc, tensor cores)
 // retention_step_kernel   one token: state update, output, head norm and gate, a cluster of CTAs per head
 #include <cooperative_groups.h>
 #include "mix_common.cuh"
@@ -9,6 +9,12 @@
 namespace cg = cooperative_groups;
 
 namespace scmx {
+
+bool retention_tc_supported(int64_t n, int H, int d, int dv, int dims, int64_t ldv);
+int64_t retention_tc_scratch(int64_t n, int H, int d, int dv);
+int retention_tc(const bf16_t* q, int64_t ldq, const bf16_t* k, int64_t ldk, const bf16_t* v, int64_t ldv, int64_t n, int H, int d, int dv,
+                 const float* cs, int dims, float kscale, const float* decay, float* state, float* o, void* scratch, int32_t* status,
+                 cudaStream_t st);
 
 template <typename T>
 struct RetArgs {
@@ -159,14 +165,26 @@ static int run_ret_scan(const RetArgs<T>& a, cudaStream_t st) {
 
 using namespace scmx;
 
+extern "C" int64_t scmx_retention_scratch(int64_t n, int H, int d, int dv, int dims, int64_t ldv) {
+    return n > 0 && H > 0 && d > 0 && dv > 0 && retention_tc_supported(n, H, d, dv, dims, ldv) ? retention_tc_scratch(n, H, d, dv) : 0;
+}
+
 extern "C" int scmx_retention(const void* q, int64_t ldq, const void* k, int64_t ldk, const void* v, int64_t ldv, int dt, int64_t n, int H,
                               int d, int dv, const float* cs, int dims, float kscale, const float* decay, float* state, float* o,
-                              void* stream) {
+                              void* scratch, int64_t scratch_bytes, int32_t* status, void* stream) {
     SCMX_DT_OK("retention", dt);
     SCMX_REQUIRE(q && k && v && decay && state && o, SCMX_EINVAL, "retention: null buffer");
     SCMX_REQUIRE(n >= 0 && H > 0 && d > 0 && dv > 0 && dims >= 0 && dims <= d && dims % 2 == 0 && (dims == 0 || cs), SCMX_EINVAL,
                  "retention: n=%lld heads=%d size=%d values=%d rotated=%d", (long long)n, H, d, dv, dims);
     if (n == 0) return SCMX_OK;
+    if (scratch != nullptr) {
+        SCMX_REQUIRE(dt == 0 && status && retention_tc_supported(n, H, d, dv, dims, ldv), SCMX_ELIMIT,
+                     "retention: no tensor-core form for head sizes %d / %d", d, dv);
+        SCMX_REQUIRE(((uintptr_t)v & 15) == 0 && ((uintptr_t)scratch & 255) == 0 && scratch_bytes >= retention_tc_scratch(n, H, d, dv), SCMX_EINVAL,
+                     "retention: scratch of %lld bytes or an unaligned pointer", (long long)scratch_bytes);
+        return retention_tc((const bf16_t*)q, ldq, (const bf16_t*)k, ldk, (const bf16_t*)v, ldv, n, H, d, dv, cs, dims, kscale, decay, state, o,
+                            scratch, status, (cudaStream_t)stream);
+    }
 #define FILL(T)                                                                                                           \
     RetArgs<T> a;                                                                                                          \
     a.q = (const T*)q; a.k = (const T*)k; a.v = (const T*)v; a.cs = cs; a.decay = decay; a.state = state; a.o = o;         \

@@ -381,6 +381,8 @@ __device__ __forceinline__ void umma_commit_pair(uint32_t bar) {
 int silu_lut_ptr(cudaStream_t st, const uint16_t** out);
 int make_map_u8(CUtensorMap* map, const void* ptr, int64_t rows, int64_t row_bytes, int box_bytes, int box_rows, int swizzle_bytes,
                 int64_t pitch = 0);
+int make_map_planes(CUtensorMap* map, const void* ptr, int64_t planes, int64_t rows, int64_t row_bytes, int64_t pitch, int64_t plane_pitch,
+                    int box_rows);
 int check_common(const char* who, int64_t N, int64_t K, int epi, const float* xscale, const float* wscale, const void* out,
                  const int32_t* status);
 

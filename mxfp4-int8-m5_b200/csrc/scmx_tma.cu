@@ -38,4 +38,22 @@ int make_map_u8(CUtensorMap* map, const void* ptr, int64_t rows, int64_t row_byt
     return SCMX_OK;
 }
 
+// A stack of `planes` byte matrices [rows, row_bytes] (rows `pitch`, planes `plane_pitch` bytes apart, both multiples of 16), box =
+// 128 bytes x box_rows of one plane, 128-byte swizzle, zero fill outside.
+int make_map_planes(CUtensorMap* map, const void* ptr, int64_t planes, int64_t rows, int64_t row_bytes, int64_t pitch, int64_t plane_pitch,
+                    int box_rows) {
+    EncodeTiledFn fn = encode_fn();
+    SCMX_REQUIRE(fn != nullptr, SCMX_ECUDA, "cuTensorMapEncodeTiled is not available from this driver");
+    const cuuint64_t dims[3] = {(cuuint64_t)row_bytes, (cuuint64_t)rows, (cuuint64_t)planes};
+    const cuuint64_t strides[2] = {(cuuint64_t)pitch, (cuuint64_t)plane_pitch};
+    const cuuint32_t box[3] = {128, (cuuint32_t)box_rows, 1};
+    const cuuint32_t estr[3] = {1, 1, 1};
+    const CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_UINT8, 3, const_cast<void*>(ptr), dims, strides, box, estr,
+                          CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                          CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    SCMX_REQUIRE(r == CUDA_SUCCESS, SCMX_ECUDA, "cuTensorMapEncodeTiled failed with CUresult %d (planes=%lld rows=%lld row_bytes=%lld)", (int)r,
+                 (long long)planes, (long long)rows, (long long)row_bytes);
+    return SCMX_OK;
+}
+
 }  // namespace scmx

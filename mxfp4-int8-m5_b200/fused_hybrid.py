@@ -35,6 +35,7 @@ class HybridLayer:
             self.w_in = mix("q", "k", "v", "g")
             self.sizes = [self.H * self.d] * 2 + [self.H * self.dv] * 2
             self.decay = torch.tensor(m["decay"], dtype=torch.float32, device=dev)
+            self.form = 0 if min(m["decay"]) > 0 else 1          # the chunked form works with logarithms of the decays
         else:
             self.H, self.G, self.d, self.dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
             self.scale, self.diff = float(m["scale"]), float(m["diff"])
@@ -87,7 +88,7 @@ class FusedHybrid:
 
     def _retention(self, ly, h, c):
         q, k, v, g = ly.w_in(h).split(ly.sizes, 1)
-        o = X.retention(q, k, v, self.table(ly)[c.offset:], ly.dims, ly.kscale, ly.decay, c.kv)
+        o = X.retention(q, k, v, self.table(ly)[c.offset:], ly.dims, ly.kscale, ly.decay, c.kv, ly.form)
         return X.head_norm_gate(o, g, self.eps)
 
     def _attention(self, ly, h, c):

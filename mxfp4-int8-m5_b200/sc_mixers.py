@@ -151,12 +151,21 @@ def rotary_table(base, dims, rows, device):
     return torch.cat([torch.cos(ang), torch.sin(ang)], 1).float().contiguous()
 
 
-def retention(q, k, v, cs, dims, kscale, decay, state):
-    """q, k [T, H d], v [T, H dv] -> o [T, H, dv] float32; cs: the table rows of this portion; state [H, d, dv] is advanced."""
+RETENTION_TC_MIN = 32       # shorter portions go token by token
+
+
+def retention(q, k, v, cs, dims, kscale, decay, state, form=0):
+    """q, k [T, H d], v [T, H dv] -> o [T, H, dv] float32; cs: the table rows of this portion; state [H, d, dv] is advanced.
+    form: 0 automatic, 1 token by token, 2 chunks on tensor cores (bfloat16, positive decays)."""
     T, (H, d, dv) = q.shape[0], state.shape
     o = torch.empty((T, H, dv), dtype=torch.float32, device=q.device)
+    nbytes = 0
+    if q.dtype == torch.bfloat16 and form != 1 and (form == 2 or T >= RETENTION_TC_MIN):
+        nbytes = 0 if v.data_ptr() % 16 else _lib.mixers().scmx_retention_scratch(T, H, d, dv, dims, _ld(v))
+    assert nbytes or form != 2, "no tensor-core form for these sizes"
+    scratch = torch.empty(nbytes, dtype=torch.uint8, device=q.device) if nbytes else None
     _lib.mcall("scmx_retention", _lib.ptr(q), _ld(q), _lib.ptr(k), _ld(k), _lib.ptr(v), _ld(v), _dt(q), T, H, d, dv, _lib.ptr(cs), dims, kscale,
-               _lib.ptr(decay), _lib.ptr(state), _lib.ptr(o), _lib.stream())
+               _lib.ptr(decay), _lib.ptr(state), _lib.ptr(o), _lib.ptr(scratch), nbytes, _lib.ptr(_lib.mixer_status_buffer()), _lib.stream())
     return o
 
 
@@ -184,12 +193,13 @@ def qk_norm_append(q, k, v, H, G, qw, kw, eps, cache, q_dtype, pos_dev=None):
     return qo
 
 
-def diff_attention(q, cache, H, G, scale, lam, diff, eps):
-    """q [2 H, T, d] at positions cache.offset .. (their keys and values already in the cache) -> [T, H dv]."""
+def diff_attention(q, cache, H, G, scale, lam, diff, eps, form=0):
+    """q [2 H, T, d] at positions cache.offset .. (their keys and values already in the cache) -> [T, H dv].  form: 0 automatic,
+    1 CUDA cores, 2 tensor cores."""
     T, d, dv = q.shape[1], q.shape[2], cache.v.shape[2]
     o = torch.empty((T, H * dv), dtype=q.dtype, device=q.device)
     _lib.mcall("scmx_diff_attn", _lib.ptr(q), _lib.ptr(cache.k), _lib.ptr(cache.v), _dt(q), T, cache.offset, cache.k.shape[1], H, G, d, dv, scale,
-               lam, diff, eps, _lib.ptr(o), _lib.stream())
+               lam, diff, eps, _lib.ptr(o), form, _lib.ptr(_lib.mixer_status_buffer()), _lib.stream())
     return o
 
 
