@@ -72,16 +72,18 @@ int scmx_qk_norm_append(const void* q, int64_t ldq, const void* k, int64_t ldk, 
  * form: 0 = choose, 1 = CUDA cores (any sizes), 2 = tensor cores (bfloat16, sizes up to 128, multiples of 8; status: int32[4]). */
 int scmx_diff_attn(const void* q, const void* k_cache, const void* v_cache, int dt, int64_t n, int64_t pos, int64_t cap, int H, int G, int d,
                    int dv, float scale, float lambda, float diff, float eps, void* o, int form, int32_t* status, void* stream);
-/* One row of it; part f32 [G, nsplit, 2 H / G, dv + 2], counters int32 [G] (zero before the first call, left at zero), nsplit <= 32. */
+/* One row of it; part f32 [G, nsplit, 2 H / G, dv + 2], counters int32 [H] (zero before the first call, left at zero), nsplit <= 32. */
 int scmx_diff_decode(const float* q, const void* k_cache, const void* v_cache, int dt, int64_t n_pos, const int32_t* pos_dev, int64_t cap,
                      int H, int G, int d, int dv, float scale, float lambda, float diff, float eps, int nsplit, float* part,
                      int32_t* counters, float* o, void* stream);
 
 /* out [M, N] = A [M, K] . W [N, K]^T, bfloat16 operands, float32 accumulation; act 1: xIELU with a_pos = softplus(p) and
  * a_neg = 1/2 + softplus(q).  The pitches are multiples of 8; the output pitch covers N rounded up to 16 bytes (the padding is
- * written).  tile: 0 = choose, 64 / 128 = one CTA per 128 x tile, 256 = CTA pairs.  status: int32[4]. */
+ * written).  tile: 0 = choose, 64 / 128 = one CTA per 128 x tile, 256 = CTA pairs.  splits > 1: K is cut
+ * into that many ranges computed side by side (no activation; part: float [splits][M][N rounded up to 4]), for products with few
+ * output tiles.  status: int32[4]. */
 int scmx_gemm_bf16(const void* A, int64_t lda, const void* W, int64_t ldw, int64_t M, int64_t N, int64_t K, int act, float a_pos, float a_neg,
-                   void* out, int out_f32, int64_t ldo, int tile, int32_t* status, void* stream);
+                   void* out, int out_f32, int64_t ldo, int tile, int splits, float* part, int32_t* status, void* stream);
 /* out [N] = W [N, K] x.  epi 0: plain; 1: xIELU; 2: the first C rows pass the causal convolution + SiLU of scmx_conv_silu.
  * Rows of W are zero padded to a multiple of 8 columns. */
 int scmx_gemv_x(const void* W, int64_t ldw, int dt, const float* x, int64_t N, int64_t K, int epi, float a_pos, float a_neg,

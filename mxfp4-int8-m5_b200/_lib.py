@@ -125,7 +125,8 @@ MIXER_SIGNATURES = {
                        c_int, c_vp, c_vp],
     "scmx_diff_decode": [c_vp, c_vp, c_vp, c_int, c_i64, c_vp, c_i64, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_float, c_int,
                          c_vp, c_vp, c_vp, c_vp],
-    "scmx_gemm_bf16": [c_vp, c_i64, c_vp, c_i64, c_i64, c_i64, c_i64, c_int, c_float, c_float, c_vp, c_int, c_i64, c_int, c_vp, c_vp],
+    "scmx_gemm_bf16": [c_vp, c_i64, c_vp, c_i64, c_i64, c_i64, c_i64, c_int, c_float, c_float, c_vp, c_int, c_i64, c_int, c_int, c_vp,
+                       c_vp, c_vp],
     "scmx_gemv_x": [c_vp, c_i64, c_int, c_vp, c_i64, c_i64, c_int, c_float, c_float, c_vp, c_vp, c_vp, c_int, c_int, c_vp, c_vp],
     "scmx_last_error_string": [],
 }

@@ -23,6 +23,7 @@ struct PrepArgs {
     const int32_t* pos_dev;
     int64_t n, ldq, ldk, ldv, pos, cap;
     int nq, nk, nv, d, dv;           // nq = 2 H, nk = 2 G, nv = G
+    int lpv;                         // lanes per q / k vector in the vector form, 0: element by element
     float eps;
 };
 
@@ -33,6 +34,46 @@ __global__ void __launch_bounds__(256) qk_norm_append_kernel(const PrepArgs<TI, 
     const int64_t t = blockIdx.x;
     const int64_t row = (a.pos_dev != nullptr ? (int64_t)a.pos_dev[0] : a.pos) + t;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    if (a.lpv > 0) {
+        // vectors of at most 256 elements, multiples of 8, aligned: lpv lanes (a power of two) hold 8 elements each
+        const int per = 32 / a.lpv, sub = lane / a.lpv, e = 8 * (lane % a.lpv);
+        for (int u0 = warp * per; u0 < a.nq + a.nk; u0 += 8 * per) {      // uniform over the warp
+            const int u = u0 + sub;
+            const bool ok = u < a.nq + a.nk && e < a.d, isq = u < a.nq;
+            const int j = isq ? u : u - a.nq;
+            float x[8] = {};
+            if (ok) ld8((isq ? a.q + t * a.ldq : a.k + t * a.ldk) + (int64_t)j * a.d + e, x);
+            float ss = 0.0f;
+#pragma unroll
+            for (int i = 0; i < 8; ++i) ss += x[i] * x[i];
+            for (int o = a.lpv / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+            if (!ok) continue;
+            const float inv = rms_inv_f32(ss, a.d, a.eps);
+            float w[8];
+            ld8((isq ? a.qw : a.kw) + e, w);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) x[i] *= inv * w[i];
+            if (isq) {
+                TQ* o = a.qo + ((int64_t)j * a.n + t) * a.d + e;
+                st4(o, x[0], x[1], x[2], x[3]);
+                st4(o + 4, x[4], x[5], x[6], x[7]);
+            } else if (row < a.cap) {
+                TC* o = a.kc + ((int64_t)j * a.cap + row) * a.d + e;
+                st4(o, x[0], x[1], x[2], x[3]);
+                st4(o + 4, x[4], x[5], x[6], x[7]);
+            }
+        }
+        if (row < a.cap)
+            for (int i = 8 * threadIdx.x; i < a.nv * a.dv; i += 2048) {
+                const int j = i / a.dv, f = i - j * a.dv;
+                float x[8];
+                ld8(a.v + t * a.ldv + i, x);
+                TC* o = a.vc + ((int64_t)j * a.cap + row) * a.dv + f;
+                st4(o, x[0], x[1], x[2], x[3]);
+                st4(o + 4, x[4], x[5], x[6], x[7]);
+            }
+        return;
+    }
     for (int u = warp; u < a.nq + a.nk + a.nv; u += 8) {
         if (u < a.nq + a.nk) {
             const bool isq = u < a.nq;
@@ -159,31 +200,51 @@ struct DiffDecodeArgs {
     const float* q;          // [2 H, d]
     const T *k, *v;          // caches
     const int32_t* pos_dev;
-    float* part;             // [G, nsplit, 2 R, dv + 2]: unnormalized output, running maximum (log2), running sum
-    int32_t* counters;       // [G], zero before the first call; left at zero
+    float* part;             // [groups, nsplit, 2 R, dv + 2]: unnormalized output, running maximum (log2), running sum
+    int32_t* counters;       // [groups], zero before the first call; left at zero
     float* o;                // [H dv]
     int64_t n_pos, cap;
-    int H, G, d, dv, nsplit;
+    int H, G, d, dv, nsplit, ct, nch;      // G: groups of query heads, nch of them per key/value head
     float scale, lambda, diff, eps;
+};
+
+// Eight stored values as loaded, converted on use.
+template <typename T> struct Raw8;
+template <> struct Raw8<bf16_t> {
+    uint4 w;
+    __device__ __forceinline__ void load(const bf16_t* p) { w = *reinterpret_cast<const uint4*>(p); }
+    __device__ __forceinline__ void get(float (&x)[8]) const {
+        x[0] = bf16_lo(w.x); x[1] = bf16_hi(w.x); x[2] = bf16_lo(w.y); x[3] = bf16_hi(w.y);
+        x[4] = bf16_lo(w.z); x[5] = bf16_hi(w.z); x[6] = bf16_lo(w.w); x[7] = bf16_hi(w.w);
+    }
+};
+template <> struct Raw8<float> {
+    float4 a, b;
+    __device__ __forceinline__ void load(const float* p) { a = reinterpret_cast<const float4*>(p)[0]; b = reinterpret_cast<const float4*>(p)[1]; }
+    __device__ __forceinline__ void get(float (&x)[8]) const {
+        x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w; x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w;
+    }
 };
 
 constexpr int DD_P = 64;          // positions per tile
 constexpr int DD_MIN_CHUNK = 64;  // positions per split at least
 
-// NV: accumulators per thread, 2 R dv <= 256 NV.  Query vectors of a key/value head: 2 r + m for head r of the group, map m.
-template <typename T, int NV>
+// Query vectors of a key/value head: 2 r + m for head r of the group, map m; QP = their number padded to 4, 8, 16 or 32.  For the
+// weighted values a thread owns columns c and c + CT (CT a power of two, dv <= 2 CT) of every query vector over every
+// (256 / CT)-th position of a tile, so that a value read from shared memory serves all query vectors.
+template <typename T, int QP>
 __global__ void __launch_bounds__(256) diff_decode_kernel(const DiffDecodeArgs<T> a) {
     extern __shared__ __align__(16) float sm[];
     const int d = a.d, dv = a.dv, R = a.H / a.G, Q = 2 * R;
     const int dq = (d + 7) & ~7;
-    float* sq = sm;                          // [Q][dq], zero padded
-    float* sv = sq + Q * dq;                 // [DD_P][dv]
-    float* sp = sv + DD_P * dv;              // [Q][DD_P]
-    float* ml = sp + Q * DD_P;               // [Q][3]
+    float* sp = sm;                          // [DD_P][QP] scores, then weights
+    float* sq = sp + DD_P * QP;              // [Q][dq], zero padded
+    float* sv = sq + Q * dq;                 // [DD_P][dv] values; at the end [groups][QP][2 CT] and the splits' weights
+    __shared__ float ml[QP][3];              // running maximum (log2), running sum, correction
     __shared__ int ticket;
     pdl_launch_dependents();
     pdl_wait();
-    const int g = blockIdx.x, split = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int g = blockIdx.x, kvh = g / a.nch, split = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     int64_t n = a.pos_dev != nullptr ? (int64_t)a.pos_dev[0] + 1 : a.n_pos;
     n = n < 1 ? 1 : (n > a.cap ? a.cap : n);
     int64_t chunk = (n + a.nsplit - 1) / a.nsplit;
@@ -195,27 +256,36 @@ __global__ void __launch_bounds__(256) diff_decode_kernel(const DiffDecodeArgs<T
         const int r = i / dq, e = i - r * dq;
         sq[i] = e < d ? a.q[(int64_t)(g * Q + r) * d + e] * (a.scale * 1.4426950408889634f) : 0.0f;
     }
-    for (int i = tid; i < Q; i += 256) {
-        ml[3 * i] = -INFINITY;
-        ml[3 * i + 1] = 0.0f;
+    for (int i = tid; i < QP; i += 256) {
+        ml[i][0] = -INFINITY;
+        ml[i][1] = 0.0f;
     }
-    float acc[NV];
-    int orow[NV];
+    const int CT = a.ct, col = tid & (CT - 1), grp = tid / CT, groups = 256 / CT;
+    const bool c1 = col + CT < dv;
+    float acc[QP][2];
 #pragma unroll
-    for (int j = 0; j < NV; ++j) {
-        acc[j] = 0.0f;
-        orow[j] = (tid + 256 * j) / dv;
-    }
-    const bool vec = (d & 7) == 0;
-    __syncthreads();
+    for (int r = 0; r < QP; ++r) acc[r][0] = acc[r][1] = 0.0f;
+    const bool vec = (d & 7) == 0, vecv = (dv & 7) == 0 && dv <= 256;
+    const int p = tid >> 2, j4 = tid & 3;    // scores: four lanes per position
     for (int64_t tb = t0; tb < t1; tb += DD_P) {
-        // scores: four lanes per position
-        const int p = tid >> 2, j4 = tid & 3;
+        const int np = (int)min((int64_t)DD_P, t1 - tb);
+        const T* vr = a.v + ((int64_t)kvh * a.cap + tb) * dv;
+        // the tile's values: up to 8 loads of 8 elements per thread, in flight while the scores are computed
+        constexpr int VL = sizeof(T) == 2 ? 8 : 4;
+        Raw8<T> vreg[VL];
+        const int nvec = DD_P * dv / 8;
+        if (vecv) {
+#pragma unroll
+            for (int i = 0; i < VL; ++i)
+                if (tid + 256 * i < nvec && 8 * (tid + 256 * i) < np * dv) vreg[i].load(vr + 8 * (tid + 256 * i));
+        }
+        __syncthreads();                     // queries staged; the previous tile's weights and values are consumed
         const int64_t t = tb + p;
         for (int m = 0; m < 2; ++m) {
-            const T* kr = a.k + ((int64_t)(2 * g + m) * a.cap + (t < t1 ? t : t0)) * d;
+            const T* kr = a.k + ((int64_t)(2 * kvh + m) * a.cap + (t < t1 ? t : t0)) * d;
             for (int r0 = 0; r0 < R; r0 += 4) {
                 float s[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+#pragma unroll 4
                 for (int e = 8 * j4; e < dq; e += 32) {
                     float kv[8];
                     if (vec) ld8(kr + e, kv);
@@ -225,69 +295,96 @@ __global__ void __launch_bounds__(256) diff_decode_kernel(const DiffDecodeArgs<T
 #pragma unroll
                     for (int r = 0; r < 4; ++r)
                         if (r0 + r < R) {
-                            const float* qq = sq + (2 * (r0 + r) + m) * dq + e;
-#pragma unroll
-                            for (int i = 0; i < 8; ++i) s[r] = fmaf(qq[i], kv[i], s[r]);
+                            const float4* qq = reinterpret_cast<const float4*>(sq + (2 * (r0 + r) + m) * dq + e);
+                            const float4 x = qq[0], y = qq[1];
+                            s[r] = fmaf(x.x, kv[0], s[r]); s[r] = fmaf(x.y, kv[1], s[r]); s[r] = fmaf(x.z, kv[2], s[r]); s[r] = fmaf(x.w, kv[3], s[r]);
+                            s[r] = fmaf(y.x, kv[4], s[r]); s[r] = fmaf(y.y, kv[5], s[r]); s[r] = fmaf(y.z, kv[6], s[r]); s[r] = fmaf(y.w, kv[7], s[r]);
                         }
                 }
 #pragma unroll
                 for (int r = 0; r < 4; ++r) {
                     s[r] += __shfl_xor_sync(0xffffffffu, s[r], 1);
                     s[r] += __shfl_xor_sync(0xffffffffu, s[r], 2);
-                    if (j4 == 0 && r0 + r < R) sp[(2 * (r0 + r) + m) * DD_P + p] = t < t1 ? s[r] : -INFINITY;
+                    if (j4 == 0 && r0 + r < R) sp[p * QP + 2 * (r0 + r) + m] = t < t1 ? s[r] : -INFINITY;
                 }
             }
         }
-        const int np = (int)min((int64_t)DD_P, t1 - tb);
-        const T* vr = a.v + ((int64_t)g * a.cap + tb) * dv;
-        if ((dv & 7) == 0) {
-            for (int i = tid * 8; i < DD_P * dv; i += 256 * 8) {
+        if (vecv) {
+#pragma unroll
+            for (int i = 0; i < VL; ++i) {
+                const int o = 8 * (tid + 256 * i);
+                if (o < 8 * nvec) {
+                    float x[8] = {};
+                    if (o < np * dv) vreg[i].get(x);
+                    reinterpret_cast<float4*>(sv + o)[0] = make_float4(x[0], x[1], x[2], x[3]);
+                    reinterpret_cast<float4*>(sv + o)[1] = make_float4(x[4], x[5], x[6], x[7]);
+                }
+            }
+            for (int o = 8 * (tid + 256 * VL); o < 8 * nvec; o += 2048) {
                 float x[8] = {};
-                if (i < np * dv) ld8(vr + i, x);
-                reinterpret_cast<float4*>(sv + i)[0] = make_float4(x[0], x[1], x[2], x[3]);
-                reinterpret_cast<float4*>(sv + i)[1] = make_float4(x[4], x[5], x[6], x[7]);
+                if (o < np * dv) ld8(vr + o, x);
+                reinterpret_cast<float4*>(sv + o)[0] = make_float4(x[0], x[1], x[2], x[3]);
+                reinterpret_cast<float4*>(sv + o)[1] = make_float4(x[4], x[5], x[6], x[7]);
             }
         } else {
             for (int i = tid; i < DD_P * dv; i += 256) sv[i] = i < np * dv ? ldf(vr + i) : 0.0f;
         }
         __syncthreads();
         for (int r = warp; r < Q; r += 8) {
-            const float s0 = sp[r * DD_P + lane], s1 = sp[r * DD_P + 32 + lane], m0 = ml[3 * r];
+            const float s0 = sp[lane * QP + r], s1 = sp[(32 + lane) * QP + r], m0 = ml[r][0];
             const float mn = fmaxf(m0, warp_max(fmaxf(s0, s1)));      // finite: the tile has at least one position
-            const float p0 = exp2f(s0 - mn), p1 = exp2f(s1 - mn), l = warp_sumf(p0 + p1);
-            sp[r * DD_P + lane] = p0;
-            sp[r * DD_P + 32 + lane] = p1;
+            const float p0 = ex2_approx(s0 - mn), p1 = ex2_approx(s1 - mn), l = warp_sumf(p0 + p1);
+            sp[lane * QP + r] = p0;
+            sp[(32 + lane) * QP + r] = p1;
             __syncwarp();
             if (lane == 0) {
-                const float corr = exp2f(m0 - mn);
-                ml[3 * r] = mn;
-                ml[3 * r + 1] = ml[3 * r + 1] * corr + l;
-                ml[3 * r + 2] = corr;
+                const float corr = ex2_approx(m0 - mn);
+                ml[r][0] = mn;
+                ml[r][1] = ml[r][1] * corr + l;
+                ml[r][2] = corr;
             }
         }
         __syncthreads();
 #pragma unroll
-        for (int j = 0; j < NV; ++j) {
-            const int r = orow[j];
+        for (int r = 0; r < QP; ++r)
             if (r < Q) {
-                const float* pp = sp + r * DD_P;
-                const float* vv = sv + (tid + 256 * j - r * dv);
-                float o = acc[j] * ml[3 * r + 2];
-#pragma unroll 8
-                for (int i = 0; i < DD_P; ++i) o = fmaf(pp[i], vv[i * dv], o);
-                acc[j] = o;
+                acc[r][0] *= ml[r][2];
+                acc[r][1] *= ml[r][2];
             }
-        }
-        __syncthreads();
+        if (col < dv)
+#pragma unroll 4
+            for (int i = grp; i < DD_P; i += groups) {
+                const float v0 = sv[i * dv + col], v1 = c1 ? sv[i * dv + col + CT] : 0.0f;
+#pragma unroll
+                for (int r = 0; r < QP; r += 4) {
+                    const float4 w = *reinterpret_cast<const float4*>(sp + i * QP + r);
+                    acc[r][0] = fmaf(w.x, v0, acc[r][0]); acc[r][1] = fmaf(w.x, v1, acc[r][1]);
+                    acc[r + 1][0] = fmaf(w.y, v0, acc[r + 1][0]); acc[r + 1][1] = fmaf(w.y, v1, acc[r + 1][1]);
+                    acc[r + 2][0] = fmaf(w.z, v0, acc[r + 2][0]); acc[r + 2][1] = fmaf(w.z, v1, acc[r + 2][1]);
+                    acc[r + 3][0] = fmaf(w.w, v0, acc[r + 3][0]); acc[r + 3][1] = fmaf(w.w, v1, acc[r + 3][1]);
+                }
+            }
     }
+    // sum over the position groups, then this split's partial state
+    __syncthreads();
+#pragma unroll
+    for (int r = 0; r < QP; ++r)
+        if (r < Q) {
+            sv[(grp * Q + r) * 2 * CT + col] = acc[r][0];
+            sv[(grp * Q + r) * 2 * CT + CT + col] = acc[r][1];
+        }
+    __syncthreads();
     const int ps = dv + 2;
     float* part = a.part + ((int64_t)g * a.nsplit + split) * Q * ps;
-#pragma unroll
-    for (int j = 0; j < NV; ++j)
-        if (orow[j] < Q) part[orow[j] * ps + (tid + 256 * j - orow[j] * dv)] = acc[j];
+    for (int i = tid; i < Q * dv; i += 256) {
+        const int r = i / dv, e = i - r * dv;
+        float s = 0.0f;
+        for (int k = 0; k < groups; ++k) s += sv[(k * Q + r) * 2 * CT + e];
+        part[r * ps + e] = s;
+    }
     for (int r = tid; r < Q; r += 256) {
-        part[r * ps + dv] = ml[3 * r];
-        part[r * ps + dv + 1] = ml[3 * r + 1];
+        part[r * ps + dv] = ml[r][0];
+        part[r * ps + dv + 1] = ml[r][1];
     }
     __threadfence();
     __syncthreads();
@@ -297,30 +394,42 @@ __global__ void __launch_bounds__(256) diff_decode_kernel(const DiffDecodeArgs<T
     __threadfence();
     // the last CTA of this key/value head: weights of the splits, then both maps, the difference, its norm
     const float* pg = a.part + (int64_t)g * a.nsplit * Q * ps;
-    float* cf = sv;                          // [Q][nsplit]: exp2(m_s - m) / sum
+    float* cf = sv;                          // [Q][32]: 2^(m_s - m) / sum
+    float* sx = sv + Q * 32;                 // [R][dv]
     for (int r = warp; r < Q; r += 8) {
         const float m = lane < active ? __ldcg(pg + ((int64_t)lane * Q + r) * ps + dv) : -INFINITY;
         const float l = lane < active ? __ldcg(pg + ((int64_t)lane * Q + r) * ps + dv + 1) : 0.0f;
-        const float mm = warp_max(m), c = lane < active ? exp2f(m - mm) : 0.0f;
+        const float mm = warp_max(m), c = lane < active ? ex2_approx(m - mm) : 0.0f;
         const float sum = warp_sumf(c * l);
         cf[r * 32 + lane] = c / sum;
     }
     __syncthreads();
+    for (int i = tid; i < R * dv; i += 256) {
+        const int r = i / dv, e = i - r * dv;
+        const float* pr = pg + 2 * r * ps + e;
+        float a1 = 0.0f, a2 = 0.0f;
+        for (int s0 = 0; s0 < active; s0 += 8) {
+            float u[8], v[8];
+#pragma unroll
+            for (int s = 0; s < 8; ++s) {
+                const bool ok = s0 + s < active;
+                u[s] = ok ? __ldcg(pr + (int64_t)(s0 + s) * Q * ps) : 0.0f;
+                v[s] = ok ? __ldcg(pr + (int64_t)(s0 + s) * Q * ps + ps) : 0.0f;
+            }
+#pragma unroll
+            for (int s = 0; s < 8; ++s) {
+                a1 = fmaf(cf[(2 * r) * 32 + s0 + s], u[s], a1);
+                a2 = fmaf(cf[(2 * r + 1) * 32 + s0 + s], v[s], a2);
+            }
+        }
+        sx[i] = a1 - a.lambda * a2;
+    }
+    __syncthreads();
     for (int r = warp; r < R; r += 8) {
         float ss = 0.0f;
-        for (int e = lane; e < dv; e += 32) {
-            float a1 = 0.0f, a2 = 0.0f;
-            for (int s = 0; s < active; ++s) {
-                const float* p = pg + ((int64_t)s * Q + 2 * r) * ps + e;
-                a1 = fmaf(cf[(2 * r) * 32 + s], __ldcg(p), a1);
-                a2 = fmaf(cf[(2 * r + 1) * 32 + s], __ldcg(p + ps), a2);
-            }
-            const float x = a1 - a.lambda * a2;
-            a.o[(int64_t)(g * R + r) * dv + e] = x;
-            ss += x * x;
-        }
+        for (int e = lane; e < dv; e += 32) ss += sx[r * dv + e] * sx[r * dv + e];
         const float inv = rms_inv_f32(warp_sumf(ss), dv, a.eps) * (1.0f - a.diff);
-        for (int e = lane; e < dv; e += 32) a.o[(int64_t)(g * R + r) * dv + e] *= inv;
+        for (int e = lane; e < dv; e += 32) a.o[(int64_t)(g * R + r) * dv + e] = sx[r * dv + e] * inv;
     }
     if (tid == 0) a.counters[g] = 0;
 }
@@ -334,24 +443,34 @@ static int run_diff_attn(const DiffAttnArgs<T>& a, cudaStream_t st) {
     return SCMX_OK;
 }
 
-template <typename T, int NV>
-static int run_diff_decode_nv(const DiffDecodeArgs<T>& a, size_t smem, cudaStream_t st) {
-    SCMX_CUDA_OK(cudaFuncSetAttribute(diff_decode_kernel<T, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    SCMX_PDL_OK("diff_decode_kernel", launch_pdl(diff_decode_kernel<T, NV>, dim3(a.G, a.nsplit), dim3(256), smem, st, a));
+template <typename T, int QP>
+static int run_diff_decode_q(const DiffDecodeArgs<T>& a, cudaStream_t st) {
+    const int Q = 2 * (a.H / a.G), groups = 256 / a.ct;
+    size_t stage = (size_t)DD_P * a.dv;                                   // values, group sums, combination share this area
+    stage = stage > (size_t)groups * Q * 2 * a.ct ? stage : (size_t)groups * Q * 2 * a.ct;
+    stage = stage > (size_t)Q * 32 + (size_t)Q / 2 * a.dv ? stage : (size_t)Q * 32 + (size_t)Q / 2 * a.dv;
+    const size_t smem = ((size_t)DD_P * QP + (size_t)Q * ((a.d + 7) & ~7) + stage) * 4;
+    SCMX_REQUIRE(smem <= 220 * 1024, SCMX_ELIMIT, "diff_decode: %d query heads per key/value head of sizes %d / %d", Q / 2, a.d, a.dv);
+    SCMX_CUDA_OK(cudaFuncSetAttribute(diff_decode_kernel<T, QP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    SCMX_PDL_OK("diff_decode_kernel", launch_pdl(diff_decode_kernel<T, QP>, dim3(a.G, a.nsplit), dim3(256), smem, st, a));
     return SCMX_OK;
 }
 template <typename T>
-static int run_diff_decode(const DiffDecodeArgs<T>& a, cudaStream_t st) {
-    const int Q = 2 * (a.H / a.G), need = (Q * a.dv + 255) / 256;
-    const size_t stage = (size_t)DD_P * a.dv > (size_t)Q * 32 ? (size_t)DD_P * a.dv : (size_t)Q * 32;
-    const size_t smem = ((size_t)Q * ((a.d + 7) & ~7) + stage + (size_t)Q * DD_P + 3 * Q) * 4;
-    SCMX_REQUIRE(smem <= 220 * 1024 && need <= 64, SCMX_ELIMIT, "diff_decode: %d query heads per key/value head of sizes %d / %d", Q / 2, a.d, a.dv);
-    if (need <= 1) return run_diff_decode_nv<T, 1>(a, smem, st);
-    if (need <= 2) return run_diff_decode_nv<T, 2>(a, smem, st);
-    if (need <= 4) return run_diff_decode_nv<T, 4>(a, smem, st);
-    if (need <= 8) return run_diff_decode_nv<T, 8>(a, smem, st);
-    if (need <= 16) return run_diff_decode_nv<T, 16>(a, smem, st);
-    return run_diff_decode_nv<T, 64>(a, smem, st);
+static int run_diff_decode(DiffDecodeArgs<T> a, cudaStream_t st) {
+    // at most 16 query heads per CTA: larger groups are cut into equal parts that read the same keys and values
+    const int R = a.H / a.G;
+    int part = R < 16 ? R : 16;
+    while (R % part) --part;
+    a.nch = R / part;
+    a.G *= a.nch;
+    const int Q = 2 * part;
+    SCMX_REQUIRE(a.dv <= 512, SCMX_ELIMIT, "diff_decode: %d values per head (512 at most)", a.dv);
+    a.ct = 1;
+    while (2 * a.ct < a.dv) a.ct *= 2;
+    if (Q <= 4) return run_diff_decode_q<T, 4>(a, st);
+    if (Q <= 8) return run_diff_decode_q<T, 8>(a, st);
+    if (Q <= 16) return run_diff_decode_q<T, 16>(a, st);
+    return run_diff_decode_q<T, 32>(a, st);
 }
 
 template <typename TI, typename TC, typename TQ>
@@ -362,6 +481,12 @@ static int run_prep(const void* q, int64_t ldq, const void* k, int64_t ldk, cons
     a.q = (const TI*)q; a.k = (const TI*)k; a.v = (const TI*)v; a.qw = qw; a.kw = kw; a.qo = (TQ*)qo; a.kc = (TC*)kc; a.vc = (TC*)vc;
     a.pos_dev = pos_dev; a.n = n; a.ldq = ldq; a.ldk = ldk; a.ldv = ldv; a.pos = pos; a.cap = cap;
     a.nq = 2 * H; a.nk = 2 * G; a.nv = G; a.d = d; a.dv = dv; a.eps = eps;
+    auto al = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+    a.lpv = 0;
+    if (d % 8 == 0 && d <= 256 && dv % 8 == 0 && ldq % 8 == 0 && ldk % 8 == 0 && ldv % 8 == 0 && al(q) && al(k) && al(v) && al(qw) && al(kw) && al(qo)) {
+        a.lpv = 1;
+        while (8 * a.lpv < d) a.lpv *= 2;
+    }
     SCMX_PDL_OK("qk_norm_append_kernel", launch_pdl(qk_norm_append_kernel<TI, TC, TQ>, dim3((unsigned)n), dim3(256), 0, st, a));
     return SCMX_OK;
 }

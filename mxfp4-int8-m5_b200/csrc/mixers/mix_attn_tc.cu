@@ -41,11 +41,6 @@ struct TaSmem {
     static constexpr int TOTAL = ROW_OFF + 4 * 128 * 4 + 1024;
 };
 
-__device__ __forceinline__ float ex2_approx(float x) {
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
 __device__ __forceinline__ void softmax_bar() { asm volatile("bar.sync 2, 256;" ::: "memory"); }
 
 template <int KB, int VB, int KS>

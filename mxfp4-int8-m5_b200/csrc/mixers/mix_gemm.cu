@@ -14,25 +14,27 @@ struct BgArgs {
     float a_pos, a_neg;          // xIELU: softplus(p), 1/2 + softplus(q)
     void* out;
     int64_t ldo;                 // elements
+    int splits;                  // > 1: K is cut into this many ranges; range s goes to out + s * split_stride (float32, no activation)
+    int64_t split_stride;        // elements
     int32_t* status;
     uint64_t wait_ns;
 };
 
 // Staged 32 rows x 128 bytes -> global memory, full lines, 4 rows per instruction; `valid` bytes of the unit (a multiple of 16).
-__device__ __forceinline__ void bg_drain(const BgArgs& a, const uint8_t* stg, int lane, int row0, size_t row_bytes, size_t col_byte0, int valid) {
+__device__ __forceinline__ void bg_drain(const BgArgs& a, uint8_t* out, const uint8_t* stg, int lane, int row0, size_t row_bytes, size_t col_byte0, int valid) {
     const int piece = lane & 7, rsub = lane >> 3;
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
         const int rl = 4 * i + rsub, row = row0 + rl;
         const uint4 v = *reinterpret_cast<const uint4*>(stg + rl * EPI_PITCH + piece * 16);
         if (row < a.M && piece * 16 < valid)
-            *reinterpret_cast<uint4*>(static_cast<uint8_t*>(a.out) + (size_t)row * row_bytes + col_byte0 + piece * 16) = v;
+            *reinterpret_cast<uint4*>(out + (size_t)row * row_bytes + col_byte0 + piece * 16) = v;
     }
 }
 
 // One warp's 32 rows x BN/2 accumulator columns (see epilogue_warp of the INT8 kernel for the staging layout).
 template <int BN>
-__device__ __forceinline__ void bg_epilogue(const BgArgs& a, uint32_t taddr, int row0, int n0, uint8_t* stg, int lane) {
+__device__ __forceinline__ void bg_epilogue(const BgArgs& a, uint8_t* out, uint32_t taddr, int row0, int n0, uint8_t* stg, int lane) {
     constexpr int CHUNKS = BN / 64;           // 32-column chunks
     uint8_t* my = stg + lane * EPI_PITCH;
     const int esz = a.out_f32 ? 4 : 2;
@@ -54,7 +56,7 @@ __device__ __forceinline__ void bg_epilogue(const BgArgs& a, uint32_t taddr, int
             for (int j = 0; j < 8; ++j) reinterpret_cast<uint4*>(my)[j] = make_uint4(v[4 * j], v[4 * j + 1], v[4 * j + 2], v[4 * j + 3]);
             __syncwarp();
             const int col = n0 + c * 32;
-            bg_drain(a, stg, lane, row0, row_bytes, (size_t)col * 4, min(128, (npad - col) * 4));
+            bg_drain(a, out, stg, lane, row0, row_bytes, (size_t)col * 4, min(128, (npad - col) * 4));
             __syncwarp();
         } else {
             uint4* o = reinterpret_cast<uint4*>(my + 64 * (c & 1));
@@ -68,7 +70,7 @@ __device__ __forceinline__ void bg_epilogue(const BgArgs& a, uint32_t taddr, int
             if ((c & 1) || c + 1 == CHUNKS) {
                 __syncwarp();
                 const int col = n0 + (c & ~1) * 32;
-                bg_drain(a, stg, lane, row0, row_bytes, (size_t)col * 2, min((c & 1) ? 128 : 64, (npad - col) * 2));
+                bg_drain(a, out, stg, lane, row0, row_bytes, (size_t)col * 2, min((c & 1) ? 128 : 64, (npad - col) * 2));
                 __syncwarp();
             }
         }
@@ -141,8 +143,8 @@ __device__ __forceinline__ void gemm_bf16_body(const CUtensorMap& tmA, const CUt
     constexpr int TM_ROWS = PAIR ? 2 * BM : BM;
     const int worker = PAIR ? blockIdx.x >> 1 : blockIdx.x, nworkers = PAIR ? gridDim.x >> 1 : gridDim.x;
     const int tiles_m = (a.M + TM_ROWS - 1) / TM_ROWS, tiles_n = (a.N + BN - 1) / BN;
-    const int total = tiles_m * tiles_n;
-    const int num_kb = (2 * a.K + BK - 1) / BK;
+    const int per_split = tiles_m * tiles_n, total = per_split * a.splits;
+    const int all_kb = (2 * a.K + BK - 1) / BK;
     int fail = 0;
 
     if (warp == 0) {
@@ -150,19 +152,20 @@ __device__ __forceinline__ void gemm_bf16_body(const CUtensorMap& tmA, const CUt
             int stage = 0;
             uint32_t phase = 0;
             for (int t = worker; t < total && fail == 0; t += nworkers) {
-                const int nt = t / tiles_m, mt = t - nt * tiles_m;
+                const int sp = t / per_split, tt = t - sp * per_split, nt = tt / tiles_m, mt = tt - nt * tiles_m;
+                const int kb0 = (int)((int64_t)all_kb * sp / a.splits), num_kb = (int)((int64_t)all_kb * (sp + 1) / a.splits) - kb0;
                 const int row0 = mt * TM_ROWS + (int)rank * BM, brow = nt * BN + (PAIR ? (int)rank * (BN / 2) : 0);
                 for (int kb = 0; kb < num_kb; ++kb) {
                     if (int w = mbar_wait(bar_empty + 8 * stage, phase ^ 1, abort_flag, a.wait_ns)) { fail = w == 1 ? 1 : -1; break; }
                     const uint32_t sa = sbase + stage * L::STAGE_BYTES, sb = sa + L::A_BYTES;
                     if (PAIR) {
                         if (leader) mbar_expect_tx(bar_full + 8 * stage, 2 * L::STAGE_BYTES);
-                        tma_load_2d_pair(sa, &tmA, kb * BK, row0, full_leader + 8 * stage);
-                        tma_load_2d_pair(sb, &tmB, kb * BK, brow, full_leader + 8 * stage);
+                        tma_load_2d_pair(sa, &tmA, (kb0 + kb) * BK, row0, full_leader + 8 * stage);
+                        tma_load_2d_pair(sb, &tmB, (kb0 + kb) * BK, brow, full_leader + 8 * stage);
                     } else {
                         mbar_expect_tx(bar_full + 8 * stage, L::STAGE_BYTES);
-                        tma_load_2d(sa, &tmA, kb * BK, row0, bar_full + 8 * stage);
-                        tma_load_2d(sb, &tmB, kb * BK, brow, bar_full + 8 * stage);
+                        tma_load_2d(sa, &tmA, (kb0 + kb) * BK, row0, bar_full + 8 * stage);
+                        tma_load_2d(sb, &tmB, (kb0 + kb) * BK, brow, bar_full + 8 * stage);
                     }
                     if (++stage == STAGES) { stage = 0; phase ^= 1; }
                 }
@@ -179,6 +182,8 @@ __device__ __forceinline__ void gemm_bf16_body(const CUtensorMap& tmA, const CUt
                 if (w0) { fail = w0 == 1 ? 2 : -1; break; }
                 tc_fence_after();
                 const uint32_t d_tmem = tmem_base + acc * BN;
+                const int sp = t / per_split;
+                const int num_kb = (int)((int64_t)all_kb * (sp + 1) / a.splits) - (int)((int64_t)all_kb * sp / a.splits);
                 for (int kb = 0; kb < num_kb; ++kb) {
                     if (int w = mbar_wait(bar_full + 8 * stage, phase, abort_flag, a.wait_ns)) { fail = w == 1 ? 3 : -1; break; }
                     tc_fence_after();
@@ -205,13 +210,14 @@ __device__ __forceinline__ void gemm_bf16_body(const CUtensorMap& tmA, const CUt
         const int q = warp & 3, chalf = (warp - 2) >> 2;
         uint32_t acc = 0, acc_phase = 0;
         for (int t = worker; t < total && fail == 0; t += nworkers) {
-            const int nt = t / tiles_m, mt = t - nt * tiles_m;
+            const int sp = t / per_split, tt = t - sp * per_split, nt = tt / tiles_m, mt = tt - nt * tiles_m;
+            uint8_t* out = static_cast<uint8_t*>(a.out) + (size_t)sp * a.split_stride * 4;
             const int n0 = nt * BN + chalf * (BN / 2), wrow0 = mt * TM_ROWS + (int)rank * BM + 32 * q;
             if (int w = mbar_wait(bar_tfull + 8 * acc, acc_phase, abort_flag, a.wait_ns)) fail = w == 1 ? 4 : -1;
             epilogue_bar();         // the epilogue threads agree on giving up before anyone touches TMEM
             if (*abort_flag) { if (!fail) fail = -1; break; }
             tc_fence_after();
-            bg_epilogue<BN>(a, tmem_base + acc * BN + chalf * (BN / 2) + ((uint32_t)(32 * q) << 16), wrow0, n0,
+            bg_epilogue<BN>(a, out, tmem_base + acc * BN + chalf * (BN / 2) + ((uint32_t)(32 * q) << 16), wrow0, n0,
                             smem + L::EPI_OFF + (warp - 2) * EPI_STAGE_WARP, lane);
             tc_fence_before();
             __syncwarp();
@@ -276,11 +282,30 @@ static int launch_bg(const void* A, int64_t lda, const void* W, int64_t ldw, con
     rc = make_map_u8(&tmB, W, a.N, 2 * (int64_t)a.K, BK, PAIR ? BN / 2 : BN, 128, 2 * ldw);
     if (rc) return rc;
     constexpr int rows = PAIR ? 2 * BM : BM;
-    const int64_t tiles = ((a.M + rows - 1) / rows) * (int64_t)((a.N + BN - 1) / BN);
+    const int64_t tiles = ((a.M + rows - 1) / rows) * (int64_t)((a.N + BN - 1) / BN) * a.splits;
     int workers = PAIR ? sm_count() / 2 : sm_count();
     if (tiles < workers) workers = (int)tiles;
     SCMX_PDL_OK("gemm_bf16", launch_pdl(kernel, dim3(PAIR ? 2 * workers : workers), dim3(CTA_THREADS), (size_t)L::TOTAL, st, tmA, tmB, a));
     return SCMX_OK;
+}
+
+// Sum of the K ranges' partial products, in order of the ranges -> the output type.
+__global__ void __launch_bounds__(256) gemm_reduce_kernel(const float* part, int splits, int64_t stride, int64_t rows, int quads, int64_t ldp,
+                                                          int out_f32, void* out, int64_t ldo) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int64_t i = (int64_t)blockIdx.x * 256 + threadIdx.x;
+    if (i >= rows * quads) return;
+    const int64_t r = i / quads;
+    const int c = 4 * (int)(i - r * quads);
+    float4 s = make_float4(0, 0, 0, 0);
+#pragma unroll 8
+    for (int k = 0; k < splits; ++k) {
+        const float4 v = __ldcg(reinterpret_cast<const float4*>(part + k * stride + r * ldp + c));
+        s.x += v.x; s.y += v.y; s.z += v.z; s.w += v.w;
+    }
+    if (out_f32) st4(static_cast<float*>(out) + r * ldo + c, s.x, s.y, s.z, s.w);
+    else st4(static_cast<bf16_t*>(out) + r * ldo + c, s.x, s.y, s.z, s.w);
 }
 
 }  // namespace scmx
@@ -288,7 +313,8 @@ static int launch_bg(const void* A, int64_t lda, const void* W, int64_t ldw, con
 using namespace scmx;
 
 extern "C" int scmx_gemm_bf16(const void* A, int64_t lda, const void* W, int64_t ldw, int64_t M, int64_t N, int64_t K, int act, float a_pos,
-                              float a_neg, void* out, int out_f32, int64_t ldo, int tile, int32_t* status, void* stream) {
+                              float a_neg, void* out, int out_f32, int64_t ldo, int tile, int splits, float* part, int32_t* status,
+                              void* stream) {
     SCMX_REQUIRE(A && W && out && status, SCMX_EINVAL, "gemm_bf16: null buffer");
     SCMX_REQUIRE(M >= 0 && N > 0 && K > 0 && M < (1ll << 30) && N < (1ll << 30) && K < (1ll << 29), SCMX_EINVAL, "gemm_bf16: M=%lld N=%lld K=%lld",
                  (long long)M, (long long)N, (long long)K);
@@ -302,12 +328,25 @@ extern "C" int scmx_gemm_bf16(const void* A, int64_t lda, const void* W, int64_t
     if (M == 0) return SCMX_OK;
     BgArgs a;
     a.M = (int)M; a.N = (int)N; a.K = (int)K; a.out_f32 = out_f32 ? 1 : 0; a.act = act; a.a_pos = a_pos; a.a_neg = a_neg;
-    a.out = out; a.ldo = ldo; a.status = status; a.wait_ns = g_wait_limit_ns;
+    a.out = out; a.ldo = ldo; a.status = status; a.wait_ns = g_wait_limit_ns; a.splits = 1; a.split_stride = 0;
     const cudaStream_t st = (cudaStream_t)stream;
     if (tile == 0) {
         const int64_t m = (M + 127) / 128;
         if (M > 128 && N >= 256 && ((M + 255) / 256) * ((N + 255) / 256) * 2 >= sm_count() / 2) tile = 256;
         else tile = m * ((N + 127) / 128) >= sm_count() / 2 ? 128 : 64;
+    }
+    if (splits > 1) {
+        SCMX_REQUIRE(part && ((uintptr_t)part & 15) == 0 && act == 0 && splits <= (2 * K + BK - 1) / BK, SCMX_EINVAL,
+                     "gemm_bf16: %d ranges of K=%lld need a buffer and no activation", splits, (long long)K);
+        const int64_t ldp = (N + 3) / 4 * 4;
+        a.out = part; a.out_f32 = 1; a.ldo = ldp; a.splits = splits; a.split_stride = M * ldp;
+        const int rc = tile == 256 ? launch_bg<256, 5, true>(A, lda, W, ldw, a, st)
+                     : tile == 128 ? launch_bg<128, 5, false>(A, lda, W, ldw, a, st) : launch_bg<64, 7, false>(A, lda, W, ldw, a, st);
+        if (rc) return rc;
+        const int quads = (int)(ldp / 4);
+        SCMX_PDL_OK("gemm_reduce_kernel", launch_pdl(gemm_reduce_kernel, dim3((unsigned)((M * quads + 255) / 256)), dim3(256), 0, st, (const float*)part,
+                                                     splits, a.split_stride, M, quads, ldp, out_f32 ? 1 : 0, out, ldo));
+        return SCMX_OK;
     }
     if (tile == 256) return launch_bg<256, 5, true>(A, lda, W, ldw, a, st);
     if (tile == 128) return launch_bg<128, 5, false>(A, lda, W, ldw, a, st);

@@ -68,9 +68,15 @@ __global__ void __launch_bounds__(256) gemv_x_kernel(const GvArgs a) {
     };
     fetch(first);
     pdl_wait();
-    for (int i = tid; i < nv * 8; i += 256) {
-        const float x = i < a.K ? a.x[i] : 0.0f;
-        reinterpret_cast<float*>(xs + ((i >> 2) & 1) * nv + (i >> 3))[i & 3] = x;
+    if ((a.K & 3) == 0 && ((uintptr_t)a.x & 15) == 0) {
+#pragma unroll 8
+        for (int i = tid; i < 2 * nv; i += 256)
+            xs[(i & 1) * nv + (i >> 1)] = 4 * i < a.K ? *reinterpret_cast<const float4*>(a.x + 4 * i) : make_float4(0, 0, 0, 0);
+    } else {
+        for (int i = tid; i < nv * 8; i += 256) {
+            const float x = i < a.K ? a.x[i] : 0.0f;
+            reinterpret_cast<float*>(xs + ((i >> 2) & 1) * nv + (i >> 3))[i & 3] = x;
+        }
     }
     __syncthreads();
     float s[GV_ROWS] = {};

@@ -111,21 +111,40 @@ __global__ void __launch_bounds__(256) retention_step_kernel(const RetStepArgs a
     const int h = blockIdx.y, rank = (int)cl.block_rank(), nc = (int)cl.num_blocks(), tid = threadIdx.x;
     const int64_t pos = min(a.pos_dev != nullptr ? (int64_t)a.pos_dev[0] : a.pos, a.cs_rows - 1);
     const float* cs = a.cs + pos * a.dims;
+    const int e0 = rank * a.cw, cw = min(a.cw, a.dv - e0);      // cw may be <= 0 on a trailing rank
+    const int groups = cw > 0 ? 256 / cw : 0;
+    const int grp = cw > 0 ? tid / cw : 0, col = cw > 0 ? tid - grp * cw : 0;
+    const bool work = grp < groups;
+    const float decay = a.decay[h];
+    // the first rows of this thread's column, its value and gate are requested before q and k are staged
+    constexpr int PRE = 16;
+    float* S = a.state + (int64_t)h * a.d * a.dv + e0 + col;
+    float pre[PRE], v = 0.0f;
+#pragma unroll
+    for (int j = 0; j < PRE; ++j) {
+        const int i = grp + j * groups;
+        pre[j] = work && i < a.d ? S[(int64_t)i * a.dv] : 0.0f;
+    }
+    if (work) v = a.v[(int64_t)h * a.dv + e0 + col];
+    const float gate = tid < cw ? a.g[(int64_t)h * a.dv + e0 + tid] : 0.0f;
     for (int i = tid; i < a.d; i += 256) {
         sq[i] = rotated(a.q + (int64_t)h * a.d, i, a.dims, cs);
         sk[i] = rotated(a.k + (int64_t)h * a.d, i, a.dims, cs) * a.kscale;
     }
     __syncthreads();
-    const int e0 = rank * a.cw, cw = min(a.cw, a.dv - e0);      // cw may be <= 0 on a trailing rank
-    const int groups = cw > 0 ? 256 / cw : 0;
-    const int grp = cw > 0 ? tid / cw : 0, col = cw > 0 ? tid - grp * cw : 0;
-    const float decay = a.decay[h];
     float part = 0.0f;
-    if (grp < groups) {
-        const float v = a.v[(int64_t)h * a.dv + e0 + col];
-        float* S = a.state + (int64_t)h * a.d * a.dv + e0 + col;
+    if (work) {
+#pragma unroll
+        for (int j = 0; j < PRE; ++j) {
+            const int i = grp + j * groups;
+            if (i < a.d) {
+                const float s = fmaf(decay, pre[j], sk[i] * v);
+                S[(int64_t)i * a.dv] = s;
+                part = fmaf(sq[i], s, part);
+            }
+        }
 #pragma unroll 8
-        for (int i = grp; i < a.d; i += groups) {
+        for (int i = grp + PRE * groups; i < a.d; i += groups) {
             const float s = fmaf(decay, S[(int64_t)i * a.dv], sk[i] * v);
             S[(int64_t)i * a.dv] = s;
             part = fmaf(sq[i], s, part);
@@ -147,7 +166,7 @@ __global__ void __launch_bounds__(256) retention_step_kernel(const RetStepArgs a
     }
     if (tid < cw) {
         const int64_t i = (int64_t)h * a.dv + e0 + tid;
-        a.y[i] = o * rms_inv_f32(total, a.dv, a.eps) * silu_f32(a.g[i]);
+        a.y[i] = o * rms_inv_f32(total, a.dv, a.eps) * silu_f32(gate);
     }
 }
 

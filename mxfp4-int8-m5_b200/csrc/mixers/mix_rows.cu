@@ -128,41 +128,72 @@ __global__ void __launch_bounds__(256) norm_rows_kernel(const float* x, const in
 }
 
 // ---- causal depthwise convolution + SiLU --------------------------------------------------------------------------------
-constexpr int CONV_T = 16;      // tokens per thread
+constexpr int CONV_T = 8;       // tokens per thread
 
-// TAPS > 0: window in registers; TAPS = 0: any number of taps, inputs re-read.
+// TAPS > 0: two channels per thread, all inputs of the thread's tokens in registers; TAPS = 0: one channel, any number of taps.
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(256) conv_silu_kernel(const T* x, int64_t ldx, int64_t n_tok, int C, int taps, const float* w,
                                                         const float* b, const float* tail, T* out, int64_t ldo) {
     pdl_launch_dependents();
     pdl_wait();
-    const int c = blockIdx.x * 256 + threadIdx.x;
-    if (c >= C) return;
     const int64_t t0 = (int64_t)blockIdx.y * CONV_T;
     const int64_t t1 = t0 + CONV_T < n_tok ? t0 + CONV_T : n_tok;
-    const int K = TAPS > 0 ? TAPS : taps;
-    // input of token t, which may lie before this portion (then it is part of the carried tail)
-    auto in = [&](int64_t t) -> float { return t >= 0 ? ldf(x + t * ldx + c) : tail[(int64_t)c * (K - 1) + (t + K - 1)]; };
-    const float bias = b[c];
     if (TAPS > 0) {
-        float win[TAPS > 0 ? TAPS : 1], ww[TAPS > 0 ? TAPS : 1];
+        constexpr int W = CONV_T + (TAPS > 0 ? TAPS : 1) - 1;
+        const int c = 2 * (blockIdx.x * 256 + threadIdx.x);
+        if (c >= C) return;
+        // C is even and rows are 2-element aligned (host side); a token before this portion lies in the carried tail
+        float2 in[W];
+        if (t0 >= TAPS - 1 && t1 == t0 + CONV_T) {
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j) ww[j] = w[(int64_t)c * TAPS + j];
+            for (int i = 0; i < W; ++i) {
+                const T* p = x + (t0 - (TAPS - 1) + i) * ldx + c;
+                if (sizeof(T) == 2) {
+                    const uint32_t u = *reinterpret_cast<const uint32_t*>(p);
+                    in[i] = make_float2(bf16_lo(u), bf16_hi(u));
+                } else {
+                    in[i] = make_float2(ldf(p), ldf(p + 1));
+                }
+            }
+        } else {
 #pragma unroll
-        for (int j = 1; j < TAPS; ++j) win[j] = in(t0 - TAPS + j);
-        for (int64_t t = t0; t < t1; ++t) {
+            for (int i = 0; i < W; ++i) {
+                const int64_t t = t0 - (TAPS - 1) + i;
+                in[i] = make_float2(0.0f, 0.0f);
+                if (t >= 0 && t < t1) in[i] = make_float2(ldf(x + t * ldx + c), ldf(x + t * ldx + c + 1));
+                if (t < 0) in[i] = make_float2(tail[(int64_t)c * (TAPS - 1) + t + TAPS - 1], tail[(int64_t)(c + 1) * (TAPS - 1) + t + TAPS - 1]);
+            }
+        }
+        const float2 bias = make_float2(b[c], b[c + 1]);
+        float2 ww[TAPS > 0 ? TAPS : 1];
 #pragma unroll
-            for (int j = 0; j + 1 < TAPS; ++j) win[j] = win[j + 1];
-            win[TAPS > 0 ? TAPS - 1 : 0] = ldf(x + t * ldx + c);
-            float s = bias;
+        for (int j = 0; j < TAPS; ++j) ww[j] = make_float2(w[(int64_t)c * TAPS + j], w[(int64_t)(c + 1) * TAPS + j]);
 #pragma unroll
-            for (int j = 0; j < TAPS; ++j) s = fmaf(ww[j], win[j], s);
-            stf(out + t * ldo + c, silu_f32(s));
+        for (int i = 0; i < CONV_T; ++i) {
+            if (t0 + i >= t1) break;
+            float2 s = bias;
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) {
+                s.x = fmaf(ww[j].x, in[i + j].x, s.x);
+                s.y = fmaf(ww[j].y, in[i + j].y, s.y);
+            }
+            T* o = out + (t0 + i) * ldo + c;
+            if (sizeof(T) == 2) {
+                *reinterpret_cast<uint32_t*>(o) = pack_bf16x2(silu_f32(s.x), silu_f32(s.y));
+            } else {
+                stf(o, silu_f32(s.x));
+                stf(o + 1, silu_f32(s.y));
+            }
         }
     } else {
+        const int c = blockIdx.x * 256 + threadIdx.x;
+        if (c >= C) return;
         for (int64_t t = t0; t < t1; ++t) {
-            float s = bias;
-            for (int j = 0; j < K; ++j) s = fmaf(w[(int64_t)c * K + j], in(t - (K - 1) + j), s);
+            float s = b[c];
+            for (int j = 0; j < taps; ++j) {
+                const int64_t u = t - (taps - 1) + j;
+                s = fmaf(w[(int64_t)c * taps + j], u >= 0 ? ldf(x + u * ldx + c) : tail[(int64_t)c * (taps - 1) + (u + taps - 1)], s);
+            }
             stf(out + t * ldo + c, silu_f32(s));
         }
     }
@@ -186,7 +217,7 @@ __global__ void __launch_bounds__(256) conv_tail_kernel(const T* x, int64_t ldx,
 // out[t, h, :] = o[t, h, :] / rms * silu(g[t, h, :]); one warp per (token, head).
 template <typename T>
 __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* o, const T* g, int64_t ldg, int64_t n, int H, int dv, float eps,
-                                                             T* out) {
+                                                             int vec, T* out) {
     pdl_launch_dependents();
     pdl_wait();
     const int64_t i = (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5);
@@ -197,6 +228,24 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* o, con
     const float* p = o + i * dv;
     const T* gp = g + t * ldg + (int64_t)h * dv;
     float ss = 0.0f;
+    if (vec) {                      // rows of four aligned values; up to 4 groups per lane stay in registers
+        float4 v[4], gv[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int e = 4 * (lane + 32 * j);
+            v[j] = e < dv ? *reinterpret_cast<const float4*>(p + e) : make_float4(0, 0, 0, 0);
+            gv[j] = e < dv ? ld4(gp + e) : make_float4(0, 0, 0, 0);
+            ss += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
+        }
+        const float inv = rms_inv_f32(warp_sumf(ss), dv, eps);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int e = 4 * (lane + 32 * j);
+            if (e < dv) st4(out + i * dv + e, v[j].x * inv * silu_f32(gv[j].x), v[j].y * inv * silu_f32(gv[j].y), v[j].z * inv * silu_f32(gv[j].z),
+                            v[j].w * inv * silu_f32(gv[j].w));
+        }
+        return;
+    }
     for (int e = lane; e < dv; e += 32) ss += p[e] * p[e];
     const float inv = rms_inv_f32(warp_sumf(ss), dv, eps);
     for (int e = lane; e < dv; e += 32) stf(out + i * dv + e, p[e] * inv * silu_f32(ldf(gp + e)));
@@ -237,11 +286,13 @@ static int run_res_norm(const ResNormArgs& a, int64_t T_, cudaStream_t st) {
 template <typename T>
 static int run_conv(const T* x, int64_t ldx, int64_t n_tok, int C, int taps, const float* w, const float* b, float* tail, T* out,
                     int64_t ldo, cudaStream_t st) {
-    const dim3 grid((C + 255) / 256, (unsigned)((n_tok + CONV_T - 1) / CONV_T)), block(256);
+    const bool pairs = C % 2 == 0 && ldx % 2 == 0 && ldo % 2 == 0 && ((uintptr_t)x & 3) == 0 && taps <= 4;
+    const int per = pairs ? 512 : 256;
+    const dim3 grid((C + per - 1) / per, (unsigned)((n_tok + CONV_T - 1) / CONV_T)), block(256);
     const float* ct = tail;
     cudaError_t e;
 #define CASE(n) case n: e = launch_pdl(conv_silu_kernel<T, n>, grid, block, 0, st, x, ldx, n_tok, C, taps, w, b, ct, out, ldo); break
-    switch (taps) {
+    switch (pairs ? taps : 0) {
         CASE(1); CASE(2); CASE(3); CASE(4);
         default: e = launch_pdl(conv_silu_kernel<T, 0>, grid, block, 0, st, x, ldx, n_tok, C, taps, w, b, ct, out, ldo);
     }
@@ -307,12 +358,14 @@ extern "C" int scmx_head_norm_gate(const float* o, const void* g, int64_t ldg, i
     SCMX_REQUIRE(o && g && out && T >= 0 && H > 0 && dv > 0 && ldg >= (int64_t)H * dv, SCMX_EINVAL, "head_norm_gate: bad argument");
     if (T == 0) return SCMX_OK;
     const int64_t n = T * H;
+    const int esz = dt == 0 ? 2 : 4;
+    const int vec = dv % 4 == 0 && dv <= 512 && ldg % 4 == 0 && (uintptr_t)g % (4 * esz) == 0;
     const dim3 grid((unsigned)((n + 7) / 8)), block(256);
     const cudaStream_t st = (cudaStream_t)stream;
     if (dt == 0)
-        SCMX_PDL_OK("head_norm_gate_kernel", launch_pdl(head_norm_gate_kernel<bf16_t>, grid, block, 0, st, o, (const bf16_t*)g, ldg, n, H, dv, eps, (bf16_t*)out));
+        SCMX_PDL_OK("head_norm_gate_kernel", launch_pdl(head_norm_gate_kernel<bf16_t>, grid, block, 0, st, o, (const bf16_t*)g, ldg, n, H, dv, eps, vec, (bf16_t*)out));
     else
-        SCMX_PDL_OK("head_norm_gate_kernel", launch_pdl(head_norm_gate_kernel<float>, grid, block, 0, st, o, (const float*)g, ldg, n, H, dv, eps, (float*)out));
+        SCMX_PDL_OK("head_norm_gate_kernel", launch_pdl(head_norm_gate_kernel<float>, grid, block, 0, st, o, (const float*)g, ldg, n, H, dv, eps, vec, (float*)out));
     return SCMX_OK;
 }
 

@@ -34,7 +34,8 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(const ScanArgs<T> a) {
     constexpr int SC_T = NP > 128 ? 16 : 32;      // tokens per tile
     constexpr int XE = (SC_T * CPC + SC_THREADS - 1) / SC_THREADS;      // staged x / dt / z values per thread and tile
     constexpr int BE = (SC_T * NP + SC_THREADS - 1) / SC_THREADS;
-    __shared__ __align__(16) float sx[SC_T][CPC], sdt[SC_T][CPC], sz[SC_T][CPC];
+    __shared__ __align__(16) float2 sd[SC_T][CPC];       // step, step * x
+    __shared__ __align__(16) float2 so[SC_T][CPC];       // D x, silu(z)
     __shared__ __align__(16) float sB[SC_T][NP], sC[SC_T][NP];
     __shared__ float sy[SC_T][CPC + 1];
     pdl_launch_dependents();
@@ -57,23 +58,24 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(const ScanArgs<T> a) {
     const int fc = tid % CPC, fr = tid / CPC;
     const bool fok = c0 + fc < a.C;
     const float bias = fok ? a.dt_bias[c0 + fc] : 0.0f, Dc = fok ? a.D[c0 + fc] : 0.0f;
-    float px[XE], pd[XE], pz[XE], pB[BE], pC[BE];
+    float pd[XE];
+    T px[XE], pz[XE], pB[BE], pC[BE];       // as stored: converted when staged, so that the loads stay in flight
     auto fetch = [&](int64_t t0) {
 #pragma unroll
         for (int i = 0; i < XE; ++i) {
             const int64_t t = t0 + fr + i * FS;
             const bool ok = fok && fr + i * FS < SC_T && t < a.n;
-            px[i] = ok ? ldf(a.x + t * a.ldx + c0 + fc) : 0.0f;
+            px[i] = ok ? a.x[t * a.ldx + c0 + fc] : T(0);
             pd[i] = ok ? a.dtp[t * a.ldt + c0 + fc] : 0.0f;
-            pz[i] = ok ? ldf(a.z + t * a.ldz + c0 + fc) : 0.0f;
+            pz[i] = ok ? a.z[t * a.ldz + c0 + fc] : T(0);
         }
 #pragma unroll
         for (int i = 0; i < BE; ++i) {
             const int e = tid + i * SC_THREADS, r = e / NP, n = e % NP;
             const int64_t t = t0 + r;
             const bool ok = r < SC_T && n < a.N && t < a.n;
-            pB[i] = ok ? ldf(a.bc + t * a.ldbc + n) : 0.0f;
-            pC[i] = ok ? ldf(a.bc + t * a.ldbc + a.N + n) : 0.0f;
+            pB[i] = ok ? a.bc[t * a.ldbc + n] : T(0);
+            pC[i] = ok ? a.bc[t * a.ldbc + a.N + n] : T(0);
         }
     };
     fetch(0);
@@ -82,39 +84,63 @@ __global__ void __launch_bounds__(SC_THREADS) scan_kernel(const ScanArgs<T> a) {
         for (int i = 0; i < XE; ++i) {
             const int r = fr + i * FS;
             if (r >= SC_T) break;
-            sx[r][fc] = px[i];
-            sdt[r][fc] = t0 + r < a.n ? softplus_f32(pd[i] + bias) : 0.0f;      // a zero step leaves the state unchanged
-            sz[r][fc] = pz[i];
+            // a zero step leaves the state unchanged
+            const float step = t0 + r < a.n ? softplus_f32(pd[i] + bias) : 0.0f, x = ldf(&px[i]);
+            sd[r][fc] = make_float2(step, step * x);
+            so[r][fc] = make_float2(Dc * x, silu_f32(ldf(&pz[i])));
         }
 #pragma unroll
         for (int i = 0; i < BE; ++i) {
             const int e = tid + i * SC_THREADS;
             if (e < SC_T * NP) {
-                sB[e / NP][e % NP] = pB[i];
-                sC[e / NP][e % NP] = pC[i];
+                sB[e / NP][e % NP] = ldf(&pB[i]);
+                sC[e / NP][e % NP] = ldf(&pC[i]);
             }
         }
         __syncthreads();
         if (t0 + SC_T < a.n) fetch(t0 + SC_T);
-#pragma unroll 4
-        for (int r = 0; r < SC_T; ++r) {
-            const float dt = sdt[r][ch], dx = dt * sx[r][ch];
-            float y = 0.0f;
+        // eight tokens at a time: everything but the chain through S is independent; the partial outputs of the channel's lanes
+        // are summed by halving (a lane keeps half of the tokens and hands over the other half), 7 shuffles for 8 tokens
+#pragma unroll 1
+        for (int r0 = 0; r0 < SC_T; r0 += 8) {
+            float y[8];
 #pragma unroll
-            for (int i = 0; i < NS; ++i) {
-                S[i] = fmaf(exp2f(dt * A2[i]), S[i], dx * sB[r][lane * NS + i]);
-                y = fmaf(S[i], sC[r][lane * NS + i], y);
+            for (int u = 0; u < 8; ++u) {
+                const float2 d = sd[r0 + u][ch];
+                y[u] = 0.0f;
+#pragma unroll
+                for (int i = 0; i < NS; ++i) {
+                    S[i] = fmaf(ex2_approx(d.x * A2[i]), S[i], d.y * sB[r0 + u][lane * NS + i]);
+                    y[u] = fmaf(S[i], sC[r0 + u][lane * NS + i], y[u]);
+                }
             }
+            int first = 0;                  // the token(s) whose sum this lane ends up with
 #pragma unroll
-            for (int o = LPC / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-            if (lane == 0) sy[r][ch] = y;
+            for (int o = 1, cnt = 8; o < LPC; o *= 2) {
+                if (cnt > 1) {
+                    cnt /= 2;
+                    const bool up = lane & o;
+#pragma unroll
+                    for (int u = 0; u < cnt; ++u) {
+                        const float give = up ? y[u] : y[u + cnt], keep = up ? y[u + cnt] : y[u];
+                        y[u] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+                    }
+                    first += up ? cnt : 0;
+                } else {
+                    y[0] += __shfl_xor_sync(0xffffffffu, y[0], o);
+                }
+            }
+            constexpr int OUT = LPC >= 8 ? 1 : 8 / LPC;
+            if (lane < 8)
+#pragma unroll
+                for (int u = 0; u < OUT; ++u) sy[r0 + first + u][ch] = y[u];
         }
         __syncthreads();
 #pragma unroll
         for (int i = 0; i < XE; ++i) {
             const int r = fr + i * FS;
             const int64_t t = t0 + r;
-            if (fok && r < SC_T && t < a.n) stf(a.y + t * a.ldy + c0 + fc, (sy[r][fc] + Dc * sx[r][fc]) * silu_f32(sz[r][fc]));
+            if (fok && r < SC_T && t < a.n) stf(a.y + t * a.ldy + c0 + fc, (sy[r][fc] + so[r][fc].x) * so[r][fc].y);
         }
         __syncthreads();
     }
@@ -169,7 +195,7 @@ __global__ void __launch_bounds__(256) scan_step_kernel(const ScanStepArgs a) {
     if (ok) {
         float* S = a.state + (int64_t)c * a.N;
         for (int n = lane; n < a.N; n += SS_LANES) {
-            const float s = fmaf(exp2f(dt * a.A2[(int64_t)c * a.N + n]), S[n], dx * sdbc[a.R + n]);
+            const float s = fmaf(ex2_approx(dt * a.A2[(int64_t)c * a.N + n]), S[n], dx * sdbc[a.R + n]);
             S[n] = s;
             y = fmaf(s, sdbc[a.R + a.N + n], y);
         }

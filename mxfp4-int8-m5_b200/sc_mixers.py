@@ -53,7 +53,12 @@ class Linear:
             self.w[:, :self.K] = w
         self.dt = _dt(w)
 
-    def __call__(self, x, out_dtype=None, act=None, tile=0):
+    def _splits(self, M):
+        """Ranges of K computed side by side when the output has few tiles (at least 512 of K each)."""
+        tiles = -(-M // 128) * -(-self.N // 64)
+        return max(1, min(8, self.K // 512, 148 // tiles)) if tiles <= 74 else 1
+
+    def __call__(self, x, out_dtype=None, act=None, tile=0, splits=None):
         """x [M, K] -> [M, N] in out_dtype (default: the weights' type)."""
         out_dtype = out_dtype or self.w.dtype
         M = x.shape[0]
@@ -67,9 +72,12 @@ class Linear:
         if _ld(x) % 8 or x.data_ptr() % 16:
             x = empty_rows(M, self.K, x.dtype, x.device).copy_(x)
         y = empty_rows(M, self.N, out_dtype, x.device)
+        if splits is None:
+            splits = 1 if act is not None else self._splits(M)
+        part = torch.empty(splits * M * ((self.N + 3) // 4 * 4), dtype=torch.float32, device=x.device) if splits > 1 else None
         _lib.mcall("scmx_gemm_bf16", _lib.ptr(x), _ld(x), _lib.ptr(self.w), self.w.shape[1], M, self.N, self.K, int(act is not None),
-                   act.a_pos if act else 0.0, act.a_neg if act else 0.0, _lib.ptr(y), int(out_dtype == torch.float32), _round8(self.N), tile,
-                   _lib.ptr(_lib.mixer_status_buffer()), _lib.stream())
+                   act.a_pos if act else 0.0, act.a_neg if act else 0.0, _lib.ptr(y), int(out_dtype == torch.float32), _round8(self.N), tile, splits,
+                   _lib.ptr(part), _lib.ptr(_lib.mixer_status_buffer()), _lib.stream())
         return y
 
     def vec(self, x, act=None, conv=None, out=None):
@@ -208,9 +216,9 @@ class DiffDecodeAttention:
 
     def __init__(self, H, G, d, dv, device, n_sm=148):
         self.H, self.G, self.d, self.dv = H, G, d, dv
-        self.nsplit = max(1, min(32, n_sm // G))
+        self.nsplit = max(1, min(32, 2 * n_sm // G))
         self.part = torch.empty((G, self.nsplit, 2 * (H // G), dv + 2), dtype=torch.float32, device=device)
-        self.counters = torch.zeros(G, dtype=torch.int32, device=device)
+        self.counters = torch.zeros(H, dtype=torch.int32, device=device)
 
     def __call__(self, q, cache, scale, lam, diff, eps, o, n_pos=None, pos_dev=None):
         _lib.mcall("scmx_diff_decode", _lib.ptr(q), _lib.ptr(cache.k), _lib.ptr(cache.v), _dt(cache.k), int(n_pos or 0), _lib.ptr(pos_dev),

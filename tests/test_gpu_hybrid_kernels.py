@@ -48,6 +48,14 @@ def test_gemm(X, M, N, K, tile, out):
     assert err(y, npy(x) @ npy(w).T) < (2e-2 if out == BF else 2e-5)
 
 
+@pytest.mark.parametrize("M,N,K,tile,splits", [(40, 24, 1000, 64, 3), (300, 72, 2048, 128, 8), (130, 300, 640, 256, 2), (5, 160, 4096, 0, None)])
+@pytest.mark.parametrize("out", [BF, F32])
+def test_gemm_split_inner(X, M, N, K, tile, splits, out):
+    x, w = rnd(1, M, K, dtype=BF), rnd(2, N, K, scale=K ** -0.5, dtype=BF)
+    y = X.Linear(w)(x, out, tile=tile, splits=splits)
+    assert err(y, npy(x) @ npy(w).T) < (2e-2 if out == BF else 2e-5)
+
+
 def test_gemm_strided_input_and_activation(X):
     x, w = rnd(3, 150, 96, dtype=BF)[:, :40], rnd(4, 136, 40, scale=0.3, dtype=BF)
     act = X.XIELU(torch.tensor([-0.8, 1.3]))
@@ -307,7 +315,7 @@ def test_attention_cuda_cores(X, scmx, H, G, d, dv, dt):
         assert err(c.prefill(X, lo, hi, 1), want[lo:hi]) < (2.5e-2 if dt == BF else 3e-5), (lo, hi)
 
 
-@pytest.mark.parametrize("H,G,d,dv", SIZES + [(2, 1, 5, 7), (16, 1, 24, 128), (6, 2, 128, 256)])
+@pytest.mark.parametrize("H,G,d,dv", SIZES + [(2, 1, 5, 7), (16, 1, 24, 128), (6, 2, 128, 256), (36, 2, 16, 8)])
 @pytest.mark.parametrize("dt", [BF, F32])
 def test_attention_decode(X, scmx, H, G, d, dv, dt):
     T = 700

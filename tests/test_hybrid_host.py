@@ -42,7 +42,8 @@ def test_arguments_are_checked_before_a_launch(scmx):
     assert lib.scmx_diff_attn(p, p, p, 0, 4, 0, 8, 3, 2, 8, 8, 1.0, 0.5, 0.5, 1e-5, p, 0, p, None) == -1     # 3 heads over 2
     assert lib.scmx_diff_attn(p, p, p, 1, 4, 0, 8, 2, 2, 8, 8, 1.0, 0.5, 0.5, 1e-5, p, 2, p, None) == -5     # float32 on tensor cores
     assert lib.scmx_diff_decode(p, p, p, 0, 9, None, 8, 2, 2, 8, 8, 1.0, 0.5, 0.5, 1e-5, 4, p, p, p, None) == -1
-    assert lib.scmx_gemm_bf16(p, 12, p, 16, 4, 8, 12, 0, 0.0, 0.0, p, 0, 8, 0, p, None) == -1                # row pitch
+    assert lib.scmx_gemm_bf16(p, 12, p, 16, 4, 8, 12, 0, 0.0, 0.0, p, 0, 8, 0, 1, None, p, None) == -1       # row pitch
+    assert lib.scmx_gemm_bf16(p, 16, p, 16, 4, 8, 12, 0, 0.0, 0.0, p, 0, 8, 0, 2, p, p, None) == -1       # two ranges of one block
     assert lib.scmx_gemv_x(p, 12, 0, p, 4, 12, 0, 0.0, 0.0, None, None, None, 0, 0, p, None) == -1
     assert lib.scmx_retention_scratch(256, 2, 20, 64, 0, 128) == 0 and lib.scmx_retention_scratch(256, 2, 64, 64, 0, 128) > 0
 
