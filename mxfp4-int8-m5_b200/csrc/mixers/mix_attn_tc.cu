@@ -59,6 +59,7 @@ __global__ void __launch_bounds__(TA_THREADS, 1) diff_attn_tc_kernel(const __gri
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
     if (threadIdx.x == 0) {
+        for (const CUtensorMap* m : {&tmQ, &tmK, &tmV}) prefetch_map(m);
         for (int i = 0; i < L::NBAR; ++i) {
             const uint32_t b = bars + 8 * i;
             mbar_init(b, b == b_p || b == b_p + 8 ? 4 : 1);      // b_p: one arrival per softmax warp of the map

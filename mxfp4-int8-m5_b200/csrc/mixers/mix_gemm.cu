@@ -109,6 +109,8 @@ __device__ __forceinline__ void gemm_bf16_body(const CUtensorMap& tmA, const CUt
     const bool leader = rank == 0;
 
     if (threadIdx.x == 0) {
+        prefetch_map(&tmA);
+        prefetch_map(&tmB);
         for (int s = 0; s < STAGES; ++s) {
             mbar_init(bar_full + 8 * s, 1);
             mbar_init(bar_empty + 8 * s, 1);

@@ -30,26 +30,65 @@ struct RetTcArgs {
     float kscale;
 };
 
+// Eight values as two bfloat16 terms.
+__device__ __forceinline__ void put_split8(bf16_t* hi, bf16_t* lo, const float (&x)[8]) {
+    uint32_t h[4], l[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        h[i] = pack_bf16x2(x[2 * i], x[2 * i + 1]);
+        l[i] = pack_bf16x2(x[2 * i] - bf16_lo(h[i]), x[2 * i + 1] - bf16_hi(h[i]));
+    }
+    *reinterpret_cast<uint4*>(hi) = make_uint4(h[0], h[1], h[2], h[3]);
+    *reinterpret_cast<uint4*>(lo) = make_uint4(l[0], l[1], l[2], l[3]);
+}
+
+// VEC: half of the rotated elements is a multiple of 8 and rows are 16-byte aligned, so that the eight partners of eight elements
+// are one vector too.
+template <bool VEC>
 __global__ void __launch_bounds__(256) ret_prep_kernel(const RetTcArgs a) {
     pdl_launch_dependents();
     pdl_wait();
     const int64_t t = blockIdx.x;
     const int64_t end = min(a.n, (t / RC + 1) * RC) - 1;
     const float* cs = a.cs + t * a.dims;
-    for (int i = 2 * threadIdx.x; i < a.H * a.d; i += 512) {      // d is even: the pair lies in one head
+    const int half = a.dims >> 1;
+    for (int i = 8 * threadIdx.x; i < a.H * a.d; i += 2048) {
         const int h = i / a.d, e = i - h * a.d;
         const bf16_t *q = a.q + t * a.ldq + (int64_t)h * a.d, *k = a.k + t * a.ldk + (int64_t)h * a.d;
-        const float f = exp2f((float)(end - t) * log2f(a.decay[h]));
+        const float f = ex2_approx((float)(end - t) * log2f(a.decay[h]));
         const int64_t o = ((int64_t)h * a.n + t) * a.d + e;
-        auto put = [&](bf16_t* hi, bf16_t* lo, float x, float y) {
-            const uint32_t u = pack_bf16x2(x, y);
-            *reinterpret_cast<uint32_t*>(hi + o) = u;
-            *reinterpret_cast<uint32_t*>(lo + o) = pack_bf16x2(x - bf16_lo(u), y - bf16_hi(u));
-        };
-        put(a.qh, a.ql, rotated(q, e, a.dims, cs), rotated(q, e + 1, a.dims, cs));
-        const float k0 = rotated(k, e, a.dims, cs) * a.kscale, k1 = rotated(k, e + 1, a.dims, cs) * a.kscale;
-        put(a.kh, a.kl, k0, k1);
-        put(a.eh, a.el, k0 * f, k1 * f);
+        float x[8], y[8];
+        if (VEC) {
+            ld8(q + e, x);
+            ld8(k + e, y);
+            if (e < a.dims) {
+                const bool lo = e < half;
+                const int p = lo ? e + half : e - half, c = lo ? e : e - half;
+                float qp[8], kp[8], cc[8], sn[8];
+                ld8(q + p, qp);
+                ld8(k + p, kp);
+                ld8(cs + c, cc);
+                ld8(cs + half + c, sn);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) {
+                    const float s = lo ? -sn[j] : sn[j];
+                    x[j] = fmaf(x[j], cc[j], qp[j] * s);
+                    y[j] = fmaf(y[j], cc[j], kp[j] * s);
+                }
+            }
+        } else {
+            for (int j = 0; j < 8; ++j) {
+                x[j] = rotated(q, e + j, a.dims, cs);
+                y[j] = rotated(k, e + j, a.dims, cs);
+            }
+        }
+        put_split8(a.qh + o, a.ql + o, x);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) y[j] *= a.kscale;
+        put_split8(a.kh + o, a.kl + o, y);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) y[j] *= f;
+        put_split8(a.eh + o, a.el + o, y);
     }
 }
 
@@ -89,6 +128,9 @@ __global__ void __launch_bounds__(RK_THREADS, 1) ret_chunk_kernel(const __grid_c
     volatile int* abort_flag = reinterpret_cast<volatile int*>(smem + 2 * RK_TILE + 36);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (threadIdx.x == 0) {
+        prefetch_map(&tmEh);
+        prefetch_map(&tmEl);
+        prefetch_map(&tmV);
         mbar_init(b_full, 1);
         mbar_init(b_full + 8, 1);
         mbar_init(b_done, 1);
@@ -208,6 +250,7 @@ __global__ void __launch_bounds__(RO_THREADS, 1)
     volatile int* abort_flag = reinterpret_cast<volatile int*>(smem + L::MISC_OFF + 4);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (threadIdx.x == 0) {
+        for (const CUtensorMap* m : {&tmQh, &tmQl, &tmKh, &tmKl, &tmSh, &tmSl, &tmV}) prefetch_map(m);
         for (int i = 0; i < 2 * STAGES + 6; ++i) {
             const uint32_t b = b_q + 8 * i;
             mbar_init(b, b == b_p || b == b_p + 8 ? 4 : 1);
@@ -338,6 +381,7 @@ __global__ void __launch_bounds__(RO_THREADS, 1)
                 tc_fence_after();
                 const uint32_t ts = tmem + 128 * t + lane_base;
                 const int dist0 = pos - 128 * t;          // distance to the tile's first key
+                const float far = (float)dist0 * l2;
                 uint32_t r[2][32];
                 tmem_ld32(ts, r[0]);
                 tmem_ld_fence(r[0]);
@@ -351,8 +395,8 @@ __global__ void __launch_bounds__(RO_THREADS, 1)
                         float x[2];
 #pragma unroll
                         for (int e = 0; e < 2; ++e) {
-                            const int dist = dist0 - (32 * b + 2 * i + e);
-                            x[e] = dist >= 0 ? __uint_as_float(v[2 * i + e]) * exp2f((float)dist * l2) : 0.0f;
+                            const int j = 32 * b + 2 * i + e;
+                            x[e] = j <= dist0 ? __uint_as_float(v[2 * i + e]) * ex2_approx(fmaf((float)-j, l2, far)) : 0.0f;
                         }
                         const uint32_t hi = pack_bf16x2(x[0], x[1]);
                         pk[i] = hi;
@@ -374,7 +418,7 @@ __global__ void __launch_bounds__(RO_THREADS, 1)
             } else {
                 // warpgroup t stores value columns 64 t .. 64 t + 63
                 tc_fence_after();
-                const float f = exp2f((float)(pos + 1) * l2);
+                const float f = ex2_approx((float)(pos + 1) * l2);
                 float* out = a.o + ((int64_t)(q0 + row) * a.H + h) * a.dv + v0;
 #pragma unroll
                 for (int b = 0; b < 2; ++b) {
@@ -463,7 +507,9 @@ int retention_tc(const bf16_t* q, int64_t ldq, const bf16_t* k, int64_t ldk, con
     if (!rc) rc = make_map_planes(&eh, a.eh, H, n, 2 * d, 2 * d, 2 * n * d, 128);
     if (!rc) rc = make_map_planes(&el, a.el, H, n, 2 * d, 2 * d, 2 * n * d, 128);
     if (rc) return rc;
-    SCMX_PDL_OK("ret_prep_kernel", launch_pdl(ret_prep_kernel, dim3((unsigned)n), dim3(256), 0, st, a));
+    const bool vec = dims % 16 == 0 && ldq % 8 == 0 && ldk % 8 == 0 && (((uintptr_t)q | (uintptr_t)k | (uintptr_t)cs) & 15) == 0;
+    SCMX_PDL_OK("ret_prep_kernel", vec ? launch_pdl(ret_prep_kernel<true>, dim3((unsigned)n), dim3(256), 0, st, a)
+                                       : launch_pdl(ret_prep_kernel<false>, dim3((unsigned)n), dim3(256), 0, st, a));
     static bool configured[64] = {};
     const int dev = current_device();
     SCMX_REQUIRE(dev >= 0, SCMX_ECUDA, "no current CUDA device (ordinal 0..63)");
