@@ -53,10 +53,15 @@ class Linear:
             self.w[:, :self.K] = w
         self.dt = _dt(w)
 
-    def _splits(self, M):
-        """Ranges of K computed side by side when the output has few tiles (at least 512 of K each)."""
-        tiles = -(-M // 128) * -(-self.N // 64)
-        return max(1, min(8, self.K // 512, 148 // tiles)) if tiles <= 74 else 1
+    def _plan(self, M, splits, n_sm=148):
+        """(tile, ranges of K computed side by side) for a product with few output tiles: the fewest bytes staged per SM, counting
+        whole waves; at least 512 of K per range.  (0, 1): leave it to the kernel."""
+        tm = -(-M // 128)
+        if tm * -(-self.N // 64) >= n_sm or splits == 1:
+            return 0, splits or 1
+        cost = lambda tile, s: -(-tm * -(-self.N // tile) * s // n_sm) / s * (128 + tile)         # noqa: E731
+        return min(((t, s) for t in (64, 128) for s in ([splits] if splits else range(1, max(1, min(8, self.K // 512)) + 1))),
+                   key=lambda c: cost(*c))
 
     def __call__(self, x, out_dtype=None, act=None, tile=0, splits=None):
         """x [M, K] -> [M, N] in out_dtype (default: the weights' type)."""
@@ -72,8 +77,9 @@ class Linear:
         if _ld(x) % 8 or x.data_ptr() % 16:
             x = empty_rows(M, self.K, x.dtype, x.device).copy_(x)
         y = empty_rows(M, self.N, out_dtype, x.device)
-        if splits is None:
-            splits = 1 if act is not None else self._splits(M)
+        if tile == 0:
+            tile, splits = self._plan(M, 1 if act is not None else splits)
+        splits = splits or 1
         part = torch.empty(splits * M * ((self.N + 3) // 4 * 4), dtype=torch.float32, device=x.device) if splits > 1 else None
         _lib.mcall("scmx_gemm_bf16", _lib.ptr(x), _ld(x), _lib.ptr(self.w), self.w.shape[1], M, self.N, self.K, int(act is not None),
                    act.a_pos if act else 0.0, act.a_neg if act else 0.0, _lib.ptr(y), int(out_dtype == torch.float32), _round8(self.N), tile, splits,
