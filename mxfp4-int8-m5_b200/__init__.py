@@ -5,6 +5,6 @@ import sys as _sys
 
 from . import _lib, sc_format, sc_kernels, sc_moe, sc_decode, w4a8, fused_dense, fused_moe, parallel  # noqa: F401
 from . import host_model, packed_io, fused_qwen3, fused_olmoe, decode  # noqa: F401
-from . import sc_mixers, fused_hybrid, registry, engine  # noqa: F401
+from . import sc_mixers, hybrid_mixers, fused_hybrid, registry, engine  # noqa: F401
 
 _sys.modules.setdefault("scmx_b200", _sys.modules[__name__])

@@ -109,7 +109,22 @@ MIXER_SIGNATURES = {
     "scmx_res_norm": [c_vp, c_i64, c_vp, c_vp, c_float, c_i64, c_int, c_vp, c_i64, c_vp, c_int, c_int, c_vp, c_vp, c_int, c_vp],
     "scmx_norm_rows": [c_vp, c_vp, c_vp, c_float, c_i64, c_int, c_vp, c_int, c_vp],
     "scmx_conv_silu": [c_vp, c_i64, c_int, c_i64, c_int, c_int, c_vp, c_vp, c_vp, c_vp, c_i64, c_vp],
-    "scmx_head_norm_gate": [c_vp, c_vp, c_i64, c_int, c_i64, c_int, c_int, c_float, c_vp, c_vp],
+    "scmx_embed_pair": [c_vp, c_vp, c_vp, c_int, c_i64, c_i64, c_int, c_float, c_i64, c_i64, c_i64, c_vp, c_vp, c_vp],
+    "scmx_add_norm": [c_vp, c_i64, c_vp, c_vp, c_float, c_float, c_i64, c_int, c_vp, c_vp, c_int, c_vp],
+    "scmx_head_norm_gate": [c_vp, c_vp, c_i64, c_int, c_vp, c_int, c_i64, c_int, c_int, c_float, c_vp, c_vp],
+    "scmx_gated_gelu": [c_vp, c_i64, c_i64, c_int, c_vp, c_vp],
+    "scmx_delta_scratch": [c_i64, c_int, c_int, c_int, c_i64],
+    "scmx_delta": [c_vp, c_i64, c_vp, c_i64, c_vp, c_i64, c_vp, c_i64, c_vp, c_i64, c_int, c_int, c_i64, c_int, c_int, c_int, c_int, c_vp, c_vp,
+                   c_vp, c_vp, c_vp, c_i64, c_vp, c_vp],
+    "scmx_delta_step": [c_vp, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp, c_i64, c_int, c_vp, c_i64, c_int, c_int, c_int, c_int, c_int, c_int, c_vp, c_vp,
+                        c_vp, c_float, c_vp, c_vp, c_vp],
+    "scmx_latent_append": [c_vp, c_i64, c_int, c_int, c_int, c_i64, c_int, c_int, c_int, c_vp, c_vp, c_vp, c_i64, c_float, c_i64, c_vp, c_vp,
+                           c_i64, c_vp, c_i64, c_i64, c_vp],
+    "scmx_latent_rotate": [c_vp, c_i64, c_int, c_vp, c_i64, c_int, c_int, c_int, c_vp],
+    "scmx_latent_absorb": [c_vp, c_i64, c_int, c_vp, c_i64, c_int, c_vp, c_i64, c_i64, c_int, c_int, c_int, c_int, c_i64, c_vp, c_vp, c_vp],
+    "scmx_latent_rows": [c_vp, c_vp, c_i64, c_int, c_i64, c_i64, c_vp, c_i64, c_i64, c_int, c_int, c_int, c_float, c_int, c_vp, c_vp],
+    "scmx_latent_value": [c_vp, c_vp, c_i64, c_int, c_i64, c_i64, c_vp, c_i64, c_i64, c_int, c_int, c_int, c_int, c_vp, c_i64, c_int, c_vp],
+    "scmx_latent_attn": [c_vp, c_i64, c_vp, c_i64, c_vp, c_i64, c_i64, c_i64, c_i64, c_i64, c_int, c_int, c_int, c_int, c_float, c_vp, c_vp, c_vp],
     "scmx_xielu": [c_vp, c_i64, c_float, c_float, c_vp],
     "scmx_selective_scan": [c_vp, c_i64, c_vp, c_i64, c_vp, c_i64, c_vp, c_i64, c_int, c_i64, c_int, c_int, c_vp, c_vp, c_vp, c_vp, c_vp,
                             c_i64, c_vp],
@@ -130,7 +145,7 @@ MIXER_SIGNATURES = {
     "scmx_gemv_x": [c_vp, c_i64, c_int, c_vp, c_i64, c_i64, c_int, c_float, c_float, c_vp, c_vp, c_vp, c_int, c_int, c_vp, c_vp],
     "scmx_last_error_string": [],
 }
-_RESTYPE = {"scmx_last_error_string": ctypes.c_char_p, "scmx_retention_scratch": c_i64}
+_RESTYPE = {"scmx_last_error_string": ctypes.c_char_p, "scmx_retention_scratch": c_i64, "scmx_delta_scratch": c_i64}
 
 _lib = None
 _mixers = None

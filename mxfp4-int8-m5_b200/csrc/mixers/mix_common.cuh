@@ -101,6 +101,13 @@ __device__ __forceinline__ float xielu_f32(float z, float a_pos, float a_neg) {
     return fmaf(0.5f, z, z > 0.0f ? a_pos * z * z : a_neg * neg);
 }
 
+__device__ __forceinline__ float sigmoid_f32(float z) { return __fdividef(1.0f, 1.0f + exp_fast(-z)); }
+// z / 2 (1 + tanh(u)) = z sigmoid(2 u), u = sqrt(2 / pi) (z + 0.044715 z^3).
+__device__ __forceinline__ float gelu_tanh_f32(float z) {
+    const float u = 0.7978845608028654f * fmaf(0.044715f * z * z, z, z);
+    return z * sigmoid_f32(2.0f * u);
+}
+
 // Element i of a head vector of size d after the rotate-half rotation of its first `dims` elements: i < dims/2 pairs with
 // i + dims/2.  cs: the position's table row, cos (dims/2) then sin (dims/2).
 template <typename T>

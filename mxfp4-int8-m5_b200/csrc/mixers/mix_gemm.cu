@@ -2,7 +2,7 @@
 // GEMM (TMA producer warp, one MMA-issuing thread, 8 epilogue warps, two accumulators in tensor memory, persistent tiles): a K
 // block is 128 bytes = 64 values, so the stages, swizzle and descriptors are the INT8 kernel's.  Large shapes run on CTA pairs
 // (256 x 256 tiles), others on single CTAs (128 x BN tiles).
-// Epilogue: float32 or bfloat16 output, optionally through xIELU.  Rows of the output are padded to a multiple of 16 bytes.
+// Epilogue: float32 or bfloat16 output, optionally through xIELU or the gated GELU.  Rows of the output are padded to a multiple of 16 bytes.
 #include "mix_tc.cuh"
 
 namespace scmx {
@@ -10,7 +10,7 @@ namespace scmx {
 struct BgArgs {
     int M, N, K;
     int out_f32;                 // 1: float output, 0: bfloat16
-    int act;                     // 0: none, 1: xIELU
+    int act;                     // 0: none, 1: xIELU, 2: gelu(gate) up, columns alternate 16 gate and 16 up
     float a_pos, a_neg;          // xIELU: softplus(p), 1/2 + softplus(q)
     void* out;
     int64_t ldo;                 // elements
@@ -33,13 +33,16 @@ __device__ __forceinline__ void bg_drain(const BgArgs& a, uint8_t* out, const ui
 }
 
 // One warp's 32 rows x BN/2 accumulator columns (see epilogue_warp of the INT8 kernel for the staging layout).
+// A 32-column chunk leaves as 32 values, or as 16 with the gated activation (16 gate columns, 16 up columns).  Chunks are staged
+// until 128 bytes of a row are full.
 template <int BN>
 __device__ __forceinline__ void bg_epilogue(const BgArgs& a, uint8_t* out, uint32_t taddr, int row0, int n0, uint8_t* stg, int lane) {
     constexpr int CHUNKS = BN / 64;           // 32-column chunks
     uint8_t* my = stg + lane * EPI_PITCH;
-    const int esz = a.out_f32 ? 4 : 2;
+    const int esz = a.out_f32 ? 4 : 2, cols = a.act == 2 ? 16 : 32, bytes = cols * esz, unit = 128 / bytes;
     const size_t row_bytes = (size_t)a.ldo * esz;
-    const int npad = a.out_f32 ? (a.N + 3) & ~3 : (a.N + 7) & ~7;
+    const int nout = a.act == 2 ? a.N / 2 : a.N, npad = a.out_f32 ? (nout + 3) & ~3 : (nout + 7) & ~7;
+    const int c0 = a.act == 2 ? n0 / 2 : n0;
     uint32_t r[2][32];
     tmem_ld32(taddr, r[0]);
     tmem_ld_fence(r[0]);
@@ -50,29 +53,31 @@ __device__ __forceinline__ void bg_epilogue(const BgArgs& a, uint8_t* out, uint3
         if (a.act == 1) {
 #pragma unroll
             for (int j = 0; j < 32; ++j) v[j] = __float_as_uint(xielu_f32(__uint_as_float(v[j]), a.a_pos, a.a_neg));
+        } else if (a.act == 2) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j) v[j] = __float_as_uint(gelu_tanh_f32(__uint_as_float(v[j])) * __uint_as_float(v[16 + j]));
         }
+        const int k = c & (unit - 1);
+        uint4* o = reinterpret_cast<uint4*>(my + bytes * k);
         if (a.out_f32) {
 #pragma unroll
-            for (int j = 0; j < 8; ++j) reinterpret_cast<uint4*>(my)[j] = make_uint4(v[4 * j], v[4 * j + 1], v[4 * j + 2], v[4 * j + 3]);
-            __syncwarp();
-            const int col = n0 + c * 32;
-            bg_drain(a, out, stg, lane, row0, row_bytes, (size_t)col * 4, min(128, (npad - col) * 4));
-            __syncwarp();
+            for (int j = 0; j < 8; ++j)
+                if (4 * j < cols) o[j] = make_uint4(v[4 * j], v[4 * j + 1], v[4 * j + 2], v[4 * j + 3]);
         } else {
-            uint4* o = reinterpret_cast<uint4*>(my + 64 * (c & 1));
 #pragma unroll
-            for (int j = 0; j < 4; ++j) {
-                uint32_t pk[4];
+            for (int j = 0; j < 4; ++j)
+                if (8 * j < cols) {
+                    uint32_t pk[4];
 #pragma unroll
-                for (int i = 0; i < 4; ++i) pk[i] = pack_bf16x2(__uint_as_float(v[8 * j + 2 * i]), __uint_as_float(v[8 * j + 2 * i + 1]));
-                o[j] = make_uint4(pk[0], pk[1], pk[2], pk[3]);
-            }
-            if ((c & 1) || c + 1 == CHUNKS) {
-                __syncwarp();
-                const int col = n0 + (c & ~1) * 32;
-                bg_drain(a, out, stg, lane, row0, row_bytes, (size_t)col * 2, min((c & 1) ? 128 : 64, (npad - col) * 2));
-                __syncwarp();
-            }
+                    for (int i = 0; i < 4; ++i) pk[i] = pack_bf16x2(__uint_as_float(v[8 * j + 2 * i]), __uint_as_float(v[8 * j + 2 * i + 1]));
+                    o[j] = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+                }
+        }
+        if (k == unit - 1 || c + 1 == CHUNKS) {
+            __syncwarp();
+            const int col = c0 + (c - k) * cols;
+            bg_drain(a, out, stg, lane, row0, row_bytes, (size_t)col * esz, min((k + 1) * bytes, (npad - col) * esz));
+            __syncwarp();
         }
         if (c + 1 < CHUNKS) tmem_ld_fence(r[(c + 1) & 1]);
     }
@@ -323,9 +328,10 @@ extern "C" int scmx_gemm_bf16(const void* A, int64_t lda, const void* W, int64_t
     SCMX_REQUIRE(lda % 8 == 0 && ldw % 8 == 0 && lda >= K && ldw >= K, SCMX_EINVAL,
                  "gemm_bf16: the row pitches %lld, %lld must be multiples of 8 that hold K=%lld", (long long)lda, (long long)ldw, (long long)K);
     const int q = out_f32 ? 4 : 8;
-    SCMX_REQUIRE(ldo % q == 0 && ldo >= (N + q - 1) / q * q, SCMX_EINVAL, "gemm_bf16: output pitch %lld for %lld columns", (long long)ldo, (long long)N);
+    SCMX_REQUIRE(act >= 0 && act <= 2 && (act != 2 || N % 32 == 0), SCMX_EINVAL, "gemm_bf16: act=%d on %lld columns", act, (long long)N);
+    const int64_t nout = act == 2 ? N / 2 : N;
+    SCMX_REQUIRE(ldo % q == 0 && ldo >= (nout + q - 1) / q * q, SCMX_EINVAL, "gemm_bf16: output pitch %lld for %lld columns", (long long)ldo, (long long)N);
     SCMX_REQUIRE(((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0 && ((uintptr_t)out & 15) == 0, SCMX_EINVAL, "gemm_bf16: pointer not 16-byte aligned");
-    SCMX_REQUIRE(act == 0 || act == 1, SCMX_EINVAL, "gemm_bf16: act=%d", act);
     SCMX_REQUIRE(tile == 0 || tile == 64 || tile == 128 || tile == 256, SCMX_EINVAL, "gemm_bf16: tile=%d", tile);
     if (M == 0) return SCMX_OK;
     BgArgs a;

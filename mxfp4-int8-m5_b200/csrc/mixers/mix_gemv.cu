@@ -1,7 +1,8 @@
 // Matrix-vector product of the decode step: out [N] = W [N, K] x, weights bfloat16 or float, x and out float32, float32
 // accumulation.  Each warp owns two rows (or a slice of their columns) and keeps up to 16 weight loads of 16 bytes per lane in
 // flight; the first batch is issued before the previous kernel of the chain has finished (weights never change).
-// Epilogues: none; xIELU; the causal convolution + SiLU of the first C rows, whose carried inputs are shifted in place.
+// Epilogues: none; xIELU; the causal convolution + SiLU of the first C rows, whose carried inputs are shifted in place; gelu(gate) up
+// of rows that alternate 16 gate and 16 up rows (a warp owns one of each).
 #include "mix_common.cuh"
 
 namespace scmx {
@@ -55,6 +56,7 @@ __global__ void __launch_bounds__(256) gemv_x_kernel(const GvArgs a) {
     const int nv = (a.K + 7) >> 3, ks = a.ks;
     const int r0 = (blockIdx.x * (8 / ks) + warp / ks) * GV_ROWS, first = (warp % ks) * 32 + lane, step = 32 * ks;
     const T* W = static_cast<const T*>(a.W);
+    auto row_of = [&](int r) { return EPI == 3 ? 32 * (r0 >> 5) + ((r0 >> 1) & 15) + 16 * r : r0 + r; };
     Vec8<T> w[GV_ROWS][U];
     auto fetch = [&](int v0) {
 #pragma unroll
@@ -62,7 +64,7 @@ __global__ void __launch_bounds__(256) gemv_x_kernel(const GvArgs a) {
 #pragma unroll
             for (int r = 0; r < GV_ROWS; ++r) {
                 const int v = v0 + u * step;
-                if (v < nv && r0 + r < a.N) w[r][u].load(W + (int64_t)(r0 + r) * a.ldw + 8 * (int64_t)v);
+                if (v < nv && r0 + r < a.N) w[r][u].load(W + (int64_t)row_of(r) * a.ldw + 8 * (int64_t)v);
                 else w[r][u].zero();
             }
     };
@@ -106,6 +108,10 @@ __global__ void __launch_bounds__(256) gemv_x_kernel(const GvArgs a) {
             for (int i = 0; i < ks; ++i) s[r] += part[warp + i][r];
         }
     }
+    if (EPI == 3) {
+        if (lane == 0 && r0 < a.N) a.out[r0 >> 1] = gelu_tanh_f32(s[0]) * s[1];
+        return;
+    }
     const int row = r0 + lane;
     if (lane >= GV_ROWS || row >= a.N) return;
     float y = lane == 0 ? s[0] : s[1];
@@ -113,7 +119,7 @@ __global__ void __launch_bounds__(256) gemv_x_kernel(const GvArgs a) {
     if (EPI == 2 && row < a.C) {
         const float* cw = a.cw + (int64_t)row * a.taps;
         float* tl = a.tail + (int64_t)row * (a.taps - 1);
-        float c = fmaf(cw[a.taps - 1], y, a.cb[row]);
+        float c = fmaf(cw[a.taps - 1], y, a.cb == nullptr ? 0.0f : a.cb[row]);
         for (int j = 0; j < a.taps - 1; ++j) {
             c = fmaf(cw[j], tl[j], c);
             tl[j] = j + 1 < a.taps - 1 ? tl[j + 1] : y;
@@ -133,7 +139,7 @@ static int run_gemv(GvArgs a, int epi, cudaStream_t st) {
     a.ks = ks;
     const int rows = 8 / ks * GV_ROWS;
     const dim3 grid((unsigned)((a.N + rows - 1) / rows)), block(256);
-    auto kernel = epi == 0 ? gemv_x_kernel<T, 0> : epi == 1 ? gemv_x_kernel<T, 1> : gemv_x_kernel<T, 2>;
+    auto kernel = epi == 0 ? gemv_x_kernel<T, 0> : epi == 1 ? gemv_x_kernel<T, 1> : epi == 2 ? gemv_x_kernel<T, 2> : gemv_x_kernel<T, 3>;
     if (smem > 40 * 1024) SCMX_CUDA_OK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     SCMX_PDL_OK("gemv_x_kernel", launch_pdl(kernel, grid, block, smem, st, a));
     return SCMX_OK;
@@ -148,8 +154,8 @@ extern "C" int scmx_gemv_x(const void* W, int64_t ldw, int dt, const float* x, i
     SCMX_DT_OK("gemv_x", dt);
     SCMX_REQUIRE(W && x && out && N > 0 && K > 0 && N < (1ll << 30) && K < (1ll << 30), SCMX_EINVAL, "gemv_x: N=%lld K=%lld", (long long)N, (long long)K);
     SCMX_REQUIRE(ldw % 8 == 0 && ldw >= K && ((uintptr_t)W & 15) == 0, SCMX_EINVAL, "gemv_x: row pitch %lld", (long long)ldw);
-    SCMX_REQUIRE(epi >= 0 && epi <= 2, SCMX_EINVAL, "gemv_x: epi=%d", epi);
-    SCMX_REQUIRE(epi != 2 || (conv_w && conv_b && C > 0 && C <= N && taps >= 1 && (taps == 1 || tail)), SCMX_EINVAL, "gemv_x: convolution epilogue");
+    SCMX_REQUIRE(epi >= 0 && epi <= 3 && (epi != 3 || N % 32 == 0), SCMX_EINVAL, "gemv_x: epi=%d on %lld rows", epi, (long long)N);
+    SCMX_REQUIRE(epi != 2 || (conv_w && C > 0 && C <= N && taps >= 1 && (taps == 1 || tail)), SCMX_EINVAL, "gemv_x: convolution epilogue");
     GvArgs a;
     a.W = W; a.x = x; a.out = out; a.ldw = ldw; a.N = (int)N; a.K = (int)K; a.ks = 1; a.a_pos = a_pos; a.a_neg = a_neg;
     a.cw = conv_w; a.cb = conv_b; a.tail = tail; a.C = C; a.taps = taps;

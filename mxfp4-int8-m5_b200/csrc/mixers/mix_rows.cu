@@ -1,5 +1,6 @@
-// Row kernels around the mixers: embedding lookup, residual update with a norm on the sublayer's output and an optional
-// average over all layers' results, row norm, causal depthwise convolution + SiLU, per-head norm + gate.
+// Row kernels around the mixers: embedding lookup (optionally with a table row per pair of tokens), residual update with a norm on
+// the sublayer's output and an optional average over all layers' results, residual update followed by the next sublayer's norm,
+// row norm, causal depthwise convolution + SiLU, per-head norm + gate.
 // The residual stream is float32; a bfloat16 copy for the next matrix product is written beside it.
 #include <cooperative_groups.h>
 #include "mix_common.cuh"
@@ -20,6 +21,136 @@ __global__ void __launch_bounds__(256) embed_kernel(const int64_t* tok, const T*
         const T raw = table[id * W + i];
         x[t * W + i] = ldf(&raw);
         if (h != nullptr) h[t * W + i] = raw;
+    }
+}
+
+// x[t] = scale table[tok[t]] + pairs[row], row = (before mul_prev + tok mul_cur) mod buckets, or `buckets` at the start of a
+// sequence (prev < 0).  Only the first CTA reads and advances prev.
+struct EmbedPairArgs {
+    const int64_t* tok;
+    int64_t* prev;           // token before this portion, negative: none
+    float* x;
+    int64_t V, T, buckets, mul_prev, mul_cur;
+    int W;
+    float scale;
+};
+template <typename T>
+__global__ void __launch_bounds__(256) embed_pair_kernel(const T* table, const T* pairs, const EmbedPairArgs a) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int64_t t = blockIdx.x;
+    int64_t id = a.tok[t];
+    id = id < 0 ? 0 : (id >= a.V ? a.V - 1 : id);
+    const T* pr = nullptr;
+    if (pairs != nullptr) {
+        const int64_t before = t > 0 ? a.tok[t - 1] : *a.prev;
+        int64_t row = a.buckets;
+        if (before >= 0) {
+            row = (before * a.mul_prev + id * a.mul_cur) % a.buckets;
+            if (row < 0) row += a.buckets;
+        }
+        pr = pairs + row * a.W;
+    }
+    for (int i = threadIdx.x; i < a.W; i += 256) {
+        const float e = ldf(table + id * a.W + i) * a.scale;
+        a.x[t * a.W + i] = pr != nullptr ? e + ldf(pr + i) : e;
+    }
+    if (t == 0 && a.prev != nullptr) {
+        __syncthreads();
+        if (threadIdx.x == 0) *a.prev = a.tok[a.T - 1];
+    }
+}
+
+// ---- residual + next norm -----------------------------------------------------------------------------------------------
+struct AddNormArgs {
+    const float* y;        // [T, ldy] sublayer output, or null
+    const float* x;        // [T, W]
+    const float* w;        // [W] norm weight of the next sublayer
+    float* x_out;          // [T, W], or null (nothing to add); may be x
+    void* h_out;           // [T, W] activation type
+    int64_t ldy;
+    int W;
+    float mult, eps;
+};
+
+// r = x + mult y;  h = r / rms(r) w.  A cluster of CTAs shares one row; each thread keeps its first groups of V values.
+template <typename T, int V>
+__global__ void __launch_bounds__(256) add_norm_kernel(const AddNormArgs a) {
+    constexpr int KEEP = 4;
+    __shared__ float red[33];
+    __shared__ float part;
+    pdl_launch_dependents();
+    cg::cluster_group cl = cg::this_cluster();
+    const int nc = (int)cl.num_blocks(), rank = (int)cl.block_rank();
+    const int64_t t = blockIdx.x / nc;
+    const int nv = a.W / V, per = (nv + nc - 1) / nc;
+    const int v0 = rank * per, v1 = min(nv, v0 + per);
+    pdl_wait();
+    const float *y = a.y == nullptr ? nullptr : a.y + t * a.ldy, *x = a.x + t * a.W;
+    float* xo = a.x_out == nullptr ? nullptr : a.x_out + t * a.W;
+    float keep[KEEP][V], ss = 0.0f;
+    auto read = [&](int i, float (&r)[V]) {
+        if (V == 4) {
+            const float4 p = *reinterpret_cast<const float4*>(x + 4 * i);
+            r[0] = p.x; r[1 % V] = p.y; r[2 % V] = p.z; r[3 % V] = p.w;
+            if (y != nullptr) {
+                const float4 q = *reinterpret_cast<const float4*>(y + 4 * i);
+                r[0] = fmaf(a.mult, q.x, r[0]); r[1 % V] = fmaf(a.mult, q.y, r[1 % V]); r[2 % V] = fmaf(a.mult, q.z, r[2 % V]); r[3 % V] = fmaf(a.mult, q.w, r[3 % V]);
+            }
+        } else {
+            r[0] = x[i];
+            if (y != nullptr) r[0] = fmaf(a.mult, y[i], r[0]);
+        }
+    };
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+        const int i = v0 + (int)threadIdx.x + 256 * k;
+        if (i < v1) {
+            read(i, keep[k]);
+        } else {
+#pragma unroll
+            for (int e = 0; e < V; ++e) keep[k][e] = 0.0f;
+        }
+    }
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k)
+#pragma unroll
+        for (int e = 0; e < V; ++e) ss += keep[k][e] * keep[k][e];
+    for (int i = v0 + (int)threadIdx.x + 256 * KEEP; i < v1; i += 256) {
+        float r[V];
+        read(i, r);
+#pragma unroll
+        for (int e = 0; e < V; ++e) ss += r[e] * r[e];
+    }
+    ss = block_sumf(ss, red);
+    if (nc > 1) {
+        if (threadIdx.x == 0) part = ss;
+        cl.sync();
+        ss = 0.0f;
+        for (int r = 0; r < nc; ++r) ss += *cl.map_shared_rank(&part, r);
+        cl.sync();              // nobody leaves while its partial sum may still be read
+    }
+    const float inv = rms_inv_f32(ss, a.W, a.eps);
+    T* h = static_cast<T*>(a.h_out) + t * a.W;
+    auto write = [&](int i, const float (&r)[V]) {
+        if (V == 4) {
+            const float4 w = *reinterpret_cast<const float4*>(a.w + 4 * i);
+            if (xo != nullptr) st4(xo + 4 * i, r[0], r[1 % V], r[2 % V], r[3 % V]);
+            st4(h + 4 * i, r[0] * inv * w.x, r[1 % V] * inv * w.y, r[2 % V] * inv * w.z, r[3 % V] * inv * w.w);
+        } else {
+            if (xo != nullptr) xo[i] = r[0];
+            stf(h + i, r[0] * inv * a.w[i]);
+        }
+    };
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+        const int i = v0 + (int)threadIdx.x + 256 * k;
+        if (i < v1) write(i, keep[k]);
+    }
+    for (int i = v0 + (int)threadIdx.x + 256 * KEEP; i < v1; i += 256) {
+        float r[V];
+        read(i, r);
+        write(i, r);
     }
 }
 
@@ -164,7 +295,7 @@ __global__ void __launch_bounds__(256) conv_silu_kernel(const T* x, int64_t ldx,
                 if (t < 0) in[i] = make_float2(tail[(int64_t)c * (TAPS - 1) + t + TAPS - 1], tail[(int64_t)(c + 1) * (TAPS - 1) + t + TAPS - 1]);
             }
         }
-        const float2 bias = make_float2(b[c], b[c + 1]);
+        const float2 bias = b == nullptr ? make_float2(0.0f, 0.0f) : make_float2(b[c], b[c + 1]);
         float2 ww[TAPS > 0 ? TAPS : 1];
 #pragma unroll
         for (int j = 0; j < TAPS; ++j) ww[j] = make_float2(w[(int64_t)c * TAPS + j], w[(int64_t)(c + 1) * TAPS + j]);
@@ -189,7 +320,7 @@ __global__ void __launch_bounds__(256) conv_silu_kernel(const T* x, int64_t ldx,
         const int c = blockIdx.x * 256 + threadIdx.x;
         if (c >= C) return;
         for (int64_t t = t0; t < t1; ++t) {
-            float s = b[c];
+            float s = b == nullptr ? 0.0f : b[c];
             for (int j = 0; j < taps; ++j) {
                 const int64_t u = t - (taps - 1) + j;
                 s = fmaf(w[(int64_t)c * taps + j], u >= 0 ? ldf(x + u * ldx + c) : tail[(int64_t)c * (taps - 1) + (u + taps - 1)], s);
@@ -214,10 +345,10 @@ __global__ void __launch_bounds__(256) conv_tail_kernel(const T* x, int64_t ldx,
 }
 
 // ---- per-head norm + gate -----------------------------------------------------------------------------------------------
-// out[t, h, :] = o[t, h, :] / rms * silu(g[t, h, :]); one warp per (token, head).
-template <typename T>
-__global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* o, const T* g, int64_t ldg, int64_t n, int H, int dv, float eps,
-                                                             int vec, T* out) {
+// out[t, h, :] = o[t, h, :] / rms * w * gate(g[t, h, :]), gate = SiLU or the sigmoid; one warp per (token, head).
+template <typename T, bool SIG>
+__global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* o, const T* g, int64_t ldg, const float* w, int64_t n, int H, int dv,
+                                                             float eps, int vec, T* out) {
     pdl_launch_dependents();
     pdl_wait();
     const int64_t i = (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5);
@@ -227,6 +358,7 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* o, con
     const int h = (int)(i - t * H);
     const float* p = o + i * dv;
     const T* gp = g + t * ldg + (int64_t)h * dv;
+    auto gate = [](float z) { return SIG ? sigmoid_f32(z) : silu_f32(z); };
     float ss = 0.0f;
     if (vec) {                      // rows of four aligned values; up to 4 groups per lane stay in registers
         float4 v[4], gv[4];
@@ -241,14 +373,16 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* o, con
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int e = 4 * (lane + 32 * j);
-            if (e < dv) st4(out + i * dv + e, v[j].x * inv * silu_f32(gv[j].x), v[j].y * inv * silu_f32(gv[j].y), v[j].z * inv * silu_f32(gv[j].z),
-                            v[j].w * inv * silu_f32(gv[j].w));
+            if (e >= dv) continue;
+            const float4 ww = w != nullptr ? *reinterpret_cast<const float4*>(w + e) : make_float4(1, 1, 1, 1);
+            st4(out + i * dv + e, v[j].x * inv * ww.x * gate(gv[j].x), v[j].y * inv * ww.y * gate(gv[j].y), v[j].z * inv * ww.z * gate(gv[j].z),
+                v[j].w * inv * ww.w * gate(gv[j].w));
         }
         return;
     }
     for (int e = lane; e < dv; e += 32) ss += p[e] * p[e];
     const float inv = rms_inv_f32(warp_sumf(ss), dv, eps);
-    for (int e = lane; e < dv; e += 32) stf(out + i * dv + e, p[e] * inv * silu_f32(ldf(gp + e)));
+    for (int e = lane; e < dv; e += 32) stf(out + i * dv + e, p[e] * inv * (w != nullptr ? w[e] : 1.0f) * gate(ldf(gp + e)));
 }
 
 // ---- xIELU of float32 values, in place ------------------------------------------------------------------------------------
@@ -257,6 +391,41 @@ __global__ void __launch_bounds__(256) xielu_kernel(float* x, int64_t n, float a
     pdl_wait();
     const int64_t i = (int64_t)blockIdx.x * 256 + threadIdx.x;
     if (i < n) x[i] = xielu_f32(x[i], a_pos, a_neg);
+}
+
+// out[r, j] = gelu(gate) up of rows whose columns alternate 16 gate and 16 up values.
+__global__ void __launch_bounds__(256) gated_gelu_kernel(const float* x, int64_t ldx, int64_t rows, int n, float* out) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int64_t i = (int64_t)blockIdx.x * 256 + threadIdx.x;
+    if (i >= rows * n) return;
+    const int64_t r = i / n;
+    const int j = (int)(i - r * n);
+    const float* p = x + r * ldx + 32 * (j >> 4) + (j & 15);
+    out[i] = gelu_tanh_f32(p[0]) * p[16];
+}
+
+template <typename T>
+static int run_add_norm(const AddNormArgs& a, int64_t T_, cudaStream_t st) {
+    const int vec = (a.W % 4 == 0 && a.ldy % 4 == 0) ? 4 : 1;
+    const int slices = (a.W / vec + 255) / 256;
+    int nc = 1;
+    while (nc < 8 && nc < slices && T_ * nc * 2 <= 148) nc *= 2;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3((unsigned)(T_ * nc));
+    cfg.blockDim = dim3(256);
+    cfg.stream = st;
+    cudaLaunchAttribute at[2];
+    at[0].id = cudaLaunchAttributeClusterDimension;
+    at[0].val.clusterDim.x = nc;
+    at[0].val.clusterDim.y = at[0].val.clusterDim.z = 1;
+    at[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    at[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = at;
+    cfg.numAttrs = g_use_pdl ? 2 : 1;
+    SCMX_PDL_OK("add_norm_kernel", vec == 4 ? cudaLaunchKernelEx(&cfg, add_norm_kernel<T, 4>, a)
+                                            : cudaLaunchKernelEx(&cfg, add_norm_kernel<T, 1>, a));
+    return SCMX_OK;
 }
 
 template <typename T>
@@ -346,26 +515,64 @@ extern "C" int scmx_norm_rows(const float* x, const int64_t* rows, const float* 
 extern "C" int scmx_conv_silu(const void* x, int64_t ldx, int dt, int64_t T, int C, int taps, const float* w, const float* b, float* tail,
                               void* out, int64_t ldo, void* stream) {
     SCMX_DT_OK("conv_silu", dt);
-    SCMX_REQUIRE(x && w && b && out && T >= 0 && C > 0 && taps >= 1 && ldx >= C && ldo >= C, SCMX_EINVAL, "conv_silu: bad argument");
+    SCMX_REQUIRE(x && w && out && T >= 0 && C > 0 && taps >= 1 && ldx >= C && ldo >= C, SCMX_EINVAL, "conv_silu: bad argument");
     SCMX_REQUIRE(taps == 1 || tail != nullptr, SCMX_EINVAL, "conv_silu: %d taps need the carried inputs", taps);
     if (T == 0) return SCMX_OK;
     if (dt == 0) return run_conv((const bf16_t*)x, ldx, T, C, taps, w, b, tail, (bf16_t*)out, ldo, (cudaStream_t)stream);
     return run_conv((const float*)x, ldx, T, C, taps, w, b, tail, (float*)out, ldo, (cudaStream_t)stream);
 }
 
-extern "C" int scmx_head_norm_gate(const float* o, const void* g, int64_t ldg, int dt, int64_t T, int H, int dv, float eps, void* out, void* stream) {
+extern "C" int scmx_embed_pair(const int64_t* tokens, const void* table, const void* pairs, int dt, int64_t V, int64_t T, int W, float scale,
+                               int64_t buckets, int64_t mul_prev, int64_t mul_cur, int64_t* prev, float* x, void* stream) {
+    SCMX_DT_OK("embed_pair", dt);
+    SCMX_REQUIRE(tokens && table && x && V > 0 && T >= 0 && W > 0, SCMX_EINVAL, "embed_pair: bad argument");
+    SCMX_REQUIRE(pairs == nullptr || (prev && buckets > 0), SCMX_EINVAL, "embed_pair: a pair table needs buckets and the token before");
+    if (T == 0) return SCMX_OK;
+    EmbedPairArgs a;
+    a.tok = tokens; a.prev = prev; a.x = x; a.V = V; a.T = T; a.buckets = buckets; a.mul_prev = mul_prev; a.mul_cur = mul_cur; a.W = W; a.scale = scale;
+    const cudaStream_t st = (cudaStream_t)stream;
+    if (dt == 0)
+        SCMX_PDL_OK("embed_pair_kernel", launch_pdl(embed_pair_kernel<bf16_t>, dim3((unsigned)T), dim3(256), 0, st, (const bf16_t*)table, (const bf16_t*)pairs, a));
+    else
+        SCMX_PDL_OK("embed_pair_kernel", launch_pdl(embed_pair_kernel<float>, dim3((unsigned)T), dim3(256), 0, st, (const float*)table, (const float*)pairs, a));
+    return SCMX_OK;
+}
+
+extern "C" int scmx_add_norm(const float* y, int64_t ldy, const float* x, const float* w, float mult, float eps, int64_t T, int W, float* x_out,
+                             void* h_out, int dt, void* stream) {
+    SCMX_DT_OK("add_norm", dt);
+    SCMX_REQUIRE(x && w && h_out && T >= 0 && W > 0, SCMX_EINVAL, "add_norm: bad argument");
+    SCMX_REQUIRE(y == nullptr || (x_out && ldy >= W), SCMX_EINVAL, "add_norm: a sublayer's output needs a pitch and a place for the sum");
+    if (T == 0) return SCMX_OK;
+    AddNormArgs a;
+    a.y = y; a.x = x; a.w = w; a.x_out = y != nullptr ? x_out : nullptr; a.h_out = h_out; a.ldy = y != nullptr ? ldy : 0; a.W = W; a.mult = mult; a.eps = eps;
+    return dt == 0 ? run_add_norm<bf16_t>(a, T, (cudaStream_t)stream) : run_add_norm<float>(a, T, (cudaStream_t)stream);
+}
+
+extern "C" int scmx_head_norm_gate(const float* o, const void* g, int64_t ldg, int dt, const float* w, int gate, int64_t T, int H, int dv, float eps,
+                                   void* out, void* stream) {
     SCMX_DT_OK("head_norm_gate", dt);
     SCMX_REQUIRE(o && g && out && T >= 0 && H > 0 && dv > 0 && ldg >= (int64_t)H * dv, SCMX_EINVAL, "head_norm_gate: bad argument");
+    SCMX_REQUIRE(gate == 0 || gate == 1, SCMX_EINVAL, "head_norm_gate: gate=%d (0 = SiLU, 1 = sigmoid)", gate);
     if (T == 0) return SCMX_OK;
     const int64_t n = T * H;
     const int esz = dt == 0 ? 2 : 4;
-    const int vec = dv % 4 == 0 && dv <= 512 && ldg % 4 == 0 && (uintptr_t)g % (4 * esz) == 0;
+    const int vec = dv % 4 == 0 && dv <= 512 && ldg % 4 == 0 && (uintptr_t)g % (4 * esz) == 0 && (uintptr_t)w % 16 == 0;
     const dim3 grid((unsigned)((n + 7) / 8)), block(256);
     const cudaStream_t st = (cudaStream_t)stream;
-    if (dt == 0)
-        SCMX_PDL_OK("head_norm_gate_kernel", launch_pdl(head_norm_gate_kernel<bf16_t>, grid, block, 0, st, o, (const bf16_t*)g, ldg, n, H, dv, eps, vec, (bf16_t*)out));
-    else
-        SCMX_PDL_OK("head_norm_gate_kernel", launch_pdl(head_norm_gate_kernel<float>, grid, block, 0, st, o, (const float*)g, ldg, n, H, dv, eps, vec, (float*)out));
+#define GO(T_, S_) SCMX_PDL_OK("head_norm_gate_kernel", launch_pdl(head_norm_gate_kernel<T_, S_>, grid, block, 0, st, o, (const T_*)g, ldg, w, n, H, dv, eps, vec, (T_*)out))
+    if (dt == 0 && gate == 0) GO(bf16_t, false);
+    else if (dt == 0) GO(bf16_t, true);
+    else if (gate == 0) GO(float, false);
+    else GO(float, true);
+#undef GO
+    return SCMX_OK;
+}
+
+extern "C" int scmx_gated_gelu(const float* x, int64_t ldx, int64_t rows, int n, float* out, void* stream) {
+    SCMX_REQUIRE(x && out && rows >= 0 && n > 0 && n % 16 == 0 && ldx >= 2 * n, SCMX_EINVAL, "gated_gelu: %d outputs per row", n);
+    if (rows == 0) return SCMX_OK;
+    SCMX_PDL_OK("gated_gelu_kernel", launch_pdl(gated_gelu_kernel, dim3((unsigned)((rows * n + 255) / 256)), dim3(256), 0, (cudaStream_t)stream, x, ldx, rows, n, out));
     return SCMX_OK;
 }
 

@@ -236,49 +236,52 @@ class DecodeHybrid(_Decoder):
         self.f, self.model, self.args, self._graph = fused, fused.model, fused.args, None
         dev, a = fused.model.device, self.args
         f32 = lambda *s: torch.empty(s, dtype=torch.float32, device=dev)    # noqa: E731
-        self.xs = f32(len(a.layers) + 1, 1, a.hidden_size)      # the embedding's and every layer's result, for the depth average
-        self.x = f32(1, a.hidden_size)
-        self.bufs = []
+        self.x, self.h, self.y = f32(1, a.hidden_size), f32(1, a.hidden_size), f32(1, a.hidden_size)
+        if not a.design.prenorm:     # the embedding's and every layer's result, for the depth average
+            self.xs = f32(len(a.layers) + 1, 1, a.hidden_size)
+        own = {}
         for ly in fused.layers:
-            b = {"y": f32(1, a.hidden_size)}
-            if ly.type == "mamba1":
-                b.update(xz=f32(2 * ly.C), dbc=f32(ly.w_x.N), s=f32(ly.C))
-            else:
-                b.update(qkv=f32(ly.w_in.N), o=f32(ly.w_o.K))
-            if ly.type == "attention":
-                b["attn"] = X.DiffDecodeAttention(ly.H, ly.G, ly.d, ly.dv, dev)
-            if ly.w_up is not None:
-                b["u"] = f32(ly.w_up.N)
-            self.bufs.append(b)
+            if ly not in own:
+                own[ly] = ly.mixer.buffers(dev)
+                if ly.w_up is not None:
+                    own[ly]["u"] = f32(ly.w_up.N // (2 if ly.act.code == 2 else 1))
+        self.bufs = [own[ly] for ly in fused.layers]
 
     def _mix(self, ly, b, x, c, pos_dev):
-        if ly.type == "mamba1":
-            xz = ly.w_in.vec(x, conv=(ly.conv_w, ly.conv_b, c.tail), out=b["xz"])
-            dbc = ly.w_x.vec(xz[:ly.C], out=b["dbc"])
-            o = X.scan_step(xz, xz[ly.C:], dbc, ly.w_dt, ly.dt_b, ly.A2, ly.D, c.ssm, b["s"])
-        elif ly.type == "retention":
-            q, k, v, g = ly.w_in.vec(x, out=b["qkv"]).split(ly.sizes)
-            o = X.retention_step(q, k, v, g, self.f.table(ly), ly.dims, ly.kscale, ly.decay, self.f.eps, c.kv, b["o"], c.offset, pos_dev)
-        else:
-            q, k, v = ly.w_in.vec(x, out=b["qkv"])[None].split(ly.sizes, 1)
-            q = X.qk_norm_append(q, k, v, ly.H, ly.G, ly.q_norm, ly.k_norm, self.f.eps, c, torch.float32, pos_dev)
-            o = b["attn"](q, c, ly.scale, ly.lam, ly.diff, self.f.eps, b["o"], n_pos=c.offset + 1, pos_dev=pos_dev)
-        return ly.w_o.vec(o, out=b["y"].view(-1))
+        return ly.mixer.w_o.vec(ly.mixer.step(self.f, x, c, b, pos_dev), out=self.y.view(-1))
 
     def _step(self, tok, cache, pos_dev):
         f = self.f
         f.ensure_positions(cache[0].capacity)
         assert pos_dev is not None or cache[0].offset < cache[0].capacity, "KV cache capacity exceeded"
-        X.embed(tok.view(-1), f.embed, self.xs[0])
+        h = (self._prenorm if self.args.design.prenorm else self._postnorm)(tok.view(-1), cache, pos_dev)
+        return f.head.vec(h[0])[None, None]
+
+    def _prenorm(self, tok, cache, pos_dev):
+        f, x, h, y, mult = self.f, self.x, self.h, self.y, self.args.residual_mult
+        f.embed(tok, cache, x)
+        nl = len(f.layers)
+        X.add_norm(None, x, f.layers[0].norm1 if nl else f.final_norm, mult, f.eps, h)
+        for i, (ly, b, c) in enumerate(zip(f.layers, self.bufs, cache)):
+            after = f.layers[i + 1].norm1 if i + 1 < nl else f.final_norm
+            self._mix(ly, b, h[0], c, pos_dev)
+            X.add_norm(y, x, after if ly.w_up is None else ly.norm2, mult, f.eps, h)
+            if ly.w_up is not None:
+                ly.feed_forward_vec(h[0], b["u"], y.view(-1))
+                X.add_norm(y, x, after, mult, f.eps, h)
+        return h
+
+    def _postnorm(self, tok, cache, pos_dev):
+        f, y = self.f, self.y
+        f.embed(tok, cache, self.xs[0])
         x = self.xs[0]
         for i, (ly, b, c) in enumerate(zip(f.layers, self.bufs, cache)):
             self._mix(ly, b, x[0], c, pos_dev)
-            y = b["y"]
             if ly.w_up is not None:
                 X.res_norm(y, x, ly.norm1, f.eps, self.x)
                 x = self.x
-                ly.w_down.vec(ly.w_up.vec(x[0], act=ly.act, out=b["u"]), out=y.view(-1))
+                ly.feed_forward_vec(x[0], b["u"], y.view(-1))
             X.res_norm(y, x, ly.norm2 if ly.w_up is not None else ly.norm1, f.eps, self.x,
                        average=(self.xs, ly.dwa, i + 1 < len(f.layers)))
             x = self.x
-        return f.head.vec(X.norm_rows(x, f.final_norm, f.eps, torch.float32)[0])[None, None]
+        return X.norm_rows(x, f.final_norm, f.eps, torch.float32)

@@ -112,6 +112,37 @@ class StateCache:
         return list(self.state.values())
 
 
+class LatentCache:
+    """Latents of one layer's attention: rows of [latent, rotated key part], each part zero padded to a multiple of 8 values."""
+
+    def __init__(self, latent, rot, capacity, device="cuda", dtype=torch.bfloat16):
+        up8 = lambda n: (n + 7) // 8 * 8      # noqa: E731
+        self.c = torch.zeros((capacity, up8(latent) + up8(rot)), dtype=dtype, device=device)
+        self.offset, self.capacity = 0, capacity
+
+    def reset(self):
+        """Forget the sequence; rows past `offset` are never read."""
+        self.offset = 0
+
+    def carried(self):
+        return []
+
+
+class TokenCache:
+    """The token before the next one, where the embedding depends on it; negative at the start of a sequence."""
+
+    def __init__(self, capacity, device="cuda"):
+        self.prev = torch.full((1,), -1, dtype=torch.long, device=device)
+        self.offset, self.capacity = 0, capacity
+
+    def reset(self):
+        self.offset = 0
+        self.prev.fill_(-1)
+
+    def carried(self):
+        return [self.prev]
+
+
 def sdpa(q, k, v, scale, causal):
     """q [hq, L, d], k / v [hk, T, d] (T >= L: the last L keys are the queries' own positions) -> [L, hq * d]."""
     hq, L, d = q.shape
@@ -288,10 +319,25 @@ class CausalLM(torch.nn.Module):
 
 @dataclass
 class LayerArgs:
-    """One entry of a hybrid model's layer list: the mixer's type and sizes, and its feed-forward (None: no second sublayer)."""
+    """One entry of a hybrid model's layer list: the mixer's type and sizes, its feed-forward (None: no second sublayer), and the
+    layer whose tensors it uses (None: its own)."""
     type: str
     mixer: dict
     mlp: dict = None
+    weights_of: int = None
+
+
+@dataclass(frozen=True)
+class Design:
+    """What the decoders of one architecture have around their mixers.  prenorm: x <- x + m sublayer(norm(x)); otherwise
+    x <- x + norm(sublayer(x)) and a weighted sum of all layers' results after every layer.  act: the feed-forward's activation,
+    "xielu" (two parameters) or "gated_gelu" (a gate projection)."""
+    prenorm: bool
+    act: str
+    tied: bool
+
+
+DESIGNS = {"sebesun": Design(False, "xielu", False), "fabezen": Design(True, "gated_gelu", True)}
 
 
 @dataclass
@@ -301,22 +347,52 @@ class HybridArgs:
     rms_norm_eps: float
     layers: list
     model_type: str = "sebesun"
+    residual_mult: float = 1.0
+    embed_scale: float = 1.0
+    bigram: dict = None          # buckets, mul_prev, mul_cur of the table added per pair of neighbouring tokens
+
+    @property
+    def design(self):
+        return DESIGNS[self.model_type]
+
+    def source(self, i):
+        """The layer whose tensors layer i uses."""
+        seen = set()
+        while self.layers[i].weights_of is not None:
+            if i in seen:
+                raise ValueError(f"layer {i}: its weights are its own through weights_of")
+            seen.add(i)
+            i = self.layers[i].weights_of
+        return i
 
     @classmethod
     def from_config(cls, cfg):
         """cfg: the dictionary of a config.json with 'vocab', 'width', 'norm' and 'layers'."""
-        layers = [LayerArgs(e["type"], dict(e["mixer"]), dict(e["mlp"]) if e.get("mlp") else None) for e in cfg["layers"]]
+        layers = [LayerArgs(e["type"], dict(e["mixer"]), dict(e["mlp"]) if e.get("mlp") else None, e.get("weights_of")) for e in cfg["layers"]]
         for i, e in enumerate(layers):
             if e.type not in MIXERS:
                 raise ValueError(f"layer {i}: mixer {e.type!r} is not one of {sorted(MIXERS)}")
             if e.mlp is not None and e.mlp.get("kind") != "dense":
                 raise ValueError(f"layer {i}: feed-forward kind {e.mlp.get('kind')!r} (only 'dense')")
             m = e.mixer
-            if e.type == "attention" and m["heads"] % m["kv_heads"]:
+            if "kv_heads" in m and m["heads"] % m["kv_heads"]:
                 raise ValueError(f"layer {i}: {m['heads']} heads over {m['kv_heads']} key/value heads")
             if e.type == "retention" and len(m["decay"]) != m["heads"]:
                 raise ValueError(f"layer {i}: {len(m['decay'])} decays for {m['heads']} heads")
-        return cls(cfg["vocab"], cfg["width"], float(cfg["norm"]["eps"]), layers, cfg["architecture"].lower())
+            if e.type == "latent_attention" and m["rot_dim"] and m["rot"]["dims"] != m["rot_dim"]:
+                raise ValueError(f"layer {i}: {m['rot']['dims']} rotated elements of a part of {m['rot_dim']}")
+            if e.weights_of is not None:
+                if not 0 <= e.weights_of < len(layers):
+                    raise ValueError(f"layer {i}: weights of layer {e.weights_of}")
+                o = layers[e.weights_of]
+                if (o.type, o.mixer, o.mlp) != (e.type, e.mixer, e.mlp):
+                    raise ValueError(f"layer {i} differs from layer {e.weights_of}, whose weights it uses")
+        emb = cfg.get("embedding") or {}
+        out = cls(cfg["vocab"], cfg["width"], float(cfg["norm"]["eps"]), layers, cfg["architecture"].lower(), float(cfg.get("residual_mult", 1.0)),
+                  float(emb.get("scale", 1.0)), dict(emb["bigram"]) if emb.get("bigram") else None)
+        for i in range(len(layers)):
+            out.source(i)
+        return out
 
 
 def _mamba1_tensors(m, D):
@@ -336,39 +412,80 @@ def _diff_attention_tensors(m, D):
             "lk2": (d,), "o": (D, h * dv)}
 
 
-# mixer type -> (tensor shapes, cache of one layer)
+def _delta_tensors(m, D, channel=False):
+    h, g, d, dv, taps = m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"]
+    out = {"q": (g * d, D), "q.conv": (g * d, taps), "k": (g * d, D), "k.conv": (g * d, taps), "v": (h * dv, D), "v.conv": (h * dv, taps),
+           "b": (h, D), "A_log": (h,), "norm": (dv,), "o": (D, h * dv)}
+    if channel:      # inner sizes of the low-rank products: the checkpoint's
+        out.update({"a1": ("decay rank", D), "a2": (h * d, "decay rank"), "dt_bias": (h * d,), "g1": ("gate rank", D), "g2": (h * dv, "gate rank")})
+    else:
+        out.update({"a": (h, D), "dt_bias": (h,), "g": (h * dv, D)})
+    return out
+
+
+def _latent_attention_tensors(m, D):
+    h, d, r, dv, R, Q = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], m["q_rank"]
+    return {"dq": (Q, D), "dq.norm": (Q,), "uq": (h * (d + r), Q), "dkv": (R + r, D), "dkv.norm": (R,), "uk": (h * d, R), "uv": (h * dv, R),
+            "o": (D, h * dv)}
+
+
+def _delta_cache(m, cap, dev, dt):
+    return StateCache({"tail": (2 * m["kv_heads"] * m["dim"] + m["heads"] * m["vdim"], m["conv"] - 1), "kv": (m["heads"], m["dim"], m["vdim"])}, cap, dev)
+
+
+# mixer type -> (tensor shapes, cache of one layer); a name instead of a size: any size, the same wherever a layer has the name
 MIXERS = {
     "mamba1": (_mamba1_tensors, lambda m, cap, dev, dt: StateCache(
         {"tail": (m["inner"], m["conv"] - 1), "ssm": (m["inner"], m["state"])}, cap, dev)),
     "retention": (_retention_tensors, lambda m, cap, dev, dt: StateCache({"kv": (m["heads"], m["dim"], m["vdim"])}, cap, dev)),
     "attention": (_diff_attention_tensors, lambda m, cap, dev, dt: KVCache(
         2 * m["kv_heads"], m["dim"], cap, dev, dt, m["kv_heads"], m["vdim"])),
+    "delta": (_delta_tensors, _delta_cache),
+    "channel_delta": (lambda m, D: _delta_tensors(m, D, True), _delta_cache),
+    "latent_attention": (_latent_attention_tensors, lambda m, cap, dev, dt: LatentCache(m["kv_rank"], m["rot_dim"], cap, dev, dt)),
 }
 
 
 class HybridLM:
-    """Weights of a decoder whose layers mix selective scans, retention and differential attention: {tensor name: tensor} in the
-    checkpoint's names, on one device, bfloat16 (the serving type) or float32."""
+    """Weights of a decoder whose layers name their mixers (selective scan, retention, differential attention, gated delta rules,
+    latent attention): {tensor name: tensor} in the checkpoint's names, on one device, bfloat16 (the serving type) or float32."""
 
     def __init__(self, args, device="cuda", dtype=torch.bfloat16):
         assert dtype in (torch.bfloat16, torch.float32)
         self.args, self.device, self.dtype, self.w = args, torch.device(device), dtype, {}
 
-    def shapes(self):
-        a = self.args
+    def shapes(self, sd=None, rank=None):
+        """{name: shape}; sizes that only a checkpoint knows come from `sd`, or are `rank`."""
+        a, ds = self.args, self.args.design
         D = a.hidden_size
-        out = {"embed": (a.vocab_size, D), "final.norm": (D,), "head": (a.vocab_size, D)}
+        out = {"embed": (a.vocab_size, D), "final.norm": (D,)}
+        if not ds.tied:
+            out["head"] = (a.vocab_size, D)
+        if a.bigram:
+            out["bigram"] = (a.bigram["buckets"] + 1, D)
         for i, e in enumerate(a.layers):
-            out.update({f"l{i}.mix.{n}": s for n, s in MIXERS[e.type][0](e.mixer, D).items()})
-            out.update({f"l{i}.norm1": (D,), f"l{i}.dwa": (i + 2,)})
+            if e.weights_of is not None:
+                continue
+            free = {}
+            for n, s in MIXERS[e.type][0](e.mixer, D).items():
+                name = f"l{i}.mix.{n}"
+                have = tuple(sd[name].shape) if sd is not None and name in sd else None
+                for j, size in enumerate(s):
+                    if isinstance(size, str):
+                        free.setdefault(size, have[j] if have and len(have) == len(s) else rank or e.mixer["vdim"])
+                out[name] = tuple(free[x] if isinstance(x, str) else x for x in s)
+            out[f"l{i}.norm1"] = (D,)
+            if not ds.prenorm:
+                out[f"l{i}.dwa"] = (i + 2,)
             if e.mlp is not None:
                 ff = e.mlp["ff"]
-                out.update({f"l{i}.norm2": (D,), f"l{i}.mlp.up": (ff, D), f"l{i}.mlp.down": (D, ff), f"l{i}.mlp.act": (2,)})
+                out.update({f"l{i}.norm2": (D,), f"l{i}.mlp.up": (ff, D), f"l{i}.mlp.down": (D, ff)})
+                out.update({f"l{i}.mlp.act": (2,)} if ds.act == "xielu" else {f"l{i}.mlp.gate": (ff, D)})
         return out
 
     def load_state_dict(self, sd):
         """sd: {name: tensor} with exactly the model's tensors."""
-        shapes = self.shapes()
+        shapes = self.shapes(sd)
         missing, extra = sorted(set(shapes) - set(sd)), sorted(set(sd) - set(shapes))
         if missing or extra:
             raise ValueError(f"checkpoint tensors: missing {missing[:5]}, unexpected {extra[:5]}")
@@ -379,20 +496,20 @@ class HybridLM:
         return self
 
     @torch.no_grad()
-    def init_random(self, seed=0):
+    def init_random(self, seed=0, rank=None):
         """Seeded synthetic weights of the architecture."""
         g = torch.Generator(device=self.device).manual_seed(seed)
-        for n, s in self.shapes().items():
+        for n, s in self.shapes(rank=rank).items():
             r = torch.randn(s, generator=g, device=self.device, dtype=torch.float32)
             leaf = n.split(".", 1)[-1]
-            if leaf in ("norm1", "norm2", "norm") or leaf.endswith((".norm", "mix.D")):
+            if leaf in ("norm1", "norm2", "norm", "mix.norm") or leaf.endswith((".norm", "mix.D")):
                 r = 1.0 + 0.1 * r
             elif leaf == "dwa":
                 r = 0.05 * r
                 r[-1] += 1.0
-            elif leaf.endswith("dt.b"):
+            elif leaf.endswith("dt.b") or leaf == "mix.dt_bias":
                 r -= 2.0
-            elif len(s) == 2 and leaf not in ("mix.A_log", "mix.conv"):
+            elif len(s) == 2 and leaf != "mix.A_log" and not leaf.endswith("conv"):
                 r /= s[1] ** 0.5
             else:
                 r *= 0.3
@@ -403,6 +520,8 @@ class HybridLM:
 def make_prompt_cache(model, capacity, device=None):
     a = model.args
     if isinstance(model, HybridLM):
-        return [MIXERS[e.type][1](e.mixer, capacity, device or model.device, model.dtype) for e in a.layers]
+        device = device or model.device
+        caches = [MIXERS[e.type][1](e.mixer, capacity, device, model.dtype) for e in a.layers]
+        return caches + [TokenCache(capacity, device)] if a.bigram else caches
     device = device or model.model.embed_tokens.weight.device
     return [KVCache(a.num_key_value_heads, a.head_dim, capacity, device) for _ in model.model.layers]

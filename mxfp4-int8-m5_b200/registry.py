@@ -77,7 +77,7 @@ def _w4a8(cfg, path, dtype, device):
     return Bundle(args.model_type, fused, DEC.DecodeQwen3(fused), args.vocab_size, _lib.check_status)
 
 
-ARCHITECTURES = {"sebesun": _hybrid, "qwen3": _w4a8, "olmoe": _w4a8}
+ARCHITECTURES = {**{name: _hybrid for name in HM.DESIGNS}, "qwen3": _w4a8, "olmoe": _w4a8}
 
 
 def architecture(cfg):

@@ -1,5 +1,5 @@
 """Torch-level calls of the sequence-mixer kernels (include/scmx_mixers.h): matrix products for bfloat16 and float32 weights,
-row kernels, selective scan, retention, differential attention.  Every function takes CUDA tensors and launches on torch's
+row kernels, selective scan, retention, differential attention, gated delta rules, latent attention.  Every function takes CUDA tensors and launches on torch's
 current stream; there is no CPU path.  Activations are bfloat16 or float32 (the weights' type); the residual stream, norms,
 scores and recurrent states are float32."""
 import torch
@@ -32,11 +32,27 @@ def empty_rows(m, n, dtype, device):
 
 
 class XIELU:
-    """The two constants of an xIELU activation from its parameters (p, q): softplus(p) and 1/2 + softplus(q)."""
+    """Epilogue code and the two constants of an xIELU activation from its parameters (p, q): softplus(p) and 1/2 + softplus(q)."""
+
+    code = 1
 
     def __init__(self, act):
         p, q = (torch.nn.functional.softplus(act.detach().double().cpu())).tolist()
         self.a_pos, self.a_neg = p, 0.5 + q
+
+
+class GatedGELU:
+    """gelu(gate) up (tanh form) of a product with W = GatedGELU.weight(gate, up): half as many outputs as rows."""
+    code, a_pos, a_neg = 2, 0.0, 0.0
+
+    @staticmethod
+    def weight(gate, up):
+        """Rows in turns of 16 gate and 16 up, zero padded to whole turns."""
+        n, k = gate.shape
+        m = (n + 15) // 16 * 16
+        w = torch.zeros((2, m, k), dtype=gate.dtype, device=gate.device)
+        w[0, :n], w[1, :n] = gate, up
+        return w.view(2, m // 16, 16, k).transpose(0, 1).reshape(2 * m, k)
 
 
 class Linear:
@@ -53,6 +69,12 @@ class Linear:
             self.w[:, :self.K] = w
         self.dt = _dt(w)
 
+    def rows(self, r0, r1):
+        """The product with some of the rows, on the same memory."""
+        out = object.__new__(Linear)
+        out.N, out.K, out.w, out.dt = r1 - r0, self.K, self.w[r0:r1], self.dt
+        return out
+
     def _plan(self, M, splits, n_sm=148):
         """(tile, ranges of K computed side by side) for a product with few output tiles: the fewest bytes staged per SM, counting
         whole waves; at least 512 of K per range.  (0, 1): leave it to the kernel."""
@@ -64,33 +86,40 @@ class Linear:
                    key=lambda c: cost(*c))
 
     def __call__(self, x, out_dtype=None, act=None, tile=0, splits=None):
-        """x [M, K] -> [M, N] in out_dtype (default: the weights' type)."""
+        """x [M, K] -> [M, N] (N / 2 with a gated activation) in out_dtype (default: the weights' type)."""
         out_dtype = out_dtype or self.w.dtype
         M = x.shape[0]
         assert x.shape[1] == self.K and x.dtype == self.w.dtype and x.is_cuda
         if self.dt == 1:
             with _full_float32():
                 y = x @ self.w[:, :self.K].T
+            if act is not None and act.code == 2:
+                out = torch.empty((M, self.N // 2), dtype=y.dtype, device=y.device)
+                _lib.mcall("scmx_gated_gelu", _lib.ptr(y), y.stride(0), M, self.N // 2, _lib.ptr(out), _lib.stream())
+                return out
             if act is not None:
                 _lib.mcall("scmx_xielu", _lib.ptr(y), y.numel(), act.a_pos, act.a_neg, _lib.stream())
             return y
         if _ld(x) % 8 or x.data_ptr() % 16:
             x = empty_rows(M, self.K, x.dtype, x.device).copy_(x)
-        y = empty_rows(M, self.N, out_dtype, x.device)
+        nout = self.N // 2 if act is not None and act.code == 2 else self.N
+        y = empty_rows(M, nout, out_dtype, x.device)
         if tile == 0:
             tile, splits = self._plan(M, 1 if act is not None else splits)
         splits = splits or 1
         part = torch.empty(splits * M * ((self.N + 3) // 4 * 4), dtype=torch.float32, device=x.device) if splits > 1 else None
-        _lib.mcall("scmx_gemm_bf16", _lib.ptr(x), _ld(x), _lib.ptr(self.w), self.w.shape[1], M, self.N, self.K, int(act is not None),
-                   act.a_pos if act else 0.0, act.a_neg if act else 0.0, _lib.ptr(y), int(out_dtype == torch.float32), _round8(self.N), tile, splits,
+        _lib.mcall("scmx_gemm_bf16", _lib.ptr(x), _ld(x), _lib.ptr(self.w), self.w.shape[1], M, self.N, self.K, act.code if act else 0,
+                   act.a_pos if act else 0.0, act.a_neg if act else 0.0, _lib.ptr(y), int(out_dtype == torch.float32), _round8(nout), tile, splits,
                    _lib.ptr(part), _lib.ptr(_lib.mixer_status_buffer()), _lib.stream())
         return y
 
     def vec(self, x, act=None, conv=None, out=None):
-        """One float32 row [K] -> float32 [N]; conv = (weights [C, taps], bias [C], tail) for the convolution epilogue."""
+        """One float32 row [K] -> float32 [N] (N / 2 with a gated activation); conv = (weights [C, taps], bias [C] or None, tail) for
+        the convolution epilogue."""
         assert x.dtype == torch.float32 and x.numel() == self.K and x.is_contiguous()
-        out = torch.empty(self.N, dtype=torch.float32, device=x.device) if out is None else out
-        epi = 2 if conv is not None else int(act is not None)
+        epi = 2 if conv is not None else 0 if act is None else (0, 1, 3)[act.code]
+        if out is None:
+            out = torch.empty(self.N // 2 if epi == 3 else self.N, dtype=torch.float32, device=x.device)
         cw, cb, tail = conv if conv is not None else (None, None, None)
         _lib.mcall("scmx_gemv_x", _lib.ptr(self.w), self.w.shape[1], self.dt, _lib.ptr(x), self.N, self.K, epi, act.a_pos if act else 0.0,
                    act.a_neg if act else 0.0, _lib.ptr(cw), _lib.ptr(cb), _lib.ptr(tail), 0 if cw is None else cw.shape[0],
@@ -116,6 +145,19 @@ def embed(tokens, table, x, h=None):
                _lib.ptr(h), _lib.stream())
 
 
+def embed_pair(tokens, table, x, scale, pairs=None, rule=(1, 0, 0), prev=None):
+    """x [T, W] float32 <- scale table rows + pair-table rows, rule = (buckets, mul_prev, mul_cur); prev int64 [1] is advanced."""
+    _lib.require_cuda(tokens, table, x, pairs, prev)
+    _lib.mcall("scmx_embed_pair", _lib.ptr(tokens), _lib.ptr(table), _lib.ptr(pairs), _dt(table), table.shape[0], tokens.numel(), table.shape[1],
+               scale, *rule, _lib.ptr(prev), _lib.ptr(x), _lib.stream())
+
+
+def add_norm(y, x, w, mult, eps, h):
+    """x <- x + mult y in place (y None: unchanged); h = x / rms(x) w in h's type."""
+    _lib.mcall("scmx_add_norm", _lib.ptr(y), 0 if y is None else _ld(y), _lib.ptr(x), _lib.ptr(w), mult, eps, x.shape[0], x.shape[1], _lib.ptr(x),
+               _lib.ptr(h), _dt(h), _lib.stream())
+
+
 def res_norm(y, x, w, eps, x_out, h_out=None, average=None):
     """x_out = x + w * y / rms(y), or with average = (xs [n, T, W], weights [n], keep) the weighted sum of xs[: n - 1] and that
     value (stored at xs[n - 1] when keep)."""
@@ -134,7 +176,7 @@ def norm_rows(x, w, eps, dtype, rows=None):
 
 
 def conv_silu(x, w, b, tail):
-    """x [T, C] (row pitch free) -> silu(causal convolution); tail is advanced."""
+    """x [T, C] (row pitch free) -> silu(causal convolution); b may be None; tail is advanced."""
     T, C = x.shape
     out = empty_rows(T, C, x.dtype, x.device)
     _lib.mcall("scmx_conv_silu", _lib.ptr(x), _ld(x), _dt(x), T, C, w.shape[1], _lib.ptr(w), _lib.ptr(b), _lib.ptr(tail), _lib.ptr(out),
@@ -156,6 +198,85 @@ def scan_step(x, z, dbc, w_dt, dt_bias, A2, D, state, y):
     _lib.mcall("scmx_scan_step", _lib.ptr(x), _lib.ptr(z), _lib.ptr(dbc), _lib.ptr(w_dt.w), w_dt.w.shape[1], w_dt.dt, C, N, w_dt.K,
                _lib.ptr(dt_bias), _lib.ptr(A2), _lib.ptr(D), _lib.ptr(state), _lib.ptr(y), _lib.stream())
     return y
+
+
+DELTA_TC_MIN = 48           # shorter portions go token by token
+
+
+def delta(q, k, v, b, a, channel, nA, dt_bias, state, form=0):
+    """q, k [T, G d], v [T, H dv], b [T, H] -> o [T, H, dv] float32; a: decay logits [T, H], or float32 [T, H d] with `channel`; state
+    [H, d, dv] is advanced.  form: 0 automatic, 1 token by token, 2 chunks on tensor cores (bfloat16)."""
+    T, (H, d, dv) = q.shape[0], state.shape
+    o = torch.empty((T, H, dv), dtype=torch.float32, device=q.device)
+    assert not channel or a.dtype == torch.float32
+    nbytes = 0
+    if q.dtype == torch.bfloat16 and form != 1 and (form == 2 or T >= DELTA_TC_MIN):
+        nbytes = 0 if v.data_ptr() % 16 else _lib.mixers().scmx_delta_scratch(T, H, d, dv, _ld(v))
+    assert nbytes or form != 2, "no tensor-core form for these sizes"
+    scratch = torch.empty(nbytes, dtype=torch.uint8, device=q.device) if nbytes else None
+    _lib.mcall("scmx_delta", _lib.ptr(q), _ld(q), _lib.ptr(k), _ld(k), _lib.ptr(v), _ld(v), _lib.ptr(b), _ld(b), _lib.ptr(a), _ld(a), _dt(q), int(channel),
+               T, H, q.shape[1] // d, d, dv, _lib.ptr(nA), _lib.ptr(dt_bias), _lib.ptr(state), _lib.ptr(o), _lib.ptr(scratch), nbytes,
+               _lib.ptr(_lib.mixer_status_buffer()), _lib.stream())
+    return o
+
+
+def delta_step(q, k, v, b, a, g, wa, wg, nA, dt_bias, w, eps, state, y):
+    """One token; wa, wg: the low-rank second products (Linear) of a decay per channel, or None."""
+    H, d, dv = state.shape
+    _lib.mcall("scmx_delta_step", _lib.ptr(q), _lib.ptr(k), _lib.ptr(v), _lib.ptr(b), _lib.ptr(a), _lib.ptr(g), None if wa is None else _lib.ptr(wa.w),
+               0 if wa is None else wa.w.shape[1], 0 if wa is None else wa.K, None if wg is None else _lib.ptr(wg.w),
+               0 if wg is None else wg.w.shape[1], 0 if wg is None else wg.K, 0 if wa is None else wa.dt, H, q.numel() // d, d, dv, _lib.ptr(nA),
+               _lib.ptr(dt_bias), _lib.ptr(w), eps, _lib.ptr(state), _lib.ptr(y), _lib.stream())
+    return y
+
+
+def latent_append(y, Q, R, r, qw, cw, cs, eps, cache, cq_dtype, pos_dev=None):
+    """y [T, Q + R + r]: normalized query latents [T, Q]; latents and rotated key parts go to rows cache.offset .. of the cache."""
+    T = y.shape[0]
+    cq = empty_rows(T, Q, cq_dtype, y.device)
+    _lib.mcall("scmx_latent_append", _lib.ptr(y), _ld(y), _dt(y), _dt(cache.c), _dt(cq), T, Q, R, r, _lib.ptr(qw), _lib.ptr(cw), _lib.ptr(cs), cs.shape[0],
+               eps, cache.offset, _lib.ptr(pos_dev), _lib.ptr(cq), _ld(cq), _lib.ptr(cache.c), cache.c.shape[1], cache.capacity, _lib.stream())
+    return cq
+
+
+def latent_rows(q, wuk, wuv, cs, cache, H, d, r, dv, window, scale, out_dtype, pos_dev=None, n_sm=148):
+    """q [T, H (d + r)] (parts not rotated) at positions cache.offset .. -> [T, H dv], through queries in the latent space."""
+    T, R, dev = q.shape[0], wuk.K, q.device
+    qa = torch.empty((T, H, R + r), dtype=torch.float32, device=dev)
+    pos, pd = cache.offset, _lib.ptr(pos_dev)
+    _lib.mcall("scmx_latent_absorb", _lib.ptr(q), _ld(q), _dt(q), _lib.ptr(wuk.w), wuk.w.shape[1], wuk.dt, _lib.ptr(cs), cs.shape[0], T, H, d, R, r, pos, pd,
+               _lib.ptr(qa), _lib.stream())
+    groups = -(-H // (4 if H <= 16 else 8))
+    nsplit = max(1, min(32, 2 * n_sm // (groups * T)))
+    part = torch.empty((T, H, nsplit, R + 2), dtype=torch.float32, device=dev)
+    _lib.mcall("scmx_latent_rows", _lib.ptr(qa), _lib.ptr(cache.c), cache.c.shape[1], _dt(cache.c), T, pos, pd, cache.capacity, window, H, R, r, scale,
+               nsplit, _lib.ptr(part), _lib.stream())
+    o = empty_rows(T, H * dv, out_dtype, dev)
+    _lib.mcall("scmx_latent_value", _lib.ptr(part), _lib.ptr(wuv.w), wuv.w.shape[1], wuv.dt, T, pos, pd, cache.capacity, window, H, R, dv, nsplit,
+               _lib.ptr(o), _ld(o), _dt(o), _lib.stream())
+    return o
+
+
+LATENT_TC_MIN = 32          # shorter portions are attended in the latent space
+
+
+def latent_prompt_supported(q, d, r, dv, scale):
+    return False
+    return q.dtype == torch.bfloat16 and not (d % 8 or r % 8 or dv % 8) and d <= 128 and r <= 64 and dv <= 128 and scale > 0
+
+
+def latent_prompt(q, ukv, cs, cache, H, d, r, dv, R, window, scale):
+    """The same for a bfloat16 prompt portion on tensor cores: keys and values of every visible position are products of its latent
+    (ukv: W_uk over W_uv); q's rotated parts are turned in place."""
+    T, pos = q.shape[0], cache.offset
+    k0 = max(0, pos + 1 - window) if window else 0
+    rows = cache.c[k0:pos + T]
+    kv = ukv(rows[:, :R])
+    _lib.mcall("scmx_latent_rotate", _lib.ptr(q), _ld(q), _dt(q), _lib.ptr(cs[pos:]), T, H, d, r, _lib.stream())
+    o = torch.empty((T, H * dv), dtype=q.dtype, device=q.device)
+    _lib.mcall("scmx_latent_attn", _lib.ptr(q), _ld(q), _lib.ptr(kv), _ld(kv), _lib.ptr(rows[:, _round8(R):]) if r else None, rows.shape[1], T, pos, k0,
+               window, H, d, r, dv, scale, _lib.ptr(o), _lib.ptr(_lib.mixer_status_buffer()), _lib.stream())
+    return o
 
 
 def rotary_table(base, dims, rows, device):
@@ -183,10 +304,11 @@ def retention(q, k, v, cs, dims, kscale, decay, state, form=0):
     return o
 
 
-def head_norm_gate(o, g, eps):
+def head_norm_gate(o, g, eps, w=None, gate=0):
+    """o [T, H, dv] / rms * w * gate(g), gate 0 = SiLU, 1 = sigmoid."""
     T, H, dv = o.shape
     out = torch.empty((T, H * dv), dtype=g.dtype, device=o.device)
-    _lib.mcall("scmx_head_norm_gate", _lib.ptr(o), _lib.ptr(g), _ld(g), _dt(g), T, H, dv, eps, _lib.ptr(out), _lib.stream())
+    _lib.mcall("scmx_head_norm_gate", _lib.ptr(o), _lib.ptr(g), _ld(g), _dt(g), _lib.ptr(w), gate, T, H, dv, eps, _lib.ptr(out), _lib.stream())
     return out
 
 
