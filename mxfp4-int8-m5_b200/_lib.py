@@ -253,7 +253,12 @@ def _raise_status(st):
         raise ScmxError(f"device-side wait ran out: {describe_status(v[0])} (CTA or rank {v[1]}, thread {v[2]})")
 
 
-_GEMM_ROLES = {41: "retention chunk product waiting for operands", 42: "retention chunk kernel waiting for the product",
+_GEMM_ROLES = {51: "latent attention producer waiting for a free key tile", 52: "latent attention producer waiting for a free value tile",
+               53: "latent attention MMA thread waiting for operands", 54: "latent attention MMA thread waiting for softmax weights",
+               55: "latent attention softmax warp waiting for scores", 56: "latent attention softmax warp waiting for the last product",
+               61: "delta producer waiting for a free stage", 62: "delta MMA thread waiting for operands",
+               63: "delta MMA thread waiting for states or corrections", 64: "delta warp waiting for a product",
+               41: "retention chunk product waiting for operands", 42: "retention chunk kernel waiting for the product",
                43: "retention producer waiting for a free stage", 44: "retention MMA thread waiting for operands or weights",
                45: "retention warp waiting for scores or outputs",
                31: "attention producer waiting for a free key tile", 32: "attention producer waiting for a free value tile",

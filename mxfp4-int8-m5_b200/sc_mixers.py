@@ -261,7 +261,6 @@ LATENT_TC_MIN = 32          # shorter portions are attended in the latent space
 
 
 def latent_prompt_supported(q, d, r, dv, scale):
-    return False
     return q.dtype == torch.bfloat16 and not (d % 8 or r % 8 or dv % 8) and d <= 128 and r <= 64 and dv <= 128 and scale > 0
 
 
