@@ -1149,16 +1149,15 @@ def main():
     ap.add_argument("--no-overlap", action="store_true", help="decode weights on the main stream instead of a side stream")
     ap.add_argument("--no-pdl", action="store_true", help="launch without programmatic stream serialization")
     ap.add_argument("--dense-only", action="store_true", help="skip the roofline / decode / MoE / CPU sections")
-    ap.add_argument("--workload", default="all", choices=["all", "moe5", "hybrid"],
-                    help="moe5: only the large-MoE stress section; hybrid: hybrid decoders beside the closest existing model")
-    ap.add_argument("--sizes", default="", help="with --workload hybrid: widths to run, with commas between them")
+    ap.add_argument("--workload", default="all", choices=["all", "moe5", "hybrid", "fabezen"],
+                    help="moe5: only the large-MoE stress section; hybrid, fabezen: these decoders beside the closest existing model")
+    ap.add_argument("--sizes", default="", help="with --workload hybrid or fabezen: widths to run, with commas between them")
     ap.add_argument("--case", choices=["gemm", "gemmw4", "gemmlib", "rows", "gemv", "gemvbig", "gemvlist", "moe", "moe512", "ep1", "models", "decodestep", "decodechain"], help="run one small kernel case (for profiler captures) and exit")
     args = ap.parse_args()
-    if args.workload == "hybrid":
+    if args.workload in ("hybrid", "fabezen"):
         import torch
-        import bench_hybrid
-        bench_hybrid.run(importlib.import_module("mxfp4-int8-m5_b200"), torch, peaks(), ClockSampler(0),
-                         args.sizes.split(",") if args.sizes else None)
+        importlib.import_module("bench_" + args.workload).run(importlib.import_module("mxfp4-int8-m5_b200"), torch, peaks(), ClockSampler(0),
+                                                                  args.sizes.split(",") if args.sizes else None)
     elif args.case:
         run_case(args)
     elif args.impl == "reference":

@@ -75,9 +75,13 @@ class Timer:
         self.torch.cuda.empty_cache()
 
 
-def bench_kernels(pkg, torch, pk, s, T=2048, ctx=8192):
+def bench_kernels(pkg, torch, pk, s):
     """Kernels of the hybrid model and the like kernels of the closest model at the same sizes."""
-    X, S, G, HM, F = pkg.sc_mixers, pkg.sc_kernels, pkg.sc_decode, pkg.host_model, pkg.sc_format
+    return dict(hybrid=hybrid_kernels(pkg, torch, pk, s), qwen3_style=qwen3_kernels(pkg, torch, pk, s))
+
+
+def hybrid_kernels(pkg, torch, pk, s, T=2048, ctx=8192):
+    X, HM = pkg.sc_mixers, pkg.host_model
     W, C, N, R, BF, F32 = s["width"], s["inner"], s["state"], s["rank"], torch.bfloat16, torch.float32
     t = Timer(torch, pk)
     rnd = lambda *sh, dtype=BF: (torch.randn(*sh, device="cuda") * 0.5).to(dtype)          # noqa: E731
@@ -187,10 +191,14 @@ def bench_kernels(pkg, torch, pk, s, T=2048, ctx=8192):
         y, x, w, xs, dwa = rnd(1, W, dtype=F32), rnd(1, W, dtype=F32), rnd(W, dtype=F32), rnd(6, 1, W, dtype=F32), rnd(6, dtype=F32)
         return lambda: X.res_norm(y, x, w, 1e-5, x, None, (xs, dwa, True))
     t.kernel("decode residual norm + average of 6", rn1, W * 4 * 9)
-    ours = t.rows
+    return t.rows
 
-    # ---- like kernels of the closest model
+
+def qwen3_kernels(pkg, torch, pk, s, T=2048, ctx=8192):
+    S, G, HM, F = pkg.sc_kernels, pkg.sc_decode, pkg.host_model, pkg.sc_format
+    W, H, G_, ff, BF = s["width"], s["heads"], s["kv"], s["ff"], torch.bfloat16
     t = Timer(torch, pk)
+    rnd = lambda *sh, dtype=BF: (torch.randn(*sh, device="cuda") * 0.5).to(dtype)          # noqa: E731
 
     def igemm(name, n, k, epi):
         def make(i):
@@ -240,50 +248,56 @@ def bench_kernels(pkg, torch, pk, s, T=2048, ctx=8192):
         x, w = rnd(1, W), rnd(W)
         return lambda: S.rmsnorm_quant(x, w, 1e-6, 1)
     t.kernel("decode rmsnorm quant", rq1, 5 * W)
-    return dict(hybrid=ours, qwen3_style=t.rows)
+    return t.rows
 
 
-def bench_model(pkg, torch, pk, s, lengths=(512, 2048), n_tok=64):
-    """Whole models of LAYERS layers: prompt tokens/s (graph replay, last position's logits included) and greedy tokens/s after a
-    512-token prompt."""
-    HM, FQ, DEC, FH = pkg.host_model, pkg.fused_qwen3, pkg.decode, pkg.fused_hybrid
-    out, t = {}, Timer(torch, pk)
+def measure_model(torch, pk, fused, dec, vocab, lengths=(512, 2048), n_tok=64):
+    """Prompt tokens/s (graph replay, last position's logits included) and greedy tokens/s after a 512-token prompt."""
+    t = Timer(torch, pk)
+    ids = torch.randint(0, vocab, (1, max(lengths) + n_tok), device="cuda")
+    cache, res = fused.make_cache(max(lengths) + n_tok + 8), {}
 
-    def measure(fused, dec, vocab):
-        ids = torch.randint(0, vocab, (1, max(lengths) + n_tok), device="cuda")
-        cache, res = fused.make_cache(max(lengths) + n_tok + 8), {}
+    def prefill(n):
+        for c in cache:
+            c.offset = 0
+        return fused.logits(fused.hidden(ids[:, :n], cache)[:, -1:])
+    for n in lengths:
+        ms = t.replay_ms(t.graph([lambda: prefill(n)]))
+        res[f"prefill_{n}_tok_s"] = round(n / ms * 1e3)
+        res[f"prefill_{n}_ms"] = round(ms, 3)
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    with torch.no_grad():
+        for _ in range(3):                                  # the first pass captures the step
+            prefill(512)
+            e0.record()
+            dec.generate(ids[:, 512:513], cache, n_tok)
+            e1.record()
+            torch.cuda.synchronize()
+    res["decode_tok_s"] = round(n_tok / e0.elapsed_time(e1) * 1e3, 1)
+    return res
 
-        def prefill(n):
-            for c in cache:
-                c.offset = 0
-            return fused.logits(fused.hidden(ids[:, :n], cache)[:, -1:])
-        for n in lengths:
-            ms = t.replay_ms(t.graph([lambda: prefill(n)]))
-            res[f"prefill_{n}_tok_s"] = round(n / ms * 1e3)
-            res[f"prefill_{n}_ms"] = round(ms, 3)
-        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-        with torch.no_grad():
-            for _ in range(3):                                  # the first pass captures the step
-                prefill(512)
-                e0.record()
-                dec.generate(ids[:, 512:513], cache, n_tok)
-                e1.record()
-                torch.cuda.synchronize()
-        res["decode_tok_s"] = round(n_tok / e0.elapsed_time(e1) * 1e3, 1)
-        return res
 
-    model = HM.HybridLM(HM.HybridArgs.from_config(hybrid_config(s))).init_random(0)
-    fused = FH.FusedHybrid(model)
-    out["hybrid"] = measure(fused, DEC.DecodeHybrid(fused), s["vocab"])
-    out["hybrid"]["weight_gb"] = round(sum(w.numel() * 2 for w in model.w.values()) / 1e9, 3)
+def measure_hybrid(pkg, torch, pk, cfg, **init):
+    """A hybrid decoder of a configuration, random weights."""
+    model = pkg.host_model.HybridLM(pkg.host_model.HybridArgs.from_config(cfg)).init_random(0, **init)
+    fused = pkg.fused_hybrid.FusedHybrid(model)
+    out = measure_model(torch, pk, fused, pkg.decode.DecodeHybrid(fused), cfg["vocab"])
+    out["weight_gb"] = round(sum(w.numel() * 2 for w in model.w.values()) / 1e9, 3)
     del model, fused
     torch.cuda.empty_cache()
+    return out
+
+
+def bench_model(pkg, torch, pk, s):
+    """Whole models of LAYERS layers."""
+    HM, FQ, DEC = pkg.host_model, pkg.fused_qwen3, pkg.decode
+    out = {"hybrid": measure_hybrid(pkg, torch, pk, hybrid_config(s))}
     a = HM.ModelArgs(s["width"], s["ff"], LAYERS, s["heads"], s["kv"], 128, 1e-6, 1e6, s["vocab"], False)
     with torch.device("cuda"):
         model = HM.CausalLM(a)
     model.init_random(0)
     fused = FQ.FusedQwen3(model, FQ.pack_model(model, on_device=True))
-    out["qwen3_style"] = measure(fused, DEC.DecodeQwen3(fused), s["vocab"])
+    out["qwen3_style"] = measure_model(torch, pk, fused, DEC.DecodeQwen3(fused), s["vocab"])
     out["qwen3_style"]["weight_gb"] = round(fused.weight_bytes() / 1e9, 3)
     del model, fused
     torch.cuda.empty_cache()

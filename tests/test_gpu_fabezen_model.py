@@ -211,15 +211,12 @@ def test_delta_remembers_a_far_token(scmx):
             W[f"l{i}.mix.b"].mul_(0.05)
     m, T = Model(scmx, cfg, F32, 600, edit=edit), 520
     a = tokens(cfg, T, 7)
-    b = a[:500] + [(a[500] + 1) % 60] + a[501:]
-    c = a[:10] + [(a[10] + 1) % 60] + a[11:]
-    base = m.oracle(a)[-1]
-    for other in (b, c):
-        want = base - m.oracle(other)[-1]
-        for cuts in ([T], [300, 2, 217, 1]):
-            got = m.run(a, cuts)[-1] - m.run(other, cuts)[-1]
-            assert np.abs(got - want).max() < 0.05 * np.abs(want).max() + 2e-5
-    assert np.abs(base - m.oracle(b)[-1]).max() > 1e-3
+    b = a[:10] + [(a[10] + 1) % 60] + a[11:]
+    want = m.oracle(a)[-1] - m.oracle(b)[-1]
+    assert np.abs(want).max() > 0.01
+    for cuts in ([T], [300, 2, 217, 1]):
+        got = m.run(a, cuts)[-1] - m.run(b, cuts)[-1]
+        assert np.abs(got - want).max() < 0.05 * np.abs(want).max(), cuts
 
 
 def test_wanted_places(scmx):
