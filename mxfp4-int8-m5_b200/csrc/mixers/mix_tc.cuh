@@ -38,6 +38,38 @@ __device__ __forceinline__ void umma_bf16_ts(uint32_t d_tmem, uint32_t a_tmem, u
         ::"r"(d_tmem), "r"(a_tmem), "l"(bdesc), "r"(idesc), "r"(accumulate)
         : "memory");
 }
+// Forms for a whole warp that stays converged, so that descriptors live in uniform registers: only the lane with `on` issues.  Small
+// products (N = 64) need them: a single diverged thread takes longer to assemble an instruction than the tensor core to run it.
+__device__ __forceinline__ uint32_t elect_lane() {
+    uint32_t on;
+    asm volatile("{\n\t.reg .pred p;\n\telect.sync _|p, 0xffffffff;\n\tselp.b32 %0, 1, 0, p;\n\t}" : "=r"(on));
+    return on;
+}
+__device__ __forceinline__ void umma_bf16_on(uint32_t on, uint32_t d_tmem, uint64_t adesc, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
+    asm volatile(
+        "{\n\t.reg .pred p, q;\n\t"
+        "setp.ne.b32 p, %4, 0;\n\t"
+        "setp.ne.b32 q, %5, 0;\n\t"
+        "@q tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
+        ::"r"(d_tmem), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate), "r"(on)
+        : "memory");
+}
+__device__ __forceinline__ void umma_bf16_ts_on(uint32_t on, uint32_t d_tmem, uint32_t a_tmem, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
+    asm volatile(
+        "{\n\t.reg .pred p, q;\n\t"
+        "setp.ne.b32 p, %4, 0;\n\t"
+        "setp.ne.b32 q, %5, 0;\n\t"
+        "@q tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
+        ::"r"(d_tmem), "r"(a_tmem), "l"(bdesc), "r"(idesc), "r"(accumulate), "r"(on)
+        : "memory");
+}
+__device__ __forceinline__ void umma_commit_on(uint32_t on, uint32_t bar) {
+    asm volatile(
+        "{\n\t.reg .pred q;\n\tsetp.ne.b32 q, %1, 0;\n\t"
+        "@q tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n\t}" ::"r"(bar), "r"(on)
+        : "memory");
+}
+
 // A stored with M contiguous (bit 15), B with N contiguous (bit 16): rows of K, 64 values of M or N per 128-byte swizzle row.
 constexpr uint32_t IDESC_A_MN = 1u << 15, IDESC_B_MN = 1u << 16;
 // Descriptor of such a tile: 8 rows of K are 1024 bytes apart (stride offset), the next 64 values of N `block` bytes (leading
