@@ -301,7 +301,7 @@ static int run_delta_step(DeltaStepArgs a, cudaStream_t st) {
 using namespace scmx;
 
 extern "C" int64_t scmx_delta_scratch(int64_t n, int H, int d, int dv, int64_t ldv) {
-    return n > 0 && H > 0 && d > 0 && dv > 0 && delta_tc_supported(n, H, d, dv, ldv) ? delta_tc_scratch(n, H, d) : 0;
+    return n > 0 && H > 0 && d > 0 && dv > 0 && delta_tc_supported(n, H, d, dv, ldv) ? delta_tc_scratch(n, H, d, dv) : 0;
 }
 
 extern "C" int scmx_delta(const void* q, int64_t ldq, const void* k, int64_t ldk, const void* v, int64_t ldv, const void* b, int64_t ldb,
@@ -318,7 +318,7 @@ extern "C" int scmx_delta(const void* q, int64_t ldq, const void* k, int64_t ldk
     const cudaStream_t st = (cudaStream_t)stream;
     if (scratch != nullptr) {
         SCMX_REQUIRE(dt == 0 && status && delta_tc_supported(n, H, d, dv, ldv), SCMX_ELIMIT, "delta: no tensor-core form for head sizes %d / %d", d, dv);
-        SCMX_REQUIRE(((uintptr_t)v & 15) == 0 && ((uintptr_t)scratch & 255) == 0 && scratch_bytes >= delta_tc_scratch(n, H, d), SCMX_EINVAL,
+        SCMX_REQUIRE(((uintptr_t)v & 15) == 0 && ((uintptr_t)scratch & 255) == 0 && scratch_bytes >= delta_tc_scratch(n, H, d, dv), SCMX_EINVAL,
                      "delta: scratch of %lld bytes or an unaligned pointer", (long long)scratch_bytes);
         return delta_tc(a, channel != 0, scratch, status, st);
     }

@@ -16,7 +16,7 @@ struct DeltaArgs {
 };
 
 bool delta_tc_supported(int64_t n, int H, int d, int dv, int64_t ldv);
-int64_t delta_tc_scratch(int64_t n, int H, int d);
+int64_t delta_tc_scratch(int64_t n, int H, int d, int dv);
 int delta_tc(const DeltaArgs& a, bool channel, void* scratch, int32_t* status, cudaStream_t st);
 
 }  // namespace scmx

@@ -4,12 +4,13 @@
 //   (I + N) U = beta (V - (c K) S),   N_ij = beta_i (k_i . c_i / c_j k_j) for j < i,   T = (I + N)^-1 diag(beta)
 //   U = T V - W S,  W = T (c K);   O = (c Q) S + B U,  B_ij = q_i . c_i / c_j k_j for j <= i;   S' = c_end S + E^T U,  E = c_end / c K
 //
-// delta_prep_kernel    per chunk and head, all in parallel: unit vectors, decays, N, B, T, W.  Ratios c_i / c_j are formed by running
-//                      products of decays, so nothing overflows however strong the decay is
-// delta_state_kernel   per head and 128 values, chunk after chunk: S^T lives in tensor memory (a lane per value), three products per
-//                      chunk with S or U as the tensor-memory operand
-// Operands that enter the recurrence are stored as two bfloat16 terms (16 significant bits; three MMAs per product, two with V,
-// which is bfloat16 as projected); S itself is carried in float32.  Waits are bounded (status word codes 61..64).
+// delta_prep_*_kernel  per chunk and head, all in parallel: unit vectors, decays, N, B, the inverse, W, T V (one kernel per kind of
+//                      decay).  Ratios c_i / c_j are products of decays, so that nothing overflows however strong the decay is
+// delta_state_kernel   per head and 128 values, chunk after chunk: S^T lives in tensor memory (a lane per value), the products of a
+//                      chunk take S or U as the tensor-memory operand
+// Operands that enter the recurrence are stored as two bfloat16 terms (16 significant bits, three MMAs per product; raw keys,
+// queries and values are bfloat16 as projected and take one term); S itself is carried in float32.  Waits are bounded (status word
+// codes 61..64).
 #include "mix_delta.cuh"
 #include "mix_tc.cuh"
 
@@ -17,17 +18,17 @@ namespace scmx {
 
 constexpr int DC = 64;                   // tokens per chunk
 constexpr int DC_BLK = 64 * 128;         // bytes of a [64 rows x 64 values] operand block
-constexpr int DP_THREADS = 512;
 constexpr int DP_PITCH = 68;             // row pitch of the 64 x 64 matrices in shared memory
 
 struct DeltaTcArgs {
     DeltaArgs p;
     bf16_t *wh, *wl, *qh, *ql, *eh, *el;     // [items][64][D]: -W, c Q, E
-    bf16_t *th, *tl, *bh, *bl;               // [items][64][64]
+    bf16_t *bh, *bl;                         // [items][64][64]: B
+    float* uv;                               // [items][value tiles][64][128]: T V
     float* gend;                             // [items][D]: c at the chunk's end
     int32_t* status;
     uint64_t wait_ns;
-    int nc;                                  // chunks; item = chunk * H + head
+    int nc, nvt;                             // chunks, item = chunk * H + head; tiles of 128 values
 };
 
 // Two or four values as two bfloat16 terms.
@@ -49,32 +50,252 @@ __device__ __forceinline__ void mma_split(float (&d)[4], const uint32_t (&ah)[4]
     mma_16816(d, al, bh[0], bh[1]);
 }
 
-// Shared memory of the preparation, in floats.  Per channel decays: K, Q, G hold k, q, g, later k f, q f, k e with the decay products
-// f from the start of a block of 16 tokens and e to its end; PB the products of whole blocks.  One decay per head: K, Q stay, the
-// products are per token (F, E), RAT holds the ratios within a block.
-template <int D, bool CH>
-struct DpSmem {
-    static constexpr int P = D + 16;         // row pitch: eight lanes of a 128-bit load fall into distinct banks
-    static constexpr int K = 0, Q = K + 64 * P, G = Q + 64 * P, N = G + (CH ? 64 * P : 64), B = N + 64 * DP_PITCH, X = B + 64 * DP_PITCH,
-                         T = X + 64 * DP_PITCH, BETA = T + 32 * 36, PB = BETA + 64, F = PB + (CH ? 4 * D : 64), E = F + 64, RAT = E + 64,
-                         FLOATS = RAT + (CH ? 0 : 64 * 17);
-};
-
 __device__ __forceinline__ void split4(const float4 v, uint32_t& h0, uint32_t& h1, uint32_t& l0, uint32_t& l1) {
     split2(v.x, v.y, h0, l0);
     split2(v.z, v.w, h1, l1);
 }
 __device__ __forceinline__ float4 mul4(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
 __device__ __forceinline__ float4 mul4(float4 a, float b) { return make_float4(a.x * b, a.y * b, a.z * b, a.w * b); }
-__device__ __forceinline__ void half_bar() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void part_bar() { asm volatile("bar.sync 1, %0;" ::"n"(N) : "memory"); }
 
-template <int D, bool CH>
-__global__ void __launch_bounds__(DP_THREADS, 1) delta_prep_kernel(const DeltaTcArgs a) {
-    using L = DpSmem<D, CH>;
-    constexpr int P = L::P;
+// 2^(nA softplus(z) log2 e) with z2 = z log2 e: the logarithm of the sum directly in base two.
+__device__ __forceinline__ float decay_f32(float nA, float z2) {
+    float l;
+    asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(l) : "f"(1.0f + ex2_approx(-fabsf(z2))));
+    return ex2_approx(nA * (fmaxf(z2, 0.0f) + l));
+}
+
+// Operands of one 16 x 16 (A) or 16 x 8 (B) block in shared memory as two terms.  Inner index: lane t4 holds t4 + 4 e of the 16.
+__device__ __forceinline__ void block_a(const float* m, int lane, uint32_t (&ah)[4], uint32_t (&al)[4]) {
+    const float *x = m + (lane >> 2) * DP_PITCH + (lane & 3), *y = x + 8 * DP_PITCH;
+    split2(x[0], x[4], ah[0], al[0]);
+    split2(y[0], y[4], ah[1], al[1]);
+    split2(x[8], x[12], ah[2], al[2]);
+    split2(y[8], y[12], ah[3], al[3]);
+}
+template <int PITCH>
+__device__ __forceinline__ void block_b(const float* m, int lane, uint32_t (&bh)[2], uint32_t (&bl)[2]) {
+    const float* x = m + (lane & 3) * PITCH + (lane >> 2);
+    split2(x[0], x[4 * PITCH], bh[0], bl[0]);
+    split2(x[8 * PITCH], x[12 * PITCH], bh[1], bl[1]);
+}
+
+// X = (I + N)^-1 by the first four warps: diagonal blocks of 16 (a lane per column), then 32 from 16 and 64 from 32 with
+// X21 = -X22 (N21 X11), a warp per 8 columns.  Only entries below the diagonal of N are read; X above it is zero within blocks of 32.
+// sT: four areas of [32][8] floats.
+__device__ __forceinline__ void invert_unit_lower(const float* sN, float* sX, float* sT, int tid) {
+    const int lane = tid & 31, warp = tid >> 5, g = lane >> 2, t4 = lane & 3;
+    {
+        const int b0 = 16 * warp;
+        float x[16];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+            float s = i == lane ? 1.0f : 0.0f, s2 = 0.0f;
+#pragma unroll
+            for (int j = 0; j < i; ++j) {
+                if (j & 1) s2 = fmaf(-sN[(b0 + i) * DP_PITCH + b0 + j], x[j], s2);
+                else s = fmaf(-sN[(b0 + i) * DP_PITCH + b0 + j], x[j], s);
+            }
+            x[i] = s + s2;
+        }
+        if (lane < 16)
+#pragma unroll
+            for (int i = 0; i < 16; ++i) sX[(b0 + i) * DP_PITCH + b0 + lane] = x[i];
+    }
+    part_bar<128>();
+    float* tile = sT + warp * 256;
+    auto keep = [&](const float (&d)[4], float* out, int pitch, float sign) {      // a 16 x 8 result
+        *reinterpret_cast<float2*>(out + g * pitch + 2 * t4) = make_float2(sign * d[0], sign * d[1]);
+        *reinterpret_cast<float2*>(out + (g + 8) * pitch + 2 * t4) = make_float2(sign * d[2], sign * d[3]);
+    };
+    uint32_t ah[4], al[4], bh[2], bl[2];
+    {
+        const int b0 = 32 * (warp >> 1), c = b0 + 8 * (warp & 1);
+        float d[4] = {};
+        block_a(sN + (b0 + 16) * DP_PITCH + b0, lane, ah, al);
+        block_b<DP_PITCH>(sX + b0 * DP_PITCH + c, lane, bh, bl);
+        mma_split(d, ah, al, bh, bl);
+        keep(d, tile, 8, 1.0f);
+        __syncwarp();
+        float x[4] = {};
+        block_a(sX + (b0 + 16) * DP_PITCH + b0 + 16, lane, ah, al);
+        block_b<8>(tile, lane, bh, bl);
+        mma_split(x, ah, al, bh, bl);
+        keep(x, sX + (b0 + 16) * DP_PITCH + c, DP_PITCH, -1.0f);
+        const float zero[4] = {};
+        keep(zero, sX + b0 * DP_PITCH + c + 16, DP_PITCH, 1.0f);      // above the diagonal, read by the products of 32
+    }
+    part_bar<128>();
+    float d[2][4] = {}, x[2][4] = {};
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+        block_b<DP_PITCH>(sX + 16 * k * DP_PITCH + 8 * warp, lane, bh, bl);
+#pragma unroll
+        for (int m = 0; m < 2; ++m) {
+            block_a(sN + (32 + 16 * m) * DP_PITCH + 16 * k, lane, ah, al);
+            mma_split(d[m], ah, al, bh, bl);
+        }
+    }
+    __syncwarp();
+    keep(d[0], tile, 8, 1.0f);
+    keep(d[1], tile + 128, 8, 1.0f);
+    __syncwarp();
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+        block_b<8>(tile + 128 * k, lane, bh, bl);
+#pragma unroll
+        for (int m = 0; m < 2; ++m) {
+            block_a(sX + (32 + 16 * m) * DP_PITCH + 32 + 16 * k, lane, ah, al);
+            mma_split(x[m], ah, al, bh, bl);
+        }
+    }
+    keep(x[0], sX + 32 * DP_PITCH + 8 * warp, DP_PITCH, -1.0f);
+    keep(x[1], sX + 48 * DP_PITCH + 8 * warp, DP_PITCH, -1.0f);
+}
+
+// T = X diag(beta) as two terms in the order of the A operand: per block of 16 columns, word t4 + 4 u holds columns t4 + 8 u and
+// t4 + 4 + 8 u.
+constexpr int DT_PITCH = 36;             // words per row
+__device__ __forceinline__ void pack_t(const float* sX, const float* beta, uint32_t* th, uint32_t* tl, int tid, int n) {
+    for (int u = tid; u < 64 * 32; u += n) {
+        const int i = u >> 5, w = u & 31, c = 16 * (w >> 3) + (w & 3) + 8 * ((w >> 2) & 1);
+        if (16 * (w >> 3) > i) continue;             // blocks above the diagonal are not read
+        split2(c <= i ? sX[i * DP_PITCH + c] * beta[c] : 0.0f, c + 4 <= i ? sX[i * DP_PITCH + c + 4] * beta[c + 4] : 0.0f, th[i * DT_PITCH + w],
+               tl[i * DT_PITCH + w]);
+    }
+}
+
+// The lower triangle of a 64 x 64 matrix as two terms, by `n` threads.
+__device__ __forceinline__ void store_lower(const float* m, bf16_t* hi, bf16_t* lo, int item, int tid, int n) {
+    for (int u = tid; u < 512; u += n) {
+        const int i = u >> 3, j = 8 * (u & 7);
+        uint32_t hw[4], lw[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int c = j + 2 * e;
+            split2(c <= i ? m[i * DP_PITCH + c] : 0.0f, c + 1 <= i ? m[i * DP_PITCH + c + 1] : 0.0f, hw[e], lw[e]);
+        }
+        const int64_t o = ((int64_t)item * DC + i) * 64 + j;
+        *reinterpret_cast<uint4*>(hi + o) = make_uint4(hw[0], hw[1], hw[2], hw[3]);
+        *reinterpret_cast<uint4*>(lo + o) = make_uint4(lw[0], lw[1], lw[2], lw[3]);
+    }
+}
+
+// Values of 64 tokens, columns v0 .. v0 + 127, -> shared memory, zeros outside.
+constexpr int DV_PITCH = 136;
+template <int NT>
+__device__ __forceinline__ void load_values(const DeltaArgs& p, bf16_t* sV, int h, int64_t t0, int nt, int v0, int tid) {
+#pragma unroll
+    for (int i = 0; i < 1024 / NT; ++i) {
+        const int u = tid + NT * i, t = u >> 4, c = 8 * (u & 15);
+        uint4 w = make_uint4(0, 0, 0, 0);
+        if (t < nt && v0 + c < p.dv) w = *reinterpret_cast<const uint4*>(static_cast<const bf16_t*>(p.v) + (t0 + t) * p.ldv + (int64_t)h * p.dv + v0 + c);
+        *reinterpret_cast<uint4*>(sV + t * DV_PITCH + c) = w;
+    }
+}
+
+// One warp: T Y for 16 columns of Y, all 64 rows.  Inner index as in T; columns: a lane's four results of a row are neighbours, 4 t4 ..
+// column(j0, n, bh, bl): the operand of tokens j0 + t4 + 4 e, column 4 (g / 2) + (g & 1) + 2 n, in one (TERMS = 1) or two terms.
+// put(row, four results).
+template <int TERMS, typename Col, typename Put>
+__device__ __forceinline__ void lower_product(const uint32_t* th, const uint32_t* tl, int lane, Col column, Put put) {
+    const int g = lane >> 2, t4 = lane & 3;
+    float acc[4][2][4] = {};
+#pragma unroll
+    for (int jb = 0; jb < 4; ++jb) {
+        uint32_t bh[2][2], bl[2][2];
+#pragma unroll
+        for (int n = 0; n < 2; ++n) column(16 * jb, n, bh[n], bl[n]);
+#pragma unroll
+        for (int I = jb; I < 4; ++I) {
+            const int o = (16 * I + g) * DT_PITCH + 8 * jb + t4;
+            const uint32_t ah[4] = {th[o], th[o + 8 * DT_PITCH], th[o + 4], th[o + 8 * DT_PITCH + 4]};
+            const uint32_t al[4] = {tl[o], tl[o + 8 * DT_PITCH], tl[o + 4], tl[o + 8 * DT_PITCH + 4]};
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+                mma_16816(acc[I][n], ah, bh[n][0], bh[n][1]);
+                mma_16816(acc[I][n], al, bh[n][0], bh[n][1]);
+                if (TERMS == 2) mma_16816(acc[I][n], ah, bl[n][0], bl[n][1]);
+            }
+        }
+    }
+#pragma unroll
+    for (int I = 0; I < 4; ++I)
+#pragma unroll
+        for (int e = 0; e < 2; ++e)
+            put(16 * I + g + 8 * e, make_float4(acc[I][0][2 * e], acc[I][0][2 * e + 1], acc[I][1][2 * e], acc[I][1][2 * e + 1]));
+}
+
+// T V of the staged values, 16 columns per warp task.
+__device__ __forceinline__ void values_product(const DeltaTcArgs& a, const uint32_t* th, const uint32_t* tl, const bf16_t* sV, int item, int v0, int group, int lane) {
+    const int g = lane >> 2, t4 = lane & 3, ca = 16 * group + 4 * (g >> 1) + (g & 1), co = 16 * group + 4 * t4;
+    float* out = a.uv + ((int64_t)item * a.nvt + (v0 >> 7)) * DC * 128;
+    lower_product<1>(th, tl, lane,
+        [&](int j0, int n, uint32_t (&bh)[2], uint32_t (&)[2]) {
+            const bf16_t* v = sV + (j0 + t4) * DV_PITCH + ca + 2 * n;
+            bh[0] = (uint32_t)v[0] | (uint32_t)v[4 * DV_PITCH] << 16;
+            bh[1] = (uint32_t)v[8 * DV_PITCH] | (uint32_t)v[12 * DV_PITCH] << 16;
+        },
+        [&](int row, float4 r) { *reinterpret_cast<float4*>(out + row * 128 + co) = r; });
+}
+
+// -W: results of a row as two terms.
+template <int D>
+__device__ __forceinline__ void store_w(const DeltaTcArgs& a, int item, int row, int c, float4 r) {
+    uint32_t h0, l0, h1, l1;
+    split2(-r.x, -r.y, h0, l0);
+    split2(-r.z, -r.w, h1, l1);
+    const int64_t o = ((int64_t)item * DC + row) * D + c;
+    *reinterpret_cast<uint2*>(a.wh + o) = make_uint2(h0, h1);
+    *reinterpret_cast<uint2*>(a.wl + o) = make_uint2(l0, l1);
+}
+
+// Eight values as two terms, 16 bytes each.
+__device__ __forceinline__ void store_terms8(bf16_t* hi, bf16_t* lo, float4 u, float4 v) {
+    uint32_t hw[4], lw[4];
+    split4(u, hw[0], hw[1], lw[0], lw[1]);
+    split4(v, hw[2], hw[3], lw[2], lw[3]);
+    *reinterpret_cast<uint4*>(hi) = make_uint4(hw[0], hw[1], hw[2], hw[3]);
+    *reinterpret_cast<uint4*>(lo) = make_uint4(lw[0], lw[1], lw[2], lw[3]);
+}
+
+// The sums of x and y over the warp, in six shuffles.
+__device__ __forceinline__ float2 warp_sum2(float x, float y, int lane) {
+    const bool up = (lane & 16) != 0;
+    float s = (up ? y : x) + __shfl_xor_sync(0xffffffffu, up ? x : y, 16);
+#pragma unroll
+    for (int o = 8; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+    const float other = __shfl_xor_sync(0xffffffffu, s, 16);
+    return up ? make_float2(other, s) : make_float2(s, other);
+}
+
+// Row block I and key block b <= I of the pair-th pair of blocks of 16.
+__device__ __forceinline__ void block_pair(int pair, int& I, int& b) {
+    I = pair == 0 ? 0 : pair < 3 ? 1 : pair < 6 ? 2 : 3;
+    b = pair - I * (I + 1) / 2;
+}
+
+// ---- a decay per key channel ----------------------------------------------------------------------------------------------
+// Shared memory, in floats.  K, Q, G hold k, q, g, later k f, q f, k e with the decay products f from the start of a block of 16
+// tokens and e to its end; PB the products of whole blocks, PI their reciprocals.  Within a block c_i / c_j = f_i e_j / product; a
+// block with a channel below 2^-64 forms its ratios by running products instead.
+constexpr int DPC_THREADS = 512;
+template <int D>
+struct DpcSmem {
+    static constexpr int P = D + 16;         // row pitch: eight lanes of a 128-bit load fall into distinct banks
+    static constexpr int K = 0, Q = K + 64 * P, G = Q + 64 * P, N = G + 64 * P, B = N + 64 * DP_PITCH, X = B + 64 * DP_PITCH, T = X + 64 * DP_PITCH,
+                         V = T + 32 * 36, BETA = V + 64 * DV_PITCH / 2, PB = BETA + 64, PI = PB + 4 * D, STRONG = PI + 4 * D, FLOATS = STRONG + 4;
+};
+
+template <int D>
+__global__ void __launch_bounds__(DPC_THREADS, 1) delta_prep_channel_kernel(const DeltaTcArgs a) {
+    using L = DpcSmem<D>;
+    constexpr int P = L::P, VC = D / 32;
     extern __shared__ __align__(16) float sm[];
-    float *sk = sm + L::K, *sq = sm + L::Q, *sg = sm + L::G, *sN = sm + L::N, *sB = sm + L::B, *sX = sm + L::X, *sT = sm + L::T;
-    float *beta = sm + L::BETA, *pb = sm + L::PB, *sf = sm + L::F, *se = sm + L::E, *rat = sm + L::RAT;
+    float *sk = sm + L::K, *sq = sm + L::Q, *sg = sm + L::G, *sN = sm + L::N, *sB = sm + L::B, *sX = sm + L::X;
+    float *beta = sm + L::BETA, *pb = sm + L::PB, *pi = sm + L::PI;
+    bf16_t* sV = reinterpret_cast<bf16_t*>(sm + L::V);
+    int* strong = reinterpret_cast<int*>(sm + L::STRONG);
     pdl_launch_dependents();
     pdl_wait();
     const DeltaArgs& p = a.p;
@@ -84,132 +305,134 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prep_kernel(const DeltaTc
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     // ---- unit vectors, decays, beta; tokens past the end become neutral (k = q = 0, beta = 0, decay 1)
     {
-        constexpr int V = D / 32;
-        const int e = V * lane;
+        const int e = VC * lane;
         const bool in = e < p.d;
         const bf16_t *q = static_cast<const bf16_t*>(p.q) + (int64_t)kh * p.d + e, *k = static_cast<const bf16_t*>(p.k) + (int64_t)kh * p.d + e;
-        float x[4][V], y[4][V], z[4][V], bl = 0.0f, al = 0.0f, dtb[V];
+        const float* ar = static_cast<const float*>(p.a) + (int64_t)h * p.d + e;
+        uint32_t qw[4][VC / 2], kw[4][VC / 2];
+        float z[4][VC], bl = 0.0f, dtb[VC];
 #pragma unroll
         for (int r = 0; r < 4; ++r) {
             const int t = warp + 16 * r;
 #pragma unroll
-            for (int i = 0; i < V; ++i) x[r][i] = y[r][i] = z[r][i] = 0.0f;
-            if (t < nt && in) {
-                // rows are 4-byte aligned, decay rows 8-byte (host side)
+            for (int i = 0; i < VC / 2; ++i) qw[r][i] = kw[r][i] = 0;
 #pragma unroll
-                for (int i = 0; i < V; i += 2) {
-                    const uint32_t u = *reinterpret_cast<const uint32_t*>(q + (t0 + t) * p.ldq + i), w = *reinterpret_cast<const uint32_t*>(k + (t0 + t) * p.ldk + i);
-                    x[r][i] = bf16_lo(u); x[r][i + 1] = bf16_hi(u);
-                    y[r][i] = bf16_lo(w); y[r][i + 1] = bf16_hi(w);
-                    if (CH) {
-                        const float2 v = *reinterpret_cast<const float2*>(static_cast<const float*>(p.a) + (t0 + t) * p.lda + (int64_t)h * p.d + e + i);
-                        z[r][i] = v.x; z[r][i + 1] = v.y;
-                    }
+            for (int i = 0; i < VC; ++i) z[r][i] = 0.0f;
+            if (t < nt && in) {                  // rows are aligned for these loads (host side)
+                if (VC == 4) {
+                    *reinterpret_cast<uint2*>(qw[r]) = *reinterpret_cast<const uint2*>(q + (t0 + t) * p.ldq);
+                    *reinterpret_cast<uint2*>(kw[r]) = *reinterpret_cast<const uint2*>(k + (t0 + t) * p.ldk);
+                    *reinterpret_cast<float4*>(z[r]) = *reinterpret_cast<const float4*>(ar + (t0 + t) * p.lda);
+                } else {
+                    qw[r][0] = *reinterpret_cast<const uint32_t*>(q + (t0 + t) * p.ldq);
+                    kw[r][0] = *reinterpret_cast<const uint32_t*>(k + (t0 + t) * p.ldk);
+                    *reinterpret_cast<float2*>(z[r]) = *reinterpret_cast<const float2*>(ar + (t0 + t) * p.lda);
                 }
             }
-            if (lane == r && t < nt) {           // lane r keeps token r's scalars
-                bl = ldf(static_cast<const bf16_t*>(p.b) + (t0 + t) * p.ldb + h);
-                if (!CH) al = ldf(static_cast<const bf16_t*>(p.a) + (t0 + t) * p.lda + h);
-            }
         }
-        const float qs = rsqrtf((float)p.d), nA2 = p.nA[h] * 1.4426950408889634f;
+        if (lane < 4 && warp + 16 * lane < nt) bl = ldf(static_cast<const bf16_t*>(p.b) + (t0 + warp + 16 * lane) * p.ldb + h);
 #pragma unroll
-        for (int i = 0; i < V; ++i) dtb[i] = CH ? (in ? p.dtb[(int64_t)h * p.d + e + i] : 0.0f) : p.dtb[h];
+        for (int i = 0; i < VC; ++i) dtb[i] = in ? p.dtb[(int64_t)h * p.d + e + i] : 0.0f;
+        const float qs = rsqrtf((float)p.d), nA = p.nA[h];
+        load_values<DPC_THREADS>(p, sV, h, t0, nt, 0, tid);
+        if (tid < 4) strong[tid] = 0;
 #pragma unroll
         for (int r = 0; r < 4; ++r) {
             const int t = warp + 16 * r;
-            float qq = 0.0f, kk = 0.0f;
+            float x[VC], y[VC], g[VC], qq = 0.0f, kk = 0.0f;
 #pragma unroll
-            for (int i = 0; i < V; ++i) {
-                qq = fmaf(x[r][i], x[r][i], qq);
-                kk = fmaf(y[r][i], y[r][i], kk);
+            for (int i = 0; i < VC / 2; ++i) {
+                x[2 * i] = bf16_lo(qw[r][i]); x[2 * i + 1] = bf16_hi(qw[r][i]);
+                y[2 * i] = bf16_lo(kw[r][i]); y[2 * i + 1] = bf16_hi(kw[r][i]);
             }
-            // two sums in six shuffles: the halves of the warp take one each
-            const bool up = (lane & 16) != 0;
-            float s = (up ? kk : qq) + __shfl_xor_sync(0xffffffffu, up ? qq : kk, 16);
 #pragma unroll
-            for (int o = 8; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
-            const float other = __shfl_xor_sync(0xffffffffu, s, 16);
-            const float iq = qs * rsqrtf((up ? other : s) + 1e-6f), ik = rsqrtf((up ? s : other) + 1e-6f);
-#pragma unroll
-            for (int i = 0; i < V; ++i) {
-                sq[t * P + e + i] = x[r][i] * iq;
-                sk[t * P + e + i] = y[r][i] * ik;
-                if (CH) sg[t * P + e + i] = t < nt ? ex2_approx(nA2 * softplus_f32(z[r][i] + dtb[i])) : 1.0f;
+            for (int i = 0; i < VC; ++i) {
+                qq = fmaf(x[i], x[i], qq);
+                kk = fmaf(y[i], y[i], kk);
+                g[i] = t < nt ? decay_f32(nA, (z[r][i] + dtb[i]) * 1.4426950408889634f) : 1.0f;
+            }
+            const float2 s = warp_sum2(qq, kk, lane);
+            const float iq = qs * rsqrtf(s.x + 1e-6f), ik = rsqrtf(s.y + 1e-6f);
+            const int o = t * P + e;
+            if (VC == 4) {
+                *reinterpret_cast<float4*>(sq + o) = make_float4(x[0] * iq, x[1] * iq, x[VC - 2] * iq, x[VC - 1] * iq);
+                *reinterpret_cast<float4*>(sk + o) = make_float4(y[0] * ik, y[1] * ik, y[VC - 2] * ik, y[VC - 1] * ik);
+                *reinterpret_cast<float4*>(sg + o) = make_float4(g[0], g[1], g[VC - 2], g[VC - 1]);
+            } else {
+                *reinterpret_cast<float2*>(sq + o) = make_float2(x[0] * iq, x[1] * iq);
+                *reinterpret_cast<float2*>(sk + o) = make_float2(y[0] * ik, y[1] * ik);
+                *reinterpret_cast<float2*>(sg + o) = make_float2(g[0], g[1]);
             }
         }
-        if (lane < 4) {
-            const int t = warp + 16 * lane;
-            beta[t] = t < nt ? sigmoid_f32(bl) : 0.0f;
-            if (!CH) sg[t] = t < nt ? ex2_approx(nA2 * softplus_f32(al + dtb[0])) : 1.0f;
-        }
+        if (lane < 4) beta[warp + 16 * lane] = warp + 16 * lane < nt ? sigmoid_f32(bl) : 0.0f;
     }
     __syncthreads();
-    if (CH) {
-        // ---- diagonal blocks of N and B: a warp carries four keys j of a block, c_i / c_j k_j, from i = j on; lanes split the channels
-        constexpr int V = D / 32;
-        const int b0 = 16 * (warp >> 2), jg = 4 * (warp & 3);
-        float kc[4][V];
-#pragma unroll
-        for (int j = 0; j < 4; ++j)
-#pragma unroll
-            for (int i = 0; i < V; ++i) kc[j][i] = sk[(b0 + jg + j) * P + V * lane + i];
-        for (int i0 = jg; i0 < 16; i0 += 4) {
-            float s[32];
-#pragma unroll
-            for (int ii = 0; ii < 4; ++ii) {
-                const int o = (b0 + i0 + ii) * P + V * lane;
-                float k[V], q[V], g[V];
-                if (V == 4) {
-                    *reinterpret_cast<float4*>(k) = *reinterpret_cast<const float4*>(sk + o);
-                    *reinterpret_cast<float4*>(q) = *reinterpret_cast<const float4*>(sq + o);
-                    *reinterpret_cast<float4*>(g) = *reinterpret_cast<const float4*>(sg + o);
-                } else {
-                    *reinterpret_cast<float2*>(k) = *reinterpret_cast<const float2*>(sk + o);
-                    *reinterpret_cast<float2*>(q) = *reinterpret_cast<const float2*>(sq + o);
-                    *reinterpret_cast<float2*>(g) = *reinterpret_cast<const float2*>(sg + o);
-                }
-#pragma unroll
-                for (int j = 0; j < 4; ++j) {
-                    float n = 0.0f, m = 0.0f;
-#pragma unroll
-                    for (int i = 0; i < V; ++i) {
-                        if (i0 > jg || ii > j) kc[j][i] *= g[i];
-                        n = fmaf(kc[j][i], k[i], n);
-                        m = fmaf(kc[j][i], q[i], m);
-                    }
-                    s[8 * ii + 2 * j] = n;
-                    s[8 * ii + 2 * j + 1] = m;
-                }
-            }
-            // 32 sums over the warp, one per lane: lane bits from the highest choose the half that a lane keeps
-#pragma unroll
-            for (int n = 16; n > 0; n >>= 1) {
-                const bool up = (lane & n) != 0;
-#pragma unroll
-                for (int i = 0; i < n; ++i) {
-                    const float keep = up ? s[i + n] : s[i], give = up ? s[i] : s[i + n];
-                    s[i] = keep + __shfl_xor_sync(0xffffffffu, give, n);
-                }
-            }
-            const int i = b0 + i0 + (lane >> 3), j = b0 + jg + ((lane >> 1) & 3);
-            if (lane & 1) {
-                if (i >= j) sB[i * DP_PITCH + j] = s[0];
-            } else if (i > j) {
-                sN[i * DP_PITCH + j] = beta[i] * s[0];
-            }
-        }
-        __syncthreads();
-        // ---- decay products within the blocks, a thread per channel and block
-        for (int u = tid; u < 4 * D; u += DP_THREADS) {
-            const int c = u % D, b = u / D;
-            float *k = sk + 16 * b * P + c, *q = sq + 16 * b * P + c, *g = sg + 16 * b * P + c;
-            float kk[16], gg[16], f = 1.0f, e = 1.0f;
+    // ---- decay products within the blocks, a thread per channel and block
+    {
+        const int c = tid % D, b = tid / D;
+        const bool work = b < 4;
+        float *k = sk + 16 * b * P + c, *q = sq + 16 * b * P + c, *g = sg + 16 * b * P + c;
+        float kk[16], gg[16], whole = 1.0f;
+        if (work) {
 #pragma unroll
             for (int t = 0; t < 16; ++t) {
                 kk[t] = k[t * P];
                 gg[t] = g[t * P];
+                whole *= gg[t];
             }
+            if (whole < 5.4e-20f) strong[b] = 1;
+        }
+        __syncthreads();
+        if (strong[0] | strong[1] | strong[2] | strong[3]) {
+            // diagonal blocks by running products: a warp carries four keys j, c_i / c_j k_j, from i = j on; lanes split the channels
+            const int b0 = 16 * (warp >> 2), jg = 4 * (warp & 3);
+            if (strong[warp >> 2]) {
+                float kc[4][VC];
+#pragma unroll
+                for (int j = 0; j < 4; ++j)
+#pragma unroll
+                    for (int i = 0; i < VC; ++i) kc[j][i] = sk[(b0 + jg + j) * P + VC * lane + i];
+                for (int i0 = jg; i0 < 16; ++i0) {
+                    const int o = (b0 + i0) * P + VC * lane;
+                    float s[8];
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                        float n = 0.0f, m = 0.0f;
+#pragma unroll
+                        for (int i = 0; i < VC; ++i) {
+                            if (i0 > jg + j) kc[j][i] *= sg[o + i];
+                            n = fmaf(kc[j][i], sk[o + i], n);
+                            m = fmaf(kc[j][i], sq[o + i], m);
+                        }
+                        s[2 * j] = n;
+                        s[2 * j + 1] = m;
+                    }
+                    // eight sums over the warp: lane bits 4, 2, 1 choose, the others add
+#pragma unroll
+                    for (int n = 4; n > 0; n >>= 1) {
+                        const bool up = (lane & n) != 0;
+#pragma unroll
+                        for (int i = 0; i < n; ++i) {
+                            const float keep = up ? s[i + n] : s[i], give = up ? s[i] : s[i + n];
+                            s[i] = keep + __shfl_xor_sync(0xffffffffu, give, n);
+                        }
+                    }
+                    s[0] += __shfl_xor_sync(0xffffffffu, s[0], 8);
+                    s[0] += __shfl_xor_sync(0xffffffffu, s[0], 16);
+                    const int i = b0 + i0, j = b0 + jg + ((lane >> 1) & 3);
+                    if (lane < 8) {
+                        if (lane & 1) {
+                            if (i >= j) sB[i * DP_PITCH + j] = s[0];
+                        } else if (i > j) {
+                            sN[i * DP_PITCH + j] = beta[i] * s[0];
+                        }
+                    }
+                }
+            }
+            __syncthreads();
+        }
+        if (work) {
+            float f = 1.0f, e = 1.0f;
 #pragma unroll
             for (int t = 0; t < 16; ++t) {
                 f *= gg[t];
@@ -217,248 +440,277 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prep_kernel(const DeltaTc
                 q[t * P] *= f;
             }
             pb[b * D + c] = f;
+            pi[b * D + c] = __fdividef(1.0f, f);
 #pragma unroll
             for (int t = 15; t >= 0; --t) {
                 g[t * P] = kk[t] * e;
                 e *= gg[t];
             }
         }
-    } else {
-        // ---- the same per token: products from the block's start, to its end, and between its tokens
-        if (tid < 64) {
-            const int b0 = tid & ~15, j = tid & 15;
-            float f = 1.0f, e = 1.0f, r = 1.0f;
-            for (int t = 0; t < 16; ++t) {
-                const float g = sg[b0 + t];
-                if (t <= j) f *= g;
-                if (t > j) {
-                    e *= g;
-                    r *= g;
-                }
-                rat[tid * 17 + t] = r;           // key j, token t >= j
-            }
-            sf[tid] = f;
-            se[tid] = e;
-            if (j == 15) pb[tid >> 4] = f;
-        }
     }
     __syncthreads();
-    // ---- N and B by blocks of 16 rows x 8 keys: row block I against key block b (the diagonal only with one decay per head).  The inner
-    // index is permuted so that a lane's four values of a 16-step are neighbours.
-    {
-        const int g = lane >> 2, t4 = lane & 3;
-        constexpr int TASKS = CH ? 12 : 20;
-        for (int task = warp; task < TASKS; task += 16) {
-            const int pair = task >> 1, j0 = 8 * (task & 1);
-            int I, b;
-            if (CH) {
-                I = pair == 0 ? 1 : pair < 3 ? 2 : 3;
-                b = pair == 0 ? 0 : pair < 3 ? pair - 1 : pair - 3;
-            } else {
-                I = pair == 0 ? 0 : pair < 3 ? 1 : pair < 6 ? 2 : 3;
-                b = pair - I * (I + 1) / 2;
-            }
-            const float *kr = sk + (16 * I + g) * P + 4 * t4, *qr = sq + (16 * I + g) * P + 4 * t4, *kc = (CH ? sg : sk) + (16 * b + j0 + g) * P + 4 * t4;
-            float n[4] = {}, m[4] = {};
+    // ---- N and B by blocks of 16 x 16.  The inner index is permuted so that a lane's four values of a 16-step are neighbours.
+    if (warp < 10) {
+        int I, b;
+        block_pair(warp, I, b);
+        if (I != b || !strong[b]) {
+            const int g = lane >> 2, t4 = lane & 3;
+            const float *kr = sk + (16 * I + g) * P + 4 * t4, *qr = sq + (16 * I + g) * P + 4 * t4, *kc = sg + (16 * b + g) * P + 4 * t4;
+            float n[2][4] = {}, m[2][4] = {};
 #pragma unroll 2
             for (int s = 0; s < D; s += 16) {
-                uint32_t ah[4], al[4], bh[2], bl[2];
-                float4 v = *reinterpret_cast<const float4*>(kc + s);
-                if (CH) {                        // decay of the blocks between
-                    if (I - b >= 2) v = mul4(v, *reinterpret_cast<const float4*>(pb + (b + 1) * D + s + 4 * t4));
-                    if (I - b == 3) v = mul4(v, *reinterpret_cast<const float4*>(pb + (b + 2) * D + s + 4 * t4));
+                uint32_t ah[4], al[4], bh[2][2], bl[2][2];
+                float4 v[2] = {*reinterpret_cast<const float4*>(kc + s), *reinterpret_cast<const float4*>(kc + 8 * P + s)};
+                if (I != b + 1) {                // decay of the blocks between, or the block's own product taken back
+                    float4 r = *reinterpret_cast<const float4*>((I == b ? pi + b * D : pb + (b + 1) * D) + s + 4 * t4);
+                    if (I == b + 3) r = mul4(r, *reinterpret_cast<const float4*>(pb + (b + 2) * D + s + 4 * t4));
+                    v[0] = mul4(v[0], r);
+                    v[1] = mul4(v[1], r);
                 }
-                split4(v, bh[0], bh[1], bl[0], bl[1]);
+#pragma unroll
+                for (int j = 0; j < 2; ++j) split4(v[j], bh[j][0], bh[j][1], bl[j][0], bl[j][1]);
                 split4(*reinterpret_cast<const float4*>(kr + s), ah[0], ah[2], al[0], al[2]);
                 split4(*reinterpret_cast<const float4*>(kr + 8 * P + s), ah[1], ah[3], al[1], al[3]);
-                mma_split(n, ah, al, bh, bl);
+#pragma unroll
+                for (int j = 0; j < 2; ++j) mma_split(n[j], ah, al, bh[j], bl[j]);
                 split4(*reinterpret_cast<const float4*>(qr + s), ah[0], ah[2], al[0], al[2]);
                 split4(*reinterpret_cast<const float4*>(qr + 8 * P + s), ah[1], ah[3], al[1], al[3]);
-                mma_split(m, ah, al, bh, bl);
+#pragma unroll
+                for (int j = 0; j < 2; ++j) mma_split(m[j], ah, al, bh[j], bl[j]);
             }
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int i = 16 * I + g + 8 * (e >> 1), j = 16 * b + j0 + 2 * t4 + (e & 1);
-                float r = 1.0f;
-                if (!CH) {
-                    if (I == b) r = i >= j ? rat[j * 17 + (i & 15)] : 0.0f;
-                    else {
-                        r = sf[i] * se[j];
-                        for (int u = b + 1; u < I; ++u) r *= pb[u];
-                    }
-                }
-                if (i > j) sN[i * DP_PITCH + j] = beta[i] * n[e] * r;
-                if (i >= j) sB[i * DP_PITCH + j] = m[e] * r;
+            for (int u = 0; u < 8; ++u) {
+                const int e = u & 3, i = 16 * I + g + 8 * (e >> 1), j = 16 * b + 8 * (u >> 2) + 2 * t4 + (e & 1);
+                if (i > j) sN[i * DP_PITCH + j] = beta[i] * n[u >> 2][e];
+                if (i >= j) sB[i * DP_PITCH + j] = m[u >> 2][e];
             }
         }
     }
     __syncthreads();
-    if (warp < 8) {
-        // ---- X = (I + N)^-1: diagonal blocks of 16 (a lane per column), then 32 from 16 and 64 from 32: X21 = -X22 (N21 X11)
-        if (warp < 4) {
-            const int b0 = 16 * warp;
-            float x[16];
-#pragma unroll
-            for (int i = 0; i < 16; ++i) {
-                float s = i == lane ? 1.0f : 0.0f;
-#pragma unroll
-                for (int j = 0; j < i; ++j) s = fmaf(-sN[(b0 + i) * DP_PITCH + b0 + j], x[j], s);
-                x[i] = s;
-            }
-            if (lane < 16)
-#pragma unroll
-                for (int i = 0; i < 16; ++i) sX[(b0 + i) * DP_PITCH + b0 + lane] = x[i];
-        }
-        half_bar();
-        {
-            const int pr = tid >> 7, r = (tid >> 3) & 15, c = 2 * (tid & 7), b0 = 32 * pr;
-            float s0 = 0.0f, s1 = 0.0f;
-#pragma unroll
-            for (int k = 0; k < 16; ++k) {
-                const float n = sN[(b0 + 16 + r) * DP_PITCH + b0 + k];
-                const float2 xx = *reinterpret_cast<const float2*>(sX + (b0 + k) * DP_PITCH + b0 + c);
-                s0 = fmaf(n, xx.x, s0);
-                s1 = fmaf(n, xx.y, s1);
-            }
-            *reinterpret_cast<float2*>(sT + (pr * 16 + r) * 36 + c) = make_float2(s0, s1);
-            half_bar();
-            s0 = s1 = 0.0f;
-#pragma unroll
-            for (int k = 0; k < 16; ++k) {
-                const float n = sX[(b0 + 16 + r) * DP_PITCH + b0 + 16 + k];
-                const float2 tt = *reinterpret_cast<const float2*>(sT + (pr * 16 + k) * 36 + c);
-                s0 = fmaf(n, tt.x, s0);
-                s1 = fmaf(n, tt.y, s1);
-            }
-            *reinterpret_cast<float2*>(sX + (b0 + 16 + r) * DP_PITCH + b0 + c) = make_float2(-s0, -s1);
-            *reinterpret_cast<float2*>(sX + (b0 + r) * DP_PITCH + b0 + 16 + c) = make_float2(0.0f, 0.0f);   // read by the products of 32
-            half_bar();
-        }
-        {
-            const int r = tid >> 3, c = 4 * (tid & 7);
-            float4 s = make_float4(0, 0, 0, 0);
-#pragma unroll 16
-            for (int k = 0; k < 32; ++k) {
-                const float n = sN[(32 + r) * DP_PITCH + k];
-                const float4 x = *reinterpret_cast<const float4*>(sX + k * DP_PITCH + c);
-                s.x = fmaf(n, x.x, s.x); s.y = fmaf(n, x.y, s.y); s.z = fmaf(n, x.z, s.z); s.w = fmaf(n, x.w, s.w);
-            }
-            *reinterpret_cast<float4*>(sT + r * 36 + c) = s;
-            half_bar();
-            s = make_float4(0, 0, 0, 0);
-#pragma unroll 16
-            for (int k = 0; k < 32; ++k) {
-                const float n = sX[(32 + r) * DP_PITCH + 32 + k];
-                const float4 x = *reinterpret_cast<const float4*>(sT + k * 36 + c);
-                s.x = fmaf(n, x.x, s.x); s.y = fmaf(n, x.y, s.y); s.z = fmaf(n, x.z, s.z); s.w = fmaf(n, x.w, s.w);
-            }
-            *reinterpret_cast<float4*>(sX + (32 + r) * DP_PITCH + c) = make_float4(-s.x, -s.y, -s.z, -s.w);
-        }
+    if (tid < 128) {
+        invert_unit_lower(sN, sX, sm + L::T, tid);
     } else {
         // ---- meanwhile: c Q, E, B and c at the chunk's end
-        for (int u = tid - 256; u < 64 * (D / 8); u += 256) {
+        for (int u = tid - 128; u < 64 * (D / 8); u += DPC_THREADS - 128) {
             const int t = u / (D / 8), c = 8 * (u % (D / 8)), b = t >> 4;
             const int64_t o = ((int64_t)item * DC + t) * D + c;
-            uint32_t hw[4], lw[4];
+            const float4 *pf = reinterpret_cast<const float4*>(pb + c), *q = reinterpret_cast<const float4*>(sq + t * P + c), *e = reinterpret_cast<const float4*>(sg + t * P + c);
+            float4 q0 = q[0], q1 = q[1], e0 = e[0], e1 = e[1];
 #pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                float4 v = *reinterpret_cast<const float4*>(sq + t * P + c + 4 * e);
-                if (!CH) v = mul4(v, sf[t]);
-                for (int w = 0; w < b; ++w) v = CH ? mul4(v, *reinterpret_cast<const float4*>(pb + w * D + c + 4 * e)) : mul4(v, pb[w]);
-                split4(v, hw[2 * e], hw[2 * e + 1], lw[2 * e], lw[2 * e + 1]);
+            for (int w = 0; w < 4; ++w) {
+                const float4 f0 = pf[w * (D / 4)], f1 = pf[w * (D / 4) + 1];
+                if (w < b) {
+                    q0 = mul4(q0, f0);
+                    q1 = mul4(q1, f1);
+                }
+                if (w > b) {
+                    e0 = mul4(e0, f0);
+                    e1 = mul4(e1, f1);
+                }
             }
-            *reinterpret_cast<uint4*>(a.qh + o) = make_uint4(hw[0], hw[1], hw[2], hw[3]);
-            *reinterpret_cast<uint4*>(a.ql + o) = make_uint4(lw[0], lw[1], lw[2], lw[3]);
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                float4 v = *reinterpret_cast<const float4*>((CH ? sg : sk) + t * P + c + 4 * e);
-                if (!CH) v = mul4(v, se[t]);
-                for (int w = b + 1; w < 4; ++w) v = CH ? mul4(v, *reinterpret_cast<const float4*>(pb + w * D + c + 4 * e)) : mul4(v, pb[w]);
-                split4(v, hw[2 * e], hw[2 * e + 1], lw[2 * e], lw[2 * e + 1]);
-            }
-            *reinterpret_cast<uint4*>(a.eh + o) = make_uint4(hw[0], hw[1], hw[2], hw[3]);
-            *reinterpret_cast<uint4*>(a.el + o) = make_uint4(lw[0], lw[1], lw[2], lw[3]);
+            store_terms8(a.qh + o, a.ql + o, q0, q1);
+            store_terms8(a.eh + o, a.el + o, e0, e1);
         }
-        for (int u = tid - 256; u < 512; u += 256) {
-            const int i = u >> 3, j = 8 * (u & 7);
-            uint32_t hw[4], lw[4];
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int c = j + 2 * e;
-                split2(c <= i ? sB[i * DP_PITCH + c] : 0.0f, c + 1 <= i ? sB[i * DP_PITCH + c + 1] : 0.0f, hw[e], lw[e]);
-            }
-            const int64_t o = ((int64_t)item * DC + i) * 64 + j;
-            *reinterpret_cast<uint4*>(a.bh + o) = make_uint4(hw[0], hw[1], hw[2], hw[3]);
-            *reinterpret_cast<uint4*>(a.bl + o) = make_uint4(lw[0], lw[1], lw[2], lw[3]);
-        }
-        for (int c = tid - 256; c < D; c += 256)
-            a.gend[(int64_t)item * D + c] = CH ? pb[c] * pb[D + c] * pb[2 * D + c] * pb[3 * D + c] : pb[0] * pb[1] * pb[2] * pb[3];
+        store_lower(sB, a.bh, a.bl, item, tid - 128, DPC_THREADS - 128);
+        for (int c = tid - 128; c < D; c += DPC_THREADS - 128) a.gend[(int64_t)item * D + c] = pb[c] * pb[D + c] * pb[2 * D + c] * pb[3 * D + c];
     }
     __syncthreads();
-    // ---- T = X diag(beta)
-    {
-        const int i = tid >> 3, j = 8 * (tid & 7);
-        uint32_t hw[4], lw[4];
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int c = j + 2 * e;
-            split2(c <= i ? sX[i * DP_PITCH + c] * beta[c] : 0.0f, c + 1 <= i ? sX[i * DP_PITCH + c + 1] * beta[c + 1] : 0.0f, hw[e], lw[e]);
+    uint32_t *th = reinterpret_cast<uint32_t*>(sN), *tl = th + 64 * DT_PITCH;      // over N and B
+    pack_t(sX, beta, th, tl, tid, DPC_THREADS);
+    __syncthreads();
+    // ---- -W = -X (beta c K) and T V
+    for (int v0 = 0; v0 < p.dv; v0 += 128) {
+        if (v0 > 0) {
+            __syncthreads();
+            load_values<DPC_THREADS>(p, sV, h, t0, nt, v0, tid);
+            __syncthreads();
         }
-        const int64_t o = ((int64_t)item * DC + i) * 64 + j;
-        *reinterpret_cast<uint4*>(a.th + o) = make_uint4(hw[0], hw[1], hw[2], hw[3]);
-        *reinterpret_cast<uint4*>(a.tl + o) = make_uint4(lw[0], lw[1], lw[2], lw[3]);
+        const int vg = min(8, (p.dv - v0 + 15) / 16), wgroups = v0 == 0 ? D / 16 : 0;
+        for (int task = warp; task < wgroups + vg; task += DPC_THREADS / 32) {
+            if (task < wgroups) {
+                const int g = lane >> 2, t4 = lane & 3, ca = 16 * task + 4 * (g >> 1) + (g & 1);
+                float pre[2] = {1.0f, 1.0f};     // decay of the blocks before, for this lane's two columns
+                lower_product<2>(th, tl, lane,
+                    [&](int j0, int n, uint32_t (&bh)[2], uint32_t (&bl)[2]) {
+                        const float* k = sk + (j0 + t4) * P + ca + 2 * n;
+                        split2(k[0] * pre[n], k[4 * P] * pre[n], bh[0], bl[0]);
+                        split2(k[8 * P] * pre[n], k[12 * P] * pre[n], bh[1], bl[1]);
+                        pre[n] *= pb[(j0 >> 4) * D + ca + 2 * n];
+                    },
+                    [&](int row, float4 r) { store_w<D>(a, item, row, 16 * task + 4 * t4, r); });
+            } else {
+                values_product(a, th, tl, sV, item, v0, task - wgroups, lane);
+            }
+        }
     }
-    // ---- -W = -X (beta c K): a warp owns 16 channels and two row blocks (D = 128: {0, 3} or {1, 2}; D = 64: one).  Inner index (tokens):
-    // lane t4 holds tokens t4 + 4 e of a block; columns: a lane's four channels are neighbours.
+}
+
+// ---- a decay per head ------------------------------------------------------------------------------------------------------
+// k and q stay as projected (bfloat16, exact); norms and decays are factors of rows and columns.  Two CTAs share an SM.
+constexpr int DPH_THREADS = 256;
+template <int D>
+struct DphSmem {
+    static constexpr int P = D + 8;          // bfloat16 row pitch
+    static constexpr int K = 0, Q = K + 64 * P / 2, V = Q + 64 * P / 2, N = V + 64 * DV_PITCH / 2, B = N + 64 * DP_PITCH, X = B + 64 * DP_PITCH,
+                         T = X + 64 * DP_PITCH, BETA = T + 32 * 36, IQ = BETA + 64, IK = IQ + 64, G = IK + 64, C = G + 64, W = C + 64, E = W + 64, FLOATS = E + 64;
+};
+
+template <int D>
+__global__ void __launch_bounds__(DPH_THREADS, 2) delta_prep_head_kernel(const DeltaTcArgs a) {
+    using L = DphSmem<D>;
+    constexpr int P = L::P, VC = D / 32, NW = DPH_THREADS / 32;
+    extern __shared__ __align__(16) float sm[];
+    bf16_t *sk = reinterpret_cast<bf16_t*>(sm + L::K), *sq = reinterpret_cast<bf16_t*>(sm + L::Q), *sV = reinterpret_cast<bf16_t*>(sm + L::V);
+    float *sN = sm + L::N, *sB = sm + L::B, *sX = sm + L::X;
+    float *beta = sm + L::BETA, *iq = sm + L::IQ, *ik = sm + L::IK, *sg = sm + L::G, *sc = sm + L::C, *wk = sm + L::W, *we = sm + L::E;
+    pdl_launch_dependents();
+    pdl_wait();
+    const DeltaArgs& p = a.p;
+    const int item = blockIdx.x, h = item % p.H, kh = h / (p.H / p.G);
+    const int64_t t0 = (int64_t)(item / p.H) * DC;
+    const int nt = (int)min((int64_t)DC, p.n - t0);
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    // ---- raw rows, norms, decays, beta; tokens past the end become neutral
     {
+        const int e = VC * lane;
+        const bool in = e < p.d;
+        const bf16_t *q = static_cast<const bf16_t*>(p.q) + (int64_t)kh * p.d + e, *k = static_cast<const bf16_t*>(p.k) + (int64_t)kh * p.d + e;
+        const float qs = rsqrtf((float)p.d);
+        uint32_t qw[64 / NW][VC / 2], kw[64 / NW][VC / 2];
+#pragma unroll
+        for (int r = 0; r < 64 / NW; ++r) {
+            const int t = warp + NW * r;
+#pragma unroll
+            for (int i = 0; i < VC / 2; ++i) qw[r][i] = kw[r][i] = 0;
+            if (t < nt && in) {
+                if (VC == 4) {
+                    *reinterpret_cast<uint2*>(qw[r]) = *reinterpret_cast<const uint2*>(q + (t0 + t) * p.ldq);
+                    *reinterpret_cast<uint2*>(kw[r]) = *reinterpret_cast<const uint2*>(k + (t0 + t) * p.ldk);
+                } else {
+                    qw[r][0] = *reinterpret_cast<const uint32_t*>(q + (t0 + t) * p.ldq);
+                    kw[r][0] = *reinterpret_cast<const uint32_t*>(k + (t0 + t) * p.ldk);
+                }
+            }
+        }
+        if (tid < 64) {
+            float bt = 0.0f, g = 1.0f;
+            if (tid < nt) {
+                bt = sigmoid_f32(ldf(static_cast<const bf16_t*>(p.b) + (t0 + tid) * p.ldb + h));
+                g = decay_f32(p.nA[h], (ldf(static_cast<const bf16_t*>(p.a) + (t0 + tid) * p.lda + h) + p.dtb[h]) * 1.4426950408889634f);
+            }
+            beta[tid] = bt;
+            sg[tid] = g;
+        }
+        load_values<DPH_THREADS>(p, sV, h, t0, nt, 0, tid);
+#pragma unroll
+        for (int r = 0; r < 64 / NW; ++r) {
+            const int t = warp + NW * r;
+            float qq = 0.0f, kk = 0.0f;
+#pragma unroll
+            for (int i = 0; i < VC / 2; ++i) {
+                qq = fmaf(bf16_lo(qw[r][i]), bf16_lo(qw[r][i]), qq);
+                qq = fmaf(bf16_hi(qw[r][i]), bf16_hi(qw[r][i]), qq);
+                kk = fmaf(bf16_lo(kw[r][i]), bf16_lo(kw[r][i]), kk);
+                kk = fmaf(bf16_hi(kw[r][i]), bf16_hi(kw[r][i]), kk);
+                *reinterpret_cast<uint32_t*>(sq + t * P + e + 2 * i) = qw[r][i];
+                *reinterpret_cast<uint32_t*>(sk + t * P + e + 2 * i) = kw[r][i];
+            }
+            const float2 s = warp_sum2(qq, kk, lane);
+            if (lane == 0) {
+                iq[t] = qs * rsqrtf(s.x + 1e-6f);
+                ik[t] = rsqrtf(s.y + 1e-6f);
+            }
+        }
+    }
+    __syncthreads();
+    // ---- c_i / c_j for i >= j into N's place: a thread takes key j and 16 tokens
+    {
+        const int j = tid & 63, s0 = 16 * (tid >> 6);
+        float r = 1.0f;
+#pragma unroll 8
+        for (int t = 0; t < s0; ++t)
+            if (t > j) r *= sg[t];
+#pragma unroll
+        for (int t = s0; t < s0 + 16; ++t) {
+            if (t > j) r *= sg[t];
+            sN[t * DP_PITCH + j] = r;            // meant for t >= j
+            if (j == 0) sc[t] = r * sg[0];       // c itself
+        }
+    }
+    __syncthreads();
+    if (tid < 64) {
+        wk[tid] = sc[tid] * ik[tid];
+        we[tid] = sN[63 * DP_PITCH + tid] * ik[tid];      // before N is formed: the products to the chunk's end
+    }
+    __syncthreads();
+    for (int pair = warp; pair < 10; pair += NW) {
+        int I, b;
+        block_pair(pair, I, b);
         const int g = lane >> 2, t4 = lane & 3;
-        constexpr int CG = D / 16, ROWS = CG == 8 ? 2 : 1;
-        const int c0 = 16 * (warp % CG), rs = warp / CG;
-        float acc[ROWS][2][4] = {};
-        const int last = ROWS == 2 ? (rs == 0 ? 3 : 2) : rs;
-        float pre[2] = {1.0f, 1.0f};             // decay of the blocks before, for this lane's two columns
-        const int ca = c0 + 4 * (g >> 1) + (g & 1);
-        for (int jb = 0; jb <= last; ++jb) {
-            uint32_t bh[2][2], bl[2][2];
-            float v[2][4];
+        const bf16_t *kr = sk + (16 * I + g) * P + 2 * t4, *qr = sq + (16 * I + g) * P + 2 * t4, *kc = sk + (16 * b + g) * P + 2 * t4;
+        auto at = [](const bf16_t* x) { return *reinterpret_cast<const uint32_t*>(x); };
+        float n[2][4] = {}, m[2][4] = {};
+#pragma unroll 4
+        for (int s = 0; s < D; s += 16) {
+            const uint32_t ka[4] = {at(kr + s), at(kr + 8 * P + s), at(kr + s + 8), at(kr + 8 * P + s + 8)};
+            const uint32_t qa[4] = {at(qr + s), at(qr + 8 * P + s), at(qr + s + 8), at(qr + 8 * P + s + 8)};
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int j = 16 * jb + t4 + 4 * e;
-                const float w = beta[j] * (CH ? 1.0f : sf[j]);
-                v[0][e] = sk[j * P + ca] * (w * pre[0]);
-                v[1][e] = sk[j * P + ca + 2] * (w * pre[1]);
-            }
-#pragma unroll
-            for (int n = 0; n < 2; ++n) {
-                split2(v[n][0], v[n][1], bh[n][0], bl[n][0]);
-                split2(v[n][2], v[n][3], bh[n][1], bl[n][1]);
-                pre[n] *= CH ? pb[jb * D + ca + 2 * n] : pb[jb];
-            }
-#pragma unroll
-            for (int r = 0; r < ROWS; ++r) {
-                const int I = ROWS == 2 ? (r == 0 ? last : rs) : rs;
-                if (jb > I) continue;
-                const float* x = sX + (16 * I + g) * DP_PITCH + 16 * jb + t4;
-                uint32_t ah[4], al[4];
-                split2(x[0], x[4], ah[0], al[0]);
-                split2(x[8 * DP_PITCH], x[8 * DP_PITCH + 4], ah[1], al[1]);
-                split2(x[8], x[12], ah[2], al[2]);
-                split2(x[8 * DP_PITCH + 8], x[8 * DP_PITCH + 12], ah[3], al[3]);
-#pragma unroll
-                for (int n = 0; n < 2; ++n) mma_split(acc[r][n], ah, al, bh[n], bl[n]);
+            for (int j = 0; j < 2; ++j) {
+                const uint32_t b0 = at(kc + 8 * j * P + s), b1 = at(kc + 8 * j * P + s + 8);
+                mma_16816(n[j], ka, b0, b1);
+                mma_16816(m[j], qa, b0, b1);
             }
         }
 #pragma unroll
-        for (int r = 0; r < ROWS; ++r) {
-            const int I = ROWS == 2 ? (r == 0 ? last : rs) : rs;
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                uint32_t h0, l0, h1, l1;
-                split2(-acc[r][0][2 * e], -acc[r][0][2 * e + 1], h0, l0);
-                split2(-acc[r][1][2 * e], -acc[r][1][2 * e + 1], h1, l1);
-                const int64_t o = ((int64_t)item * DC + 16 * I + g + 8 * e) * D + c0 + 4 * t4;
-                *reinterpret_cast<uint2*>(a.wh + o) = make_uint2(h0, h1);
-                *reinterpret_cast<uint2*>(a.wl + o) = make_uint2(l0, l1);
+        for (int u = 0; u < 8; ++u) {
+            const int e = u & 3, i = 16 * I + g + 8 * (e >> 1), j = 16 * b + 8 * (u >> 2) + 2 * t4 + (e & 1);
+            const float r = sN[i * DP_PITCH + j] * ik[j];
+            if (i >= j) sB[i * DP_PITCH + j] = m[u >> 2][e] * r * iq[i];
+            if (i > j) sN[i * DP_PITCH + j] = n[u >> 2][e] * r * ik[i] * beta[i];
+        }
+    }
+    __syncthreads();
+    if (tid < 128) {
+        invert_unit_lower(sN, sX, sm + L::T, tid);
+    } else {
+        // ---- meanwhile: c Q, E, B and c at the chunk's end
+        for (int u = tid - 128; u < 64 * (D / 8); u += 128) {
+            const int t = u / (D / 8), c = 8 * (u % (D / 8));
+            const int64_t o = ((int64_t)item * DC + t) * D + c;
+            const float fq = iq[t] * sc[t], fe = we[t];
+            float x[8], y[8];
+            ld8(sq + t * P + c, x);
+            ld8(sk + t * P + c, y);
+            store_terms8(a.qh + o, a.ql + o, mul4(make_float4(x[0], x[1], x[2], x[3]), fq), mul4(make_float4(x[4], x[5], x[6], x[7]), fq));
+            store_terms8(a.eh + o, a.el + o, mul4(make_float4(y[0], y[1], y[2], y[3]), fe), mul4(make_float4(y[4], y[5], y[6], y[7]), fe));
+        }
+        store_lower(sB, a.bh, a.bl, item, tid - 128, 128);
+        for (int c = tid - 128; c < D; c += 128) a.gend[(int64_t)item * D + c] = sc[63];
+    }
+    __syncthreads();
+    uint32_t *th = reinterpret_cast<uint32_t*>(sN), *tl = th + 64 * DT_PITCH;      // over N and B
+    pack_t(sX, beta, th, tl, tid, DPH_THREADS);
+    __syncthreads();
+    for (int v0 = 0; v0 < p.dv; v0 += 128) {
+        if (v0 > 0) {
+            __syncthreads();
+            load_values<DPH_THREADS>(p, sV, h, t0, nt, v0, tid);
+            __syncthreads();
+        }
+        const int vg = min(8, (p.dv - v0 + 15) / 16), wgroups = v0 == 0 ? D / 16 : 0;
+        for (int task = warp; task < wgroups + vg; task += NW) {
+            if (task < wgroups) {
+                const int g = lane >> 2, t4 = lane & 3, ca = 16 * task + 4 * (g >> 1) + (g & 1);
+                lower_product<2>(th, tl, lane,
+                    [&](int j0, int n, uint32_t (&bh)[2], uint32_t (&bl)[2]) {
+                        const bf16_t* k = sk + (j0 + t4) * P + ca + 2 * n;
+                        const float* w = wk + j0 + t4;
+                        split2(ldf(k) * w[0], ldf(k + 4 * P) * w[4], bh[0], bl[0]);
+                        split2(ldf(k + 8 * P) * w[8], ldf(k + 12 * P) * w[12], bh[1], bl[1]);
+                    },
+                    [&](int row, float4 r) { store_w<D>(a, item, row, 16 * task + 4 * t4, r); });
+            } else {
+                values_product(a, th, tl, sV, item, v0, task - wgroups, lane);
             }
         }
     }
@@ -467,14 +719,15 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prep_kernel(const DeltaTc
 // ---- the recurrence over chunks -----------------------------------------------------------------------------------------
 // 576 threads: TMA warp, MMA warp (converged, one lane issues), four warpgroups that turn S into tensor-memory operands (a thread per
 // value row, 32 channels each); the first two do the same with U (32 tokens each), the others store O.  Operands stream through a ring of 16 KB slots, per chunk:
-//   V (two blocks of 64 values), {T high, T remainder}, per 64 channels {-W}, {c Q}, {E}, then {B}.
-// Tensor memory: S^T float32 0..127, its two terms 128..255 (per 32 channels: 16 columns high, 16 remainder), U^T 256..319, its
-// terms 320..383, O^T 384..511 (two buffers).
+//   per 64 channels {-W}, {c Q}, then E (D = 128: the high terms of all channels, the remainders; else both in one slot), {B}.
+// Tensor memory: S^T float32 0..127, its two terms 128..255 (per 32 channels: 16 columns high, 16 remainder), U^T 256..319 (starts
+// as T V, which the first two warpgroups put there a chunk ahead), its terms 320..383, O^T 384..511 (two buffers).
 constexpr int DT_THREADS = 576;
-constexpr int DT_SLOTS = 13, DT_SLOT = 2 * DC_BLK;
-constexpr int DT_G_OFF = DT_SLOTS * DT_SLOT;                  // float [4][128]
-constexpr int DT_BAR_OFF = DT_G_OFF + 4 * 512;                // full[], empty[], g[4], u, uw, s, sw, of[2], oe[2]
-constexpr int DT_NBAR = 2 * DT_SLOTS + 12;
+constexpr int DT_SLOTS = 11, DT_SLOT = 2 * DC_BLK;
+constexpr int DT_V_OFF = DT_SLOTS * DT_SLOT;                  // float [64][128]: T V of the next chunk
+constexpr int DT_G_OFF = DT_V_OFF + 64 * 128 * 4;             // float [4][128]
+constexpr int DT_BAR_OFF = DT_G_OFF + 4 * 512;                // full[], empty[], g[4], u, uw, s, sw, sc, of[2], oe[2], vf, ve
+constexpr int DT_NBAR = 2 * DT_SLOTS + 15;
 constexpr int DT_MISC_OFF = DT_BAR_OFF + 8 * DT_NBAR;
 constexpr int DT_SMEM = DT_MISC_OFF + 16 + 1024;
 constexpr uint32_t DT_SP = 128, DT_U = 256, DT_UP = 320, DT_O = 384;
@@ -487,8 +740,7 @@ __device__ __forceinline__ void split32(const uint32_t (&v)[32], uint32_t (&pk)[
 
 template <int DB>
 __global__ void __launch_bounds__(DT_THREADS, 1)
-    delta_state_kernel(const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmTh, const __grid_constant__ CUtensorMap tmTl,
-                       const __grid_constant__ CUtensorMap tmWh, const __grid_constant__ CUtensorMap tmWl, const __grid_constant__ CUtensorMap tmQh,
+    delta_state_kernel(const __grid_constant__ CUtensorMap tmWh, const __grid_constant__ CUtensorMap tmWl, const __grid_constant__ CUtensorMap tmQh,
                        const __grid_constant__ CUtensorMap tmQl, const __grid_constant__ CUtensorMap tmEh, const __grid_constant__ CUtensorMap tmEl,
                        const __grid_constant__ CUtensorMap tmBh, const __grid_constant__ CUtensorMap tmBl, const DeltaTcArgs a) {
     constexpr int D = 64 * DB;
@@ -496,15 +748,15 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
     uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);
     const uint32_t sbase = smem_u32(smem);
     const uint32_t b_f = sbase + DT_BAR_OFF, b_e = b_f + 8 * DT_SLOTS, b_g = b_e + 8 * DT_SLOTS, b_u = b_g + 32, b_uw = b_u + 8, b_s = b_uw + 8,
-                   b_sw = b_s + 8, b_of = b_sw + 8, b_oe = b_of + 16;
+                   b_sw = b_s + 8, b_sc = b_sw + 8, b_of = b_sc + 8, b_oe = b_of + 16, b_vf = b_oe + 16, b_ve = b_vf + 8;
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + DT_MISC_OFF);
     volatile int* abort_flag = reinterpret_cast<volatile int*>(smem + DT_MISC_OFF + 4);
     const int warp = __shfl_sync(0xffffffffu, (int)(threadIdx.x >> 5), 0), lane = threadIdx.x & 31;
     if (threadIdx.x == 0) {
-        for (const CUtensorMap* m : {&tmV, &tmTh, &tmTl, &tmWh, &tmWl, &tmQh, &tmQl, &tmEh, &tmEl, &tmBh, &tmBl}) prefetch_map(m);
+        for (const CUtensorMap* m : {&tmWh, &tmWl, &tmQh, &tmQl, &tmEh, &tmEl, &tmBh, &tmBl}) prefetch_map(m);
         for (int i = 0; i < DT_NBAR; ++i) {
             const uint32_t b = b_f + 8 * i;
-            mbar_init(b, b == b_uw || b == b_oe || b == b_oe + 8 ? 8 : b == b_sw ? 8 * DB : 1);
+            mbar_init(b, b == b_uw || b == b_ve || b == b_oe || b == b_oe + 8 ? 8 : b == b_sw || b == b_sc ? 8 * DB : 1);
         }
         *abort_flag = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
@@ -539,19 +791,20 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
             };
             for (int c = 0; c < nc && fail == 0; ++c) {
                 const int item = c * p.H + h, row = item * DC;
-                if (!slot()) break;
-                tma_load_3d(s, &tmV, 2 * v0, c * DC, h, bar);
-                tma_load_3d(s + DC_BLK, &tmV, 2 * v0 + 128, c * DC, h, bar);
                 // slot c & 3 of the decays is free: it was read before the products of chunk c - 4, whose operands left the ring
-                mbar_expect_tx(b_g + 8 * (c & 3), 4 * D);
-                bulk_load(sbase + DT_G_OFF + 512 * (c & 3), a.gend + (int64_t)item * D, 4 * D, b_g + 8 * (c & 3));
-                if (!slot()) break;
-                tma_load_2d(s, &tmTh, 0, row, bar);
-                tma_load_2d(s + DC_BLK, &tmTl, 0, row, bar);
+                bool first = true;
+                if (int w = mbar_wait(b_ve, (c & 1) ^ 1, abort_flag, a.wait_ns)) { fail = w == 1 ? 61 : -1; break; }
+                mbar_expect_tx(b_vf, 64 * 128 * 4);
+                bulk_load(sbase + DT_V_OFF, a.uv + ((int64_t)item * a.nvt + blockIdx.y) * DC * 128, 64 * 128 * 4, b_vf);
                 for (int b = 0; b < DB && fail == 0; ++b)
                     if (slot()) {
                         tma_load_2d(s, &tmWh, 128 * b, row, bar);
                         tma_load_2d(s + DC_BLK, &tmWl, 128 * b, row, bar);
+                        if (first) {
+                            mbar_expect_tx(b_g + 8 * (c & 3), 4 * D);
+                            bulk_load(sbase + DT_G_OFF + 512 * (c & 3), a.gend + (int64_t)item * D, 4 * D, b_g + 8 * (c & 3));
+                        }
+                        first = false;
                     }
                 for (int b = 0; b < DB && fail == 0; ++b)
                     if (slot()) {
@@ -560,8 +813,8 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
                     }
                 for (int b = 0; b < DB && fail == 0; ++b)
                     if (slot()) {
-                        tma_load_2d(s, &tmEh, 128 * b, row, bar);
-                        tma_load_2d(s + DC_BLK, &tmEl, 128 * b, row, bar);
+                        tma_load_2d(s, DB == 1 || b == 0 ? &tmEh : &tmEl, 0, row, bar);
+                        tma_load_2d(s + DC_BLK, DB == 2 && b == 0 ? &tmEh : &tmEl, DB == 2 ? 128 : 0, row, bar);
                     }
                 if (fail || !slot()) break;
                 tma_load_2d(s, &tmBh, 0, row, bar);
@@ -570,7 +823,7 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
         }
     } else if (warp == 1) {
         // the whole warp walks through the chunks; `on` is the lane that issues
-        constexpr uint32_t idesc = umma_idesc_bf16(128, 64), idesc_v = idesc | IDESC_A_MN, idesc_e = idesc | IDESC_B_MN;
+        constexpr uint32_t idesc = umma_idesc_bf16(128, 64), idesc_e = umma_idesc_bf16(128, D) | IDESC_B_MN;
         const uint32_t on = elect_lane();
         int st = 0;
         uint32_t ph = 0, s = 0;
@@ -600,23 +853,7 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
                 umma_bf16_ts_on(on, d, x + 16, bh + 2 * k, idesc, 1);
             }
         };
-        auto values = [&]() -> bool {      // U = T V
-            if (!next()) return false;
-            const uint64_t v = umma_desc_mn(s, DC_BLK);
-            const uint32_t vfree = b_e + 8 * st;
-            if (++st == DT_SLOTS) { st = 0; ph ^= 1; }
-            if (!next()) return false;
-            const uint64_t th = umma_desc(s), tl = umma_desc(s + DC_BLK);
-#pragma unroll
-            for (int k = 0; k < 4; ++k) {
-                umma_bf16_on(on, tmem + DT_U, v + 128 * k, th + 2 * k, idesc_v, k > 0);
-                umma_bf16_on(on, tmem + DT_U, v + 128 * k, tl + 2 * k, idesc_v, 1);
-            }
-            umma_commit_on(on, vfree);
-            done();
-            return true;
-        };
-        bool ok = values();
+        bool ok = true;
         for (int c = 0; c < nc && ok; ++c) {
             if (!wait(b_sw, c & 1, 63)) break;
 #pragma unroll
@@ -635,18 +872,25 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
                 split_product(o, tmem + DT_SP + 64 * b, b == 0);
                 done();
             }
-            if (!ok || !wait(b_uw, c & 1, 63)) break;
-#pragma unroll
-            for (int b = 0; b < DB; ++b) {
+            if (!ok || !wait(b_uw, c & 1, 63) || !wait(b_sc, c & 1, 63)) break;
+            {
                 if (!(ok = next())) break;
-                const uint64_t eh = umma_desc_mn(s, DC_BLK), el = umma_desc_mn(s + DC_BLK, DC_BLK);
+                const uint64_t eh = umma_desc_mn(s, DC_BLK);
+                uint64_t el = umma_desc_mn(s + DC_BLK, DC_BLK);
+                const uint32_t efree = b_e + 8 * st;
+                if (DB == 2) {
+                    if (++st == DT_SLOTS) { st = 0; ph ^= 1; }
+                    if (!(ok = next())) break;
+                    el = umma_desc_mn(s, DC_BLK);
+                }
 #pragma unroll
                 for (int k = 0; k < 4; ++k) {
                     const uint32_t u = tmem + DT_UP + (k >> 1) * 32 + (k & 1) * 8;
-                    umma_bf16_ts_on(on, tmem + 64 * b, u, eh + 128 * k, idesc_e, 1);
-                    umma_bf16_ts_on(on, tmem + 64 * b, u, el + 128 * k, idesc_e, 1);
-                    umma_bf16_ts_on(on, tmem + 64 * b, u + 16, eh + 128 * k, idesc_e, 1);
+                    umma_bf16_ts_on(on, tmem, u, eh + 128 * k, idesc_e, 1);
+                    umma_bf16_ts_on(on, tmem, u, el + 128 * k, idesc_e, 1);
+                    umma_bf16_ts_on(on, tmem, u + 16, eh + 128 * k, idesc_e, 1);
                 }
+                if (DB == 2) umma_commit_on(on, efree);
                 done();
             }
             if (!ok) break;
@@ -655,7 +899,6 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
             split_product(o, tmem + DT_UP, 0);
             done();
             umma_commit_on(on, b_of + 8 * (c & 1));
-            if (c + 1 < nc) ok = values();
         }
         if (!on) fail = fail > 0 ? -1 : fail;      // one lane reports
     } else {
@@ -670,10 +913,22 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
             tc_fence_after();
             return true;
         };
-        for (int c = 0; c <= nc; ++c) {
-            // S at the start of chunk c: its terms, and c_end S for the sum; after the last chunk the state is stored
+        // T V of a chunk into U's place, this warpgroup's 32 tokens
+        auto bring_values = [&](int c) -> bool {
+            if (!wait(b_vf, c & 1)) return false;
+            const float* src = reinterpret_cast<const float*>(smem + DT_V_OFF) + 32 * wg * 128 + 32 * q + lane;
+            uint32_t u[32];
+#pragma unroll
+            for (int i = 0; i < 32; ++i) u[i] = in ? __float_as_uint(src[128 * i]) : 0u;
+            __syncwarp();
+            if (lane == 0) mbar_arrive(b_ve);
+            tmem_st32(tmem + DT_U + 32 * wg + lane_base, u);
+            return true;
+        };
+        const bool go = wg >= 2 || bring_values(0);
+        for (int c = 0; c <= nc && go; ++c) {
+            // S at the start of chunk c: its terms first, then c_end S for the sum; after the last chunk the state is stored
             if (owner) {
-                if (c < nc && !wait(b_g + 8 * (c & 3), (c >> 2) & 1)) break;
                 if (c > 0 && !wait(b_s, (c - 1) & 1)) break;
                 uint32_t s[32];
                 if (c > 0) {
@@ -691,20 +946,25 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
                     uint32_t pk[32];
                     split32(s, pk);
                     tmem_st32(tmem + DT_SP + ch + lane_base, pk);
-                    const float4* g = reinterpret_cast<const float4*>(smem + DT_G_OFF + 512 * (c & 3)) + ch / 4;
+                    tmem_st_wait();
+                    tc_fence_before();
+                    __syncwarp();
+                    if (lane == 0) mbar_arrive(b_sw);
+                    if (!wait(b_g + 8 * (c & 3), (c >> 2) & 1)) break;
+                    const ulonglong2* g = reinterpret_cast<const ulonglong2*>(smem + DT_G_OFF + 512 * (c & 3)) + ch / 4;
 #pragma unroll
                     for (int i = 0; i < 8; ++i) {
-                        const float4 f = g[i];
-                        s[4 * i] = __float_as_uint(__uint_as_float(s[4 * i]) * f.x);
-                        s[4 * i + 1] = __float_as_uint(__uint_as_float(s[4 * i + 1]) * f.y);
-                        s[4 * i + 2] = __float_as_uint(__uint_as_float(s[4 * i + 2]) * f.z);
-                        s[4 * i + 3] = __float_as_uint(__uint_as_float(s[4 * i + 3]) * f.w);
+                        const ulonglong2 f = g[i];
+                        const float2 x = unpack2(mul2(pack2(__uint_as_float(s[4 * i]), __uint_as_float(s[4 * i + 1])), f.x));
+                        const float2 y = unpack2(mul2(pack2(__uint_as_float(s[4 * i + 2]), __uint_as_float(s[4 * i + 3])), f.y));
+                        s[4 * i] = __float_as_uint(x.x); s[4 * i + 1] = __float_as_uint(x.y);
+                        s[4 * i + 2] = __float_as_uint(y.x); s[4 * i + 3] = __float_as_uint(y.y);
                     }
                     tmem_st32(tmem + ch + lane_base, s);
                     tmem_st_wait();
                     tc_fence_before();
                     __syncwarp();
-                    if (lane == 0) mbar_arrive(b_sw);
+                    if (lane == 0) mbar_arrive(b_sc);
                 }
             }
             if (wg < 2) {
@@ -720,6 +980,7 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
                 tc_fence_before();
                 __syncwarp();
                 if (lane == 0) mbar_arrive(b_uw);
+                if (c + 1 < nc && !bring_values(c + 1)) break;
             } else if (c > 0) {
                 // outputs of the previous chunk, 32 tokens per warpgroup
                 const int b = (c - 1) & 1;
@@ -766,27 +1027,32 @@ bool delta_tc_supported(int64_t n, int H, int d, int dv, int64_t ldv) {
 
 static int64_t align256(int64_t b) { return (b + 255) / 256 * 256; }
 static int width(int d) { return d <= 64 ? 64 : 128; }
-int64_t delta_tc_scratch(int64_t n, int H, int d) {
+int64_t delta_tc_scratch(int64_t n, int H, int d, int dv) {
     const int64_t items = (n + DC - 1) / DC * H;
-    return 6 * align256(items * DC * width(d) * 2) + 4 * align256(items * DC_BLK) + align256(items * width(d) * 4);
+    return 6 * align256(items * DC * width(d) * 2) + 2 * align256(items * DC_BLK) + align256(items * ((dv + 127) / 128) * DC * 128 * 4) +
+           align256(items * width(d) * 4);
 }
 
-template <int D, bool CH>
-static int run_prep_tc(const DeltaTcArgs& a, cudaStream_t st) {
-    constexpr int smem = DpSmem<D, CH>::FLOATS * 4;
-    static bool configured[64] = {};
+static int run_prep_tc(void (*kernel)(DeltaTcArgs), int smem, int threads, bool (&configured)[64], const DeltaTcArgs& a, cudaStream_t st) {
     const int dev = current_device();
     SCMX_REQUIRE(dev >= 0, SCMX_ECUDA, "no current CUDA device (ordinal 0..63)");
     if (!configured[dev]) {
-        SCMX_CUDA_OK(cudaFuncSetAttribute(delta_prep_kernel<D, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+        SCMX_CUDA_OK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
         configured[dev] = true;
     }
-    SCMX_PDL_OK("delta_prep_kernel", launch_pdl(delta_prep_kernel<D, CH>, dim3((unsigned)a.nc * a.p.H), dim3(DP_THREADS), (size_t)smem, st, a));
+    SCMX_PDL_OK("delta_prep_kernel", launch_pdl(kernel, dim3((unsigned)a.nc * a.p.H), dim3(threads), (size_t)smem, st, a));
     return SCMX_OK;
 }
 
+template <int D>
+static int run_prep(bool channel, const DeltaTcArgs& a, cudaStream_t st) {
+    static bool done[2][64] = {};
+    return channel ? run_prep_tc(delta_prep_channel_kernel<D>, DpcSmem<D>::FLOATS * 4, DPC_THREADS, done[1], a, st)
+                   : run_prep_tc(delta_prep_head_kernel<D>, DphSmem<D>::FLOATS * 4, DPH_THREADS, done[0], a, st);
+}
+
 template <int DB>
-static int run_state(const CUtensorMap (&m)[11], const DeltaTcArgs& a, cudaStream_t st) {
+static int run_state(const CUtensorMap (&m)[8], const DeltaTcArgs& a, cudaStream_t st) {
     static bool configured[64] = {};
     const int dev = current_device();
     SCMX_REQUIRE(dev >= 0, SCMX_ECUDA, "no current CUDA device (ordinal 0..63)");
@@ -795,30 +1061,29 @@ static int run_state(const CUtensorMap (&m)[11], const DeltaTcArgs& a, cudaStrea
         configured[dev] = true;
     }
     SCMX_PDL_OK("delta_state_kernel", launch_pdl(delta_state_kernel<DB>, dim3(a.p.H, (a.p.dv + 127) / 128), dim3(DT_THREADS), (size_t)DT_SMEM, st, m[0], m[1],
-                                                 m[2], m[3], m[4], m[5], m[6], m[7], m[8], m[9], m[10], a));
+                                                 m[2], m[3], m[4], m[5], m[6], m[7], a));
     return SCMX_OK;
 }
 
 int delta_tc(const DeltaArgs& p, bool channel, void* scratch, int32_t* status, cudaStream_t st) {
-    SCMX_REQUIRE(p.ldq % 2 == 0 && p.ldk % 2 == 0 && (((uintptr_t)p.q | (uintptr_t)p.k) & 3) == 0 &&
-                 (!channel || (p.lda % 2 == 0 && ((uintptr_t)p.a & 7) == 0)), SCMX_EINVAL, "delta: unaligned rows");
+    SCMX_REQUIRE(p.ldq % 4 == 0 && p.ldk % 4 == 0 && (((uintptr_t)p.q | (uintptr_t)p.k) & 7) == 0 &&
+                 (!channel || (p.lda % 4 == 0 && ((uintptr_t)p.a & 15) == 0)), SCMX_EINVAL, "delta: unaligned rows");
     DeltaTcArgs a;
-    a.p = p; a.status = status; a.wait_ns = g_wait_limit_ns; a.nc = (int)((p.n + DC - 1) / DC);
+    a.p = p; a.status = status; a.wait_ns = g_wait_limit_ns; a.nc = (int)((p.n + DC - 1) / DC); a.nvt = (p.dv + 127) / 128;
     const int64_t items = (int64_t)a.nc * p.H;
     const int D = width(p.d);
     uint8_t* s = static_cast<uint8_t*>(scratch);
     bf16_t** wide[6] = {&a.wh, &a.wl, &a.qh, &a.ql, &a.eh, &a.el};
     for (auto x : wide) { *x = reinterpret_cast<bf16_t*>(s); s += align256(items * DC * D * 2); }
-    bf16_t** square[4] = {&a.th, &a.tl, &a.bh, &a.bl};
+    bf16_t** square[2] = {&a.bh, &a.bl};
     for (auto x : square) { *x = reinterpret_cast<bf16_t*>(s); s += align256(items * DC_BLK); }
+    a.uv = reinterpret_cast<float*>(s); s += align256(items * a.nvt * DC * 128 * 4);
     a.gend = reinterpret_cast<float*>(s);
-    CUtensorMap m[11];
-    int rc = make_map_planes(&m[0], p.v, p.H, p.n, 2 * p.dv, 2 * p.ldv, 2 * p.dv, DC);
-    const bf16_t* src[10] = {a.th, a.tl, a.wh, a.wl, a.qh, a.ql, a.eh, a.el, a.bh, a.bl};
-    for (int i = 0; i < 10 && !rc; ++i) rc = make_map_u8(&m[i + 1], src[i], items * DC, i >= 2 && i < 8 ? 2 * D : 128, 128, DC, 128, 0);
-    if (rc) return rc;
-    if (D == 64) rc = channel ? run_prep_tc<64, true>(a, st) : run_prep_tc<64, false>(a, st);
-    else rc = channel ? run_prep_tc<128, true>(a, st) : run_prep_tc<128, false>(a, st);
+    CUtensorMap m[8];
+    int rc = 0;
+    const bf16_t* src[8] = {a.wh, a.wl, a.qh, a.ql, a.eh, a.el, a.bh, a.bl};
+    for (int i = 0; i < 8 && !rc; ++i) rc = make_map_u8(&m[i], src[i], items * DC, i < 6 ? 2 * D : 128, 128, DC, 128, 0);
+    if (!rc) rc = D == 64 ? run_prep<64>(channel, a, st) : run_prep<128>(channel, a, st);
     if (rc) return rc;
     return D == 64 ? run_state<1>(m, a, st) : run_state<2>(m, a, st);
 }

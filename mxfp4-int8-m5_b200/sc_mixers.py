@@ -211,7 +211,9 @@ def delta(q, k, v, b, a, channel, nA, dt_bias, state, form=0):
     assert not channel or a.dtype == torch.float32
     nbytes = 0
     if q.dtype == torch.bfloat16 and form != 1 and (form == 2 or T >= DELTA_TC_MIN):
-        nbytes = 0 if v.data_ptr() % 16 else _lib.mixers().scmx_delta_scratch(T, H, d, dv, _ld(v))
+        rows = (q, k, v, a) if channel else (q, k, v)
+        aligned = not any(x.data_ptr() % 16 or _ld(x) % 8 for x in rows)
+        nbytes = _lib.mixers().scmx_delta_scratch(T, H, d, dv, _ld(v)) if aligned else 0
     assert nbytes or form != 2, "no tensor-core form for these sizes"
     scratch = torch.empty(nbytes, dtype=torch.uint8, device=q.device) if nbytes else None
     _lib.mcall("scmx_delta", _lib.ptr(q), _ld(q), _lib.ptr(k), _ld(k), _lib.ptr(v), _ld(v), _lib.ptr(b), _ld(b), _lib.ptr(a), _ld(a), _dt(q), int(channel),
