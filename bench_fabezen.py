@@ -171,7 +171,7 @@ def run(pkg, torch, pk, sampler, sizes=None):
             s = SIZES[name]
             models = {"fabezen": B.measure_hybrid(pkg, torch, pk, fabezen_config(s), rank=s["rank"]), "hybrid": B.measure_hybrid(pkg, torch, pk, like_config(s))}
             out["sizes"][name] = {"config": s, "models": models, "kernels": {"fabezen": kernels(pkg, torch, pk, s),
-                                                                            "hybrid": B.hybrid_kernels(pkg, torch, pk, B.SIZES[name])}}
+                                                                            "hybrid": B.hybrid_kernels(pkg, torch, pk, {**B.SIZES[name], "rvdim": s["vdim"]})}}
     out["clocks"] = clk.summary()
     pkg._lib.check_mixer_status()
     print(json.dumps(out))
