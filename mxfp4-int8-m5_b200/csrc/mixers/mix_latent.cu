@@ -37,6 +37,67 @@ struct LatentAppendArgs {
     int Q, R, r;
     float eps;
 };
+// Vectors of eight elements, up to AV_KEEP per thread in registers (sizes multiples of 8, aligned rows).
+constexpr int AV_THREADS = 128, AV_KEEP = 4;
+template <typename TI, typename TC, typename TQ>
+__global__ void __launch_bounds__(AV_THREADS) latent_append_vec_kernel(const LatentAppendArgs<TI, TC, TQ> a) {
+    __shared__ float red[2][AV_THREADS / 32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int64_t t = blockIdx.x, row = (a.pos_dev != nullptr ? (int64_t)a.pos_dev[0] : a.pos) + t;
+    const TI* y = a.y + t * a.ldy;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nq = a.Q / 8, nv = (a.Q + a.R) / 8;
+    float x[AV_KEEP][8], s0 = 0.0f, s1 = 0.0f;
+#pragma unroll
+    for (int k = 0; k < AV_KEEP; ++k) {
+        const int v = tid + AV_THREADS * k;
+        if (v < nv) {
+            ld8(y + 8 * v, x[k]);
+        } else {
+#pragma unroll
+            for (int i = 0; i < 8; ++i) x[k][i] = 0.0f;
+        }
+    }
+#pragma unroll
+    for (int k = 0; k < AV_KEEP; ++k) {
+        float s = 0.0f;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) s = fmaf(x[k][i], x[k][i], s);
+        if (tid + AV_THREADS * k < nq) s0 += s;
+        else s1 += s;
+    }
+    s0 = warp_sumf(s0);
+    s1 = warp_sumf(s1);
+    if (lane == 0) {
+        red[0][warp] = s0;
+        red[1][warp] = s1;
+    }
+    __syncthreads();
+    const float iq = rms_inv_f32(red[0][0] + red[0][1] + red[0][2] + red[0][3], a.Q, a.eps);
+    const float ic = rms_inv_f32(red[1][0] + red[1][1] + red[1][2] + red[1][3], a.R, a.eps);
+    const bool fits = row < a.cap;               // a device-side step beyond the cache drops the row
+#pragma unroll
+    for (int k = 0; k < AV_KEEP; ++k) {
+        const int v = tid + AV_THREADS * k;
+        if (v >= nv) continue;
+        float w[8];
+        if (v < nq) {
+            ld8(a.qw + 8 * v, w);
+            TQ* o = a.cq + t * a.ldcq + 8 * v;
+            st4(o, x[k][0] * iq * w[0], x[k][1] * iq * w[1], x[k][2] * iq * w[2], x[k][3] * iq * w[3]);
+            st4(o + 4, x[k][4] * iq * w[4], x[k][5] * iq * w[5], x[k][6] * iq * w[6], x[k][7] * iq * w[7]);
+        } else if (fits) {
+            ld8(a.cw + 8 * (v - nq), w);
+            TC* o = a.cache + row * a.ldc + 8 * (v - nq);
+            st4(o, x[k][0] * ic * w[0], x[k][1] * ic * w[1], x[k][2] * ic * w[2], x[k][3] * ic * w[3]);
+            st4(o + 4, x[k][4] * ic * w[4], x[k][5] * ic * w[5], x[k][6] * ic * w[6], x[k][7] * ic * w[7]);
+        }
+    }
+    if (!fits) return;
+    const float* cs = a.cs + (row < a.cs_rows ? row : a.cs_rows - 1) * a.r;
+    for (int i = tid; i < a.r; i += AV_THREADS) stf(a.cache + row * a.ldc + a.R + i, rotated_pair(y + a.Q + a.R, i, a.r, cs));
+}
+
 template <typename TI, typename TC, typename TQ>
 __global__ void __launch_bounds__(256) latent_append_kernel(const LatentAppendArgs<TI, TC, TQ> a) {
     __shared__ float red[2][9];
@@ -112,24 +173,36 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const AbsorbArgs<TQ,
     const int64_t t = blockIdx.z;
     const int c0 = blockIdx.x * LB_COLS, c = c0 + 2 * lane;      // the pitch covers pairs (rows are padded to 8 columns)
     const TW* w = a.wuk + (int64_t)h * a.d * a.ldw + c;
+    // the first rows are requested before the previous kernel ends: weights never change
+    constexpr int PRE = 16;
+    float2 pre[PRE];
+    auto load = [&](int e) -> float2 {
+        if (sizeof(TW) == 2) {
+            const uint32_t u = __ldg(reinterpret_cast<const uint32_t*>(w + (int64_t)e * a.ldw));
+            return make_float2(bf16_lo(u), bf16_hi(u));
+        }
+        return __ldg(reinterpret_cast<const float2*>(w + (int64_t)e * a.ldw));
+    };
+#pragma unroll
+    for (int i = 0; i < PRE; ++i) pre[i] = c < a.R && warp + 8 * i < a.d ? load(warp + 8 * i) : make_float2(0.0f, 0.0f);
     pdl_wait();
     const TQ* q = a.q + t * a.ldq + (int64_t)h * (a.d + a.r);
     float s0 = 0.0f, s1 = 0.0f;
-    if (c < a.R) {
-#pragma unroll 8
-        for (int e = warp; e < a.d; e += 8) {
-            const float x = ldf(q + e);
-            if (sizeof(TW) == 2) {
-                const uint32_t u = __ldg(reinterpret_cast<const uint32_t*>(w + (int64_t)e * a.ldw));
-                s0 = fmaf(bf16_lo(u), x, s0);
-                s1 = fmaf(bf16_hi(u), x, s1);
-            } else {
-                const float2 u = __ldg(reinterpret_cast<const float2*>(w + (int64_t)e * a.ldw));
-                s0 = fmaf(u.x, x, s0);
-                s1 = fmaf(u.y, x, s1);
-            }
+#pragma unroll
+    for (int i = 0; i < PRE; ++i)
+        if (warp + 8 * i < a.d) {
+            const float x = ldf(q + warp + 8 * i);
+            s0 = fmaf(pre[i].x, x, s0);
+            s1 = fmaf(pre[i].y, x, s1);
         }
-    }
+    if (c < a.R)
+#pragma unroll 8
+        for (int e = warp + 8 * PRE; e < a.d; e += 8) {
+            const float x = ldf(q + e);
+            const float2 u = load(e);
+            s0 = fmaf(u.x, x, s0);
+            s1 = fmaf(u.y, x, s1);
+        }
     part[warp][2 * lane] = s0;
     part[warp][2 * lane + 1] = s1;
     __syncthreads();
@@ -149,6 +222,7 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const AbsorbArgs<TQ,
 
 // ---- attention of absorbed queries --------------------------------------------------------------------------------------
 constexpr int LR_P = 32;         // positions per tile
+constexpr int LR_SPLITS = 64;    // ranges of positions at most
 
 // Positions of a row's window cut into splits of whole tiles; how many splits have any.
 struct LatentSpan {
@@ -175,9 +249,36 @@ struct LatentRowsArgs {
     float scale;
 };
 
+// Eight stored values as loaded, converted on use.
+template <typename T> struct Vec8Raw;
+template <> struct Vec8Raw<bf16_t> {
+    uint4 w;
+    __device__ __forceinline__ void load(const bf16_t* p) { w = *reinterpret_cast<const uint4*>(p); }
+    __device__ __forceinline__ void store(bf16_t* p) const { *reinterpret_cast<uint4*>(p) = w; }
+    __device__ __forceinline__ void get(float (&x)[8]) const {
+        x[0] = bf16_lo(w.x); x[1] = bf16_hi(w.x); x[2] = bf16_lo(w.y); x[3] = bf16_hi(w.y);
+        x[4] = bf16_lo(w.z); x[5] = bf16_hi(w.z); x[6] = bf16_lo(w.w); x[7] = bf16_hi(w.w);
+    }
+};
+template <> struct Vec8Raw<float> {
+    float4 a, b;
+    __device__ __forceinline__ void load(const float* p) { a = reinterpret_cast<const float4*>(p)[0]; b = reinterpret_cast<const float4*>(p)[1]; }
+    __device__ __forceinline__ void store(float* p) const { reinterpret_cast<float4*>(p)[0] = a; reinterpret_cast<float4*>(p)[1] = b; }
+    __device__ __forceinline__ void get(float (&x)[8]) const {
+        x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w; x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w;
+    }
+};
+// Two neighbouring values.
+__device__ __forceinline__ float2 ld2(const bf16_t* p) {
+    const uint32_t u = *reinterpret_cast<const uint32_t*>(p);
+    return make_float2(bf16_lo(u), bf16_hi(u));
+}
+__device__ __forceinline__ float2 ld2(const float* p) { return *reinterpret_cast<const float2*>(p); }
+
 // Grid (splits, groups of HG heads, rows).  Scores: a warp takes four positions of a tile, lanes stride over vectors of eight
-// elements, partial sums are exchanged so that every lane ends with whole ones.  Values: a thread owns NC pairs of latent columns
-// of all HG heads over every (256 / ct)-th position.
+// elements, partial sums are exchanged so that every lane ends with whole ones; the next tile is requested as soon as the scores of
+// one are formed (its first KEEP vectors per lane and position).  Values: a thread owns NC pairs of latent columns of all HG heads
+// over every (256 / ct)-th position.
 template <typename T, int HG, int NC>
 __global__ void __launch_bounds__(256) latent_rows_kernel(const LatentRowsArgs<T> a) {
     extern __shared__ __align__(16) uint8_t smb[];
@@ -213,28 +314,32 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(const LatentRowsArgs<T
     for (int h = 0; h < HG; ++h)
 #pragma unroll
         for (int c = 0; c < NC; ++c) acc[h][c][0] = acc[h][c][1] = 0.0f;
+    constexpr int KEEP = sizeof(T) == 2 ? 3 : 1;
+    Vec8Raw<T> raw[KEEP][4];
+    auto row_of = [&](int64_t tb, int p) -> const T* {
+        const int64_t t = tb + 4 * warp + p;
+        return a.cache + (t < t1 ? t : t0) * a.ldc;
+    };
+    auto request = [&](int64_t tb) {
+#pragma unroll
+        for (int k = 0; k < KEEP; ++k)
+            if (lane + 32 * k < nv)
+#pragma unroll
+                for (int p = 0; p < 4; ++p) raw[k][p].load(row_of(tb, p) + 8 * (lane + 32 * k));
+    };
+    request(t0);
     for (int64_t tb = t0; tb < t1; tb += LR_P) {
         __syncthreads();                         // queries staged; the previous tile is consumed
         float s[4 * HG];
 #pragma unroll
         for (int i = 0; i < 4 * HG; ++i) s[i] = 0.0f;
-        const T* cr[4];
-#pragma unroll
-        for (int p = 0; p < 4; ++p) {
-            const int64_t t = tb + 4 * warp + p;
-            cr[p] = a.cache + (t < t1 ? t : t0) * a.ldc;
-        }
-        for (int v = lane; v < nv; v += 32) {
+        auto use = [&](int v, const Vec8Raw<T> (&w)[4]) {
             float x[4][8];
 #pragma unroll
-            for (int p = 0; p < 4; ++p) ld8(cr[p] + 8 * v, x[p]);
-            if (8 * v < Rp)
-#pragma unroll
-                for (int p = 0; p < 4; ++p) {
-                    T* o = sc + (4 * warp + p) * Rp + 8 * v;
-                    st4(o, x[p][0], x[p][1], x[p][2], x[p][3]);
-                    st4(o + 4, x[p][4], x[p][5], x[p][6], x[p][7]);
-                }
+            for (int p = 0; p < 4; ++p) {
+                w[p].get(x[p]);
+                if (8 * v < Rp) w[p].store(sc + (4 * warp + p) * Rp + 8 * v);
+            }
 #pragma unroll
             for (int h = 0; h < HG; ++h) {
                 const float4 lo = reinterpret_cast<const float4*>(sq)[(2 * h) * nv + v], hi = reinterpret_cast<const float4*>(sq)[(2 * h + 1) * nv + v];
@@ -245,7 +350,17 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(const LatentRowsArgs<T
                     r = fmaf(x[p][4], hi.x, r); r = fmaf(x[p][5], hi.y, r); r = fmaf(x[p][6], hi.z, r); r = fmaf(x[p][7], hi.w, r);
                 }
             }
+        };
+#pragma unroll
+        for (int k = 0; k < KEEP; ++k)
+            if (lane + 32 * k < nv) use(lane + 32 * k, raw[k]);
+        for (int v = lane + 32 * KEEP; v < nv; v += 32) {
+            Vec8Raw<T> w[4];
+#pragma unroll
+            for (int p = 0; p < 4; ++p) w[p].load(row_of(tb, p) + 8 * v);
+            use(v, w);
         }
+        if (tb + LR_P < t1) request(tb + LR_P);
         // lane bits from the highest choose which half of the sums a lane keeps; what is left is added over the remaining bits
         int idx = 0;
 #pragma unroll
@@ -294,11 +409,11 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(const LatentRowsArgs<T
             for (int c = 0; c < NC; ++c) {
                 const int e = 2 * (col + a.ct * c);
                 if (e >= Rp) continue;
-                const float v0 = ldf(sc + p * Rp + e), v1 = ldf(sc + p * Rp + e + 1);
+                const float2 v = ld2(sc + p * Rp + e);
 #pragma unroll
                 for (int h = 0; h < HG; ++h) {
-                    acc[h][c][0] = fmaf(w[h], v0, acc[h][c][0]);
-                    acc[h][c][1] = fmaf(w[h], v1, acc[h][c][1]);
+                    acc[h][c][0] = fmaf(w[h], v.x, acc[h][c][0]);
+                    acc[h][c][1] = fmaf(w[h], v.y, acc[h][c][1]);
                 }
             }
         }
@@ -352,38 +467,62 @@ constexpr int LV_ROWS = 32;      // values per CTA, four per warp
 template <typename TW, typename TO>
 __global__ void __launch_bounds__(256) latent_value_kernel(const LatentValueArgs<TW, TO> a) {
     extern __shared__ __align__(16) float ctx[];         // [ldw], zero padded
-    __shared__ float cf[32];
+    __shared__ float cf[LR_SPLITS];
     pdl_launch_dependents();
-    pdl_wait();
     const int h = blockIdx.x, e0 = blockIdx.y * LV_ROWS, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    // the first vectors of this warp's rows are requested before the previous kernel ends: weights never change
+    constexpr int ROWS = LV_ROWS / 8, PRE = sizeof(TW) == 2 ? 2 : 1;
+    const TW* w = a.wuv + ((int64_t)h * a.dv + e0 + warp) * a.ldw + 8 * lane;
+    Vec8Raw<TW> pre[ROWS][PRE];
+#pragma unroll
+    for (int j = 0; j < ROWS; ++j)
+#pragma unroll
+        for (int k = 0; k < PRE; ++k)
+            if (e0 + warp + 8 * j < a.dv && 8 * lane + 256 * k < a.ldw) pre[j][k].load(w + 8 * j * a.ldw + 256 * k);
+    pdl_wait();
     const int64_t row = blockIdx.z, pos = (a.pos_dev != nullptr ? (int64_t)a.pos_dev[0] : a.pos) + row;
     const int active = latent_span(pos, a.cap, a.window, a.nsplit).active;
     const float* part = a.part + (row * a.H + h) * a.nsplit * (a.R + 2);
     if (warp == 0) {
-        const float m = lane < active ? part[lane * (a.R + 2) + a.R] : -INFINITY, l = lane < active ? part[lane * (a.R + 2) + a.R + 1] : 0.0f;
-        const float mm = warp_max(m), c = lane < active ? ex2_approx(m - mm) : 0.0f;
-        cf[lane] = c / warp_sumf(c * l);
+        float m[2], l[2];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const int sp = lane + 32 * i;
+            m[i] = sp < active ? part[sp * (a.R + 2) + a.R] : -INFINITY;
+            l[i] = sp < active ? part[sp * (a.R + 2) + a.R + 1] : 0.0f;
+        }
+        const float mm = warp_max(fmaxf(m[0], m[1])), c0 = ex2_approx(m[0] - mm), c1 = ex2_approx(m[1] - mm);
+        const float inv = 1.0f / warp_sumf(c0 * l[0] + c1 * l[1]);
+        cf[lane] = c0 * inv;
+        cf[lane + 32] = c1 * inv;
     }
     __syncthreads();
     for (int e = tid; e < a.ldw; e += 256) {
         float s = 0.0f;
         if (e < a.R)
-#pragma unroll 8
+#pragma unroll 16
             for (int i = 0; i < active; ++i) s = fmaf(cf[i], part[i * (a.R + 2) + e], s);
         ctx[e] = s;
     }
     __syncthreads();
 #pragma unroll
-    for (int j = 0; j < LV_ROWS / 8; ++j) {
+    for (int j = 0; j < ROWS; ++j) {
         const int e = e0 + warp + 8 * j;
         if (e >= a.dv) continue;
-        const TW* w = a.wuv + ((int64_t)h * a.dv + e) * a.ldw;
         float s = 0.0f;
-        for (int i = 8 * lane; i < a.ldw; i += 256) {
+        auto add = [&](const Vec8Raw<TW>& u, int i) {
             float v[8];
-            ld8(w + i, v);
+            u.get(v);
 #pragma unroll
             for (int k = 0; k < 8; ++k) s = fmaf(v[k], ctx[i + k], s);
+        };
+#pragma unroll
+        for (int k = 0; k < PRE; ++k)
+            if (8 * lane + 256 * k < a.ldw) add(pre[j][k], 8 * lane + 256 * k);
+        for (int i = 8 * lane + 256 * PRE; i < a.ldw; i += 256) {
+            Vec8Raw<TW> u;
+            u.load(w + 8 * j * a.ldw + (i - 8 * lane));
+            add(u, i);
         }
         s = warp_sumf(s);
         if (lane == 0) stf(a.out + row * a.ldo + (int64_t)h * a.dv + e, s);
@@ -411,6 +550,12 @@ static int run_append(const void* y, int64_t ldy, int64_t n, int Q, int R, int r
     LatentAppendArgs<TI, TC, TQ> a;
     a.y = (const TI*)y; a.qw = qw; a.cw = cw; a.cs = cs; a.cq = (TQ*)cq; a.cache = (TC*)cache; a.pos_dev = pos_dev; a.ldy = ldy; a.ldcq = ldcq; a.ldc = ldc;
     a.pos = pos; a.cap = cap; a.cs_rows = cs_rows; a.Q = Q; a.R = R; a.r = r; a.eps = eps;
+    auto al = [](const void* x) { return ((uintptr_t)x & 15) == 0; };
+    if (Q % 8 == 0 && R % 8 == 0 && (Q + R) / 8 <= AV_THREADS * AV_KEEP && ldy % 8 == 0 && ldcq % 8 == 0 && ldc % 8 == 0 && al(y) && al(qw) && al(cw) &&
+        al(cq) && al(cache)) {
+        SCMX_PDL_OK("latent_append_kernel", launch_pdl(latent_append_vec_kernel<TI, TC, TQ>, dim3((unsigned)n), dim3(AV_THREADS), 0, st, a));
+        return SCMX_OK;
+    }
     SCMX_PDL_OK("latent_append_kernel", launch_pdl(latent_append_kernel<TI, TC, TQ>, dim3((unsigned)n), dim3(256), 0, st, a));
     return SCMX_OK;
 }
@@ -486,7 +631,7 @@ extern "C" int scmx_latent_rows(const float* q, const void* cache, int64_t ldc, 
     LATENT_ROWS_OK("latent_rows", n);
     SCMX_REQUIRE(q && cache && part && H > 0 && R > 0 && r >= 0 && ldc % 8 == 0 && ldc >= up8(R) + up8(r) && ((uintptr_t)cache & 15) == 0, SCMX_EINVAL,
                  "latent_rows: heads %d, latent %d, rotated %d, pitch %lld", H, R, r, (long long)ldc);
-    SCMX_REQUIRE(nsplit >= 1 && nsplit <= 32 && window >= 0 && cap >= 1, SCMX_EINVAL, "latent_rows: %d splits, window %lld", nsplit, (long long)window);
+    SCMX_REQUIRE(nsplit >= 1 && nsplit <= LR_SPLITS && window >= 0 && cap >= 1, SCMX_EINVAL, "latent_rows: %d splits, window %lld", nsplit, (long long)window);
     SCMX_REQUIRE(pos_dev != nullptr || (pos >= 0 && pos + n <= cap), SCMX_EINVAL, "latent_rows: %lld rows at %lld in a cache of %lld", (long long)n,
                  (long long)pos, (long long)cap);
     SCMX_REQUIRE(R <= 1024, SCMX_ELIMIT, "latent_rows: latent size %d (1024 at most)", R);
@@ -510,7 +655,7 @@ extern "C" int scmx_latent_value(const float* part, const void* wuv, int64_t ldw
     SCMX_DT_OK("latent_value", out_dt);
     LATENT_ROWS_OK("latent_value", n);
     SCMX_REQUIRE(part && wuv && out && H > 0 && R > 0 && dv > 0 && ldw % 8 == 0 && ldw >= R && ldw <= 8192 && ((uintptr_t)wuv & 15) == 0 &&
-                 ldo >= (int64_t)H * dv && nsplit >= 1 && nsplit <= 32 && window >= 0 && cap >= 1, SCMX_EINVAL, "latent_value: heads %d of %d, latent %d", H, dv, R);
+                 ldo >= (int64_t)H * dv && nsplit >= 1 && nsplit <= LR_SPLITS && window >= 0 && cap >= 1, SCMX_EINVAL, "latent_value: heads %d of %d, latent %d", H, dv, R);
     SCMX_REQUIRE(pos_dev != nullptr || (pos >= 0 && pos + n <= cap), SCMX_EINVAL, "latent_value: %lld rows at %lld in a cache of %lld", (long long)n,
                  (long long)pos, (long long)cap);
     if (n == 0) return SCMX_OK;

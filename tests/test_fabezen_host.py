@@ -39,7 +39,7 @@ def test_arguments_are_checked_before_a_launch(scmx):
     assert b"cache of 64" in lib.scmx_last_error_string()
     assert lib.scmx_latent_rows(p, p, 24, 0, 1, 0, None, 64, 0, 2, 1040, 4, 1.0, 4, p, None) == -1
     assert lib.scmx_latent_rows(p, p, 1048, 0, 1, 0, None, 64, 0, 2, 1040, 4, 1.0, 4, p, None) == -5
-    assert lib.scmx_latent_rows(p, p, 24, 0, 1, 0, None, 64, 0, 2, 16, 4, 1.0, 33, p, None) == -1
+    assert lib.scmx_latent_rows(p, p, 24, 0, 1, 0, None, 64, 0, 2, 16, 4, 1.0, 65, p, None) == -1
     la = lambda k0, dd=64, pos=100, window=50: lib.scmx_latent_attn(p, 512, p, 512, p, 128, 4, pos, k0, window, 2, dd, 8, 64, 1.0, p, p, None)   # noqa: E731
     assert la(52) == -1 and la(0, 12) == -5 and la(0, 136) == -5 and la(1, window=0) == -1
 
