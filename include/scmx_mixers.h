@@ -106,7 +106,7 @@ int scmx_latent_rotate(void* q, int64_t ldq, int dt, const float* cs, int64_t n,
 int scmx_latent_absorb(const void* q, int64_t ldq, int q_dt, const void* wuk, int64_t ldw, int w_dt, const float* cs, int64_t cs_rows, int64_t n,
                        int H, int d, int R, int r, int64_t pos, const int32_t* pos_dev, float* out, void* stream);
 /* Softmax attention of absorbed queries (rows at pos, pos + 1, ..) over the cached latents, positions cut into nsplit <= 64
- * ranges: part float [n, H, nsplit, R + 2] for scmx_latent_value with the same pos, cap, window and nsplit.  R <= 1024. */
+ * ranges: part float [n, H, nsplit, R rounded up to 4, + 4] for scmx_latent_value with the same pos, cap, window and nsplit.  R <= 1024. */
 int scmx_latent_rows(const float* q, const void* cache, int64_t ldc, int dt, int64_t n, int64_t pos, const int32_t* pos_dev, int64_t cap,
                      int64_t window, int H, int R, int r, float scale, int nsplit, float* part, void* stream);
 /* out [n, H dv] = W_uv,h (combined latent); wuv [H dv, ldw]. */

@@ -5,8 +5,10 @@
 // latent_append_kernel   norms of the query latent and of c, rotation of the shared key part, cache rows
 // rotate_q_kernel        rotation of the queries' rotated parts in place (prompt portions before latent_attn_tc)
 // latent_absorb_kernel   queries in the latent space: [W_uk,h^T q_h, rotated part]
-// latent_rows_kernel     attention of such queries over the cache, positions split over CTAs (decode, short portions, float32)
+// latent_rows_*_kernel   attention of such queries over the cache, positions split over CTAs (decode, short portions, float32):
+//                        _mma for a bfloat16 cache, the plain one for float32
 // latent_value_kernel    combination of the splits and W_uv,h
+#include "../scmx_ptx.cuh"
 #include "mix_common.cuh"
 
 namespace scmx {
@@ -224,6 +226,10 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const AbsorbArgs<TQ,
 constexpr int LR_P = 32;         // positions per tile
 constexpr int LR_SPLITS = 64;    // ranges of positions at most
 
+// Pitch of a partial result: R values, maximum and sum, 16-byte aligned; maximum and sum start at column up4.
+__host__ __device__ __forceinline__ int up4(int n) { return (n + 3) & ~3; }
+__host__ __device__ __forceinline__ int part_pitch(int R) { return up4(R) + 4; }
+
 // Positions of a row's window cut into splits of whole tiles; how many splits have any.
 struct LatentSpan {
     int64_t lo, end, chunk;
@@ -243,7 +249,7 @@ struct LatentRowsArgs {
     const float* q;              // [n, H, R + r]
     const T* cache;              // [cap, ldc]
     const int32_t* pos_dev;
-    float* part;                 // [n, H, nsplit, R + 2]: unnormalized latent, running maximum (log2), running sum
+    float* part;                 // [n, H, nsplit, part_pitch(R)]: unnormalized latent, running maximum (log2), running sum
     int64_t pos, cap, ldc, window;
     int H, R, r, nsplit, ct;     // ct: threads across the column pairs (a power of two)
     float scale;
@@ -432,7 +438,7 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(const LatentRowsArgs<T
             __syncthreads();
         }
         if (h0 + h >= a.H) continue;             // uniform over the CTA
-        float* part = a.part + ((row * a.H + h0 + h) * a.nsplit + blockIdx.x) * (a.R + 2);
+        float* part = a.part + ((row * a.H + h0 + h) * a.nsplit + blockIdx.x) * part_pitch(a.R);
         if (grp == 0) {
 #pragma unroll
             for (int c = 0; c < NC; ++c) {
@@ -447,10 +453,156 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(const LatentRowsArgs<T
             }
         }
         if (tid == 0) {
-            part[a.R] = ml[h][0];
-            part[a.R + 1] = ml[h][1];
+            part[up4(a.R)] = ml[h][0];
+            part[up4(a.R) + 1] = ml[h][1];
         }
     }
+}
+
+// The same on mma (bfloat16 cache): eight heads per CTA, tiles of 32 positions brought by cp.async a tile ahead.  Scores: positions
+// are rows, heads columns, the warps share the inner index (each keeps its part of the queries, two terms, in registers) and their
+// sums meet in shared memory.  Values: the weights' two terms are the rows 0-7 and 8-15 of one operand, a warp owns NTV blocks of
+// eight latent columns.  KPW: 16-steps of the inner index per warp.
+__device__ __forceinline__ void mma_bf16(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+                 : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldsm4_t(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+
+constexpr int LM_H = 8;
+__host__ __device__ __forceinline__ int lm_pitch(int R, int r) { return (up8(R) + up8(r) + 15) / 16 * 16 + 8; }      // elements; rows fall into distinct banks
+
+template <int KPW, int NTV>
+__global__ void __launch_bounds__(256) latent_rows_mma_kernel(const LatentRowsArgs<bf16_t> a) {
+    extern __shared__ __align__(16) uint8_t smb[];
+    __shared__ __align__(16) float red[8][LR_P][LM_H];
+    __shared__ __align__(16) bf16_t ps[2][LM_H][LR_P + 8];               // weights, high and remainder terms
+    __shared__ float corr[LM_H];
+    const int Rp = up8(a.R), K = Rp + up8(a.r), KS = (K + 15) / 16, pitch = lm_pitch(a.R, a.r);
+    bf16_t* tile = reinterpret_cast<bf16_t*>(smb);                       // [2][LR_P][pitch]
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t4 = lane & 3, h0 = blockIdx.y * LM_H;
+    pdl_launch_dependents();
+    if (16 * KS > K)                                                     // the last 16-step's missing columns
+        for (int i = tid; i < 2 * LR_P; i += 256) *reinterpret_cast<uint4*>(tile + i * pitch + K) = make_uint4(0, 0, 0, 0);
+    pdl_wait();
+    const int64_t row = blockIdx.z, pos = (a.pos_dev != nullptr ? (int64_t)a.pos_dev[0] : a.pos) + row;
+    const LatentSpan span = latent_span(pos, a.cap, a.window, a.nsplit);
+    if ((int)blockIdx.x >= span.active) return;
+    const int64_t t0 = span.lo + blockIdx.x * span.chunk, t1 = min(span.end, t0 + span.chunk);
+    const int chunks = K / 8;
+    auto request = [&](int64_t tb, int buf) {
+        for (int i = tid; i < LR_P * chunks; i += 256) {
+            const int p = i / chunks, c = i - p * chunks;
+            const int64_t t = tb + p < t1 ? tb + p : t0;
+            asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(tile + (buf * LR_P + p) * pitch + 8 * c)), "l"(a.cache + t * a.ldc + 8 * c) : "memory");
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    request(t0, 0);
+    // queries of head g, this warp's 16-steps, scaled, as two terms
+    uint32_t qh[KPW][2], ql[KPW][2];
+    {
+        const float* q = a.q + (row * a.H + h0 + g) * (a.R + a.r);
+        const bool in = h0 + g < a.H;
+        const float f = a.scale * 1.4426950408889634f;
+        auto at = [&](int k) -> float {
+            if (!in) return 0.0f;
+            if (k < a.R) return q[k];
+            return k >= Rp && k - Rp < a.r ? q[a.R + k - Rp] : 0.0f;
+        };
+        float x[KPW][4];
+#pragma unroll
+        for (int i = 0; i < KPW; ++i) {
+            const int k = 16 * (warp + 8 * i) + 2 * t4;
+            x[i][0] = at(k); x[i][1] = at(k + 1); x[i][2] = at(k + 8); x[i][3] = at(k + 9);
+        }
+#pragma unroll
+        for (int i = 0; i < KPW; ++i)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const float u = x[i][2 * e] * f, v = x[i][2 * e + 1] * f;
+                qh[i][e] = pack_bf16x2(u, v);
+                ql[i][e] = pack_bf16x2(u - bf16_lo(qh[i][e]), v - bf16_hi(qh[i][e]));
+            }
+    }
+    float acc[NTV][4] = {};
+    float m = -INFINITY, l = 0.0f;               // of head h0 + warp
+    int buf = 0;
+    for (int64_t tb = t0; tb < t1; tb += LR_P, buf ^= 1) {
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();                         // the tile has arrived; the other buffer is consumed
+        if (tb + LR_P < t1) request(tb + LR_P, buf ^ 1);
+        const uint32_t base = smem_u32(tile + buf * LR_P * pitch);
+        float s[2][4] = {};
+        // a lane's address: rows 0-15 by lane % 16, the second eight columns for the upper half
+        const uint32_t arow = base + 2 * ((lane & 15) * pitch + 8 * (lane >> 4));
+#pragma unroll
+        for (int i = 0; i < KPW; ++i)
+            if (warp + 8 * i < KS)
+#pragma unroll
+                for (int mt = 0; mt < 2; ++mt) {
+                    uint32_t x[4];
+                    ldsm4(x, arow + 2 * (16 * mt * pitch + 16 * (warp + 8 * i)));
+                    mma_bf16(s[mt], x[0], x[1], x[2], x[3], qh[i][0], qh[i][1]);
+                    mma_bf16(s[mt], x[0], x[1], x[2], x[3], ql[i][0], ql[i][1]);
+                }
+#pragma unroll
+        for (int mt = 0; mt < 2; ++mt) {
+            *reinterpret_cast<float2*>(&red[warp][16 * mt + g][2 * t4]) = make_float2(s[mt][0], s[mt][1]);
+            *reinterpret_cast<float2*>(&red[warp][16 * mt + g + 8][2 * t4]) = make_float2(s[mt][2], s[mt][3]);
+        }
+        __syncthreads();
+        {                                        // softmax: a warp per head, a lane per position
+            float x = 0.0f;
+#pragma unroll
+            for (int w = 0; w < 8; ++w) x += red[w][lane][warp];
+            if (tb + lane >= t1) x = -INFINITY;
+            const float mn = fmaxf(m, warp_max(x)), p = ex2_approx(x - mn), c = ex2_approx(m - mn);      // finite: a tile has a position
+            l = l * c + warp_sumf(p);
+            m = mn;
+            const bf16_t hi = f32_to_bf16(p);
+            ps[0][warp][lane] = hi;
+            ps[1][warp][lane] = f32_to_bf16(p - bf16_to_f32(hi));
+            if (lane == 0) corr[warp] = c;
+        }
+        __syncthreads();
+        const float c = corr[g];
+#pragma unroll
+        for (int j = 0; j < NTV; ++j) {
+            acc[j][0] *= c; acc[j][1] *= c; acc[j][2] *= c; acc[j][3] *= c;
+        }
+        const uint32_t brow = base + 2 * ((lane & 15) * pitch + 8 * (lane >> 4));
+#pragma unroll
+        for (int kb = 0; kb < 2; ++kb) {
+            const uint32_t w0 = *reinterpret_cast<const uint32_t*>(&ps[0][g][16 * kb + 2 * t4]), w1 = *reinterpret_cast<const uint32_t*>(&ps[1][g][16 * kb + 2 * t4]);
+            const uint32_t w2 = *reinterpret_cast<const uint32_t*>(&ps[0][g][16 * kb + 2 * t4 + 8]), w3 = *reinterpret_cast<const uint32_t*>(&ps[1][g][16 * kb + 2 * t4 + 8]);
+#pragma unroll
+            for (int j = 0; j < NTV; j += 2) {
+                const int col = 8 * (warp * NTV + j);
+                if (col >= Rp) break;
+                uint32_t v[4];                   // tokens 0-7 and 8-15 of columns col .., then of col + 8 ..
+                ldsm4_t(v, brow + 2 * (16 * kb * pitch + col));
+                mma_bf16(acc[j], w0, w1, w2, w3, v[0], v[1]);
+                mma_bf16(acc[j + 1], w0, w1, w2, w3, v[2], v[3]);
+            }
+        }
+    }
+    const int pp = part_pitch(a.R);
+    if (h0 + g < a.H) {
+        float* part = a.part + ((row * a.H + h0 + g) * a.nsplit + blockIdx.x) * pp;
+#pragma unroll
+        for (int j = 0; j < NTV; ++j) {
+            const int col = 8 * (warp * NTV + j) + 2 * t4;
+            if (col < a.R) *reinterpret_cast<float2*>(part + col) = make_float2(acc[j][0] + acc[j][2], acc[j][1] + acc[j][3]);
+        }
+    }
+    if (lane == 0 && h0 + warp < a.H) *reinterpret_cast<float2*>(a.part + ((row * a.H + h0 + warp) * a.nsplit + blockIdx.x) * pp + up4(a.R)) = make_float2(m, l);
 }
 
 // ---- combination of the splits and the value product --------------------------------------------------------------------
@@ -466,7 +618,7 @@ struct LatentValueArgs {
 constexpr int LV_ROWS = 32;      // values per CTA, four per warp
 template <typename TW, typename TO>
 __global__ void __launch_bounds__(256) latent_value_kernel(const LatentValueArgs<TW, TO> a) {
-    extern __shared__ __align__(16) float ctx[];         // [ldw], zero padded
+    extern __shared__ __align__(16) float ctx[];         // [2][ldw]: halves of the sum, then the latent in the first
     __shared__ float cf[LR_SPLITS];
     pdl_launch_dependents();
     const int h = blockIdx.x, e0 = blockIdx.y * LV_ROWS, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -482,27 +634,41 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const LatentValueArgs
     pdl_wait();
     const int64_t row = blockIdx.z, pos = (a.pos_dev != nullptr ? (int64_t)a.pos_dev[0] : a.pos) + row;
     const int active = latent_span(pos, a.cap, a.window, a.nsplit).active;
-    const float* part = a.part + (row * a.H + h) * a.nsplit * (a.R + 2);
+    const int pp = part_pitch(a.R);
+    const float* part = a.part + (row * a.H + h) * a.nsplit * pp;
     if (warp == 0) {
-        float m[2], l[2];
+        float2 ml[2];
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
             const int sp = lane + 32 * i;
-            m[i] = sp < active ? part[sp * (a.R + 2) + a.R] : -INFINITY;
-            l[i] = sp < active ? part[sp * (a.R + 2) + a.R + 1] : 0.0f;
+            ml[i] = sp < active ? *reinterpret_cast<const float2*>(part + sp * pp + up4(a.R)) : make_float2(-INFINITY, 0.0f);
         }
-        const float mm = warp_max(fmaxf(m[0], m[1])), c0 = ex2_approx(m[0] - mm), c1 = ex2_approx(m[1] - mm);
-        const float inv = 1.0f / warp_sumf(c0 * l[0] + c1 * l[1]);
+        const float mm = warp_max(fmaxf(ml[0].x, ml[1].x)), c0 = ex2_approx(ml[0].x - mm), c1 = ex2_approx(ml[1].x - mm);
+        const float inv = 1.0f / warp_sumf(c0 * ml[0].y + c1 * ml[1].y);
         cf[lane] = c0 * inv;
         cf[lane + 32] = c1 * inv;
     }
     __syncthreads();
-    for (int e = tid; e < a.ldw; e += 256) {
-        float s = 0.0f;
-        if (e < a.R)
+    // two halves of the CTA take every second range, four columns per thread; the halves meet in shared memory
+    {
+        const int half = tid >> 7;
+        for (int e0_ = 4 * (tid & 127); e0_ < a.ldw; e0_ += 512) {
+            float4 s = make_float4(0, 0, 0, 0);
+            if (e0_ < a.R)
 #pragma unroll 16
-            for (int i = 0; i < active; ++i) s = fmaf(cf[i], part[i * (a.R + 2) + e], s);
-        ctx[e] = s;
+                for (int i = half; i < active; i += 2) {
+                    const float c = cf[i];
+                    const float4 v = *reinterpret_cast<const float4*>(part + i * pp + e0_);
+                    s.x = fmaf(c, v.x, s.x); s.y = fmaf(c, v.y, s.y); s.z = fmaf(c, v.z, s.z); s.w = fmaf(c, v.w, s.w);
+                }
+            // columns from R on are not results
+            if (e0_ + 1 >= a.R) s.y = 0.0f;
+            if (e0_ + 2 >= a.R) s.z = 0.0f;
+            if (e0_ + 3 >= a.R) s.w = 0.0f;
+            *reinterpret_cast<float4*>(ctx + half * a.ldw + e0_) = s;
+        }
+        __syncthreads();
+        for (int e = tid; e < a.ldw; e += 256) ctx[e] += ctx[a.ldw + e];
     }
     __syncthreads();
 #pragma unroll
@@ -542,6 +708,21 @@ static int run_latent_rows(LatentRowsArgs<T> a, int64_t n, cudaStream_t st) {
     SCMX_CUDA_OK(cudaFuncSetAttribute(latent_rows_kernel<T, HG, NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)total));
     SCMX_PDL_OK("latent_rows_kernel", launch_pdl(latent_rows_kernel<T, HG, NC>, dim3(a.nsplit, (a.H + HG - 1) / HG, (unsigned)n), dim3(256), total, st, a));
     return SCMX_OK;
+}
+
+template <int KPW, int NTV>
+static int run_latent_mma_n(const LatentRowsArgs<bf16_t>& a, int64_t n, cudaStream_t st) {
+    const size_t smem = (size_t)2 * LR_P * lm_pitch(a.R, a.r) * 2;
+    SCMX_CUDA_OK(cudaFuncSetAttribute(latent_rows_mma_kernel<KPW, NTV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    SCMX_PDL_OK("latent_rows_mma_kernel", launch_pdl(latent_rows_mma_kernel<KPW, NTV>, dim3(a.nsplit, (a.H + LM_H - 1) / LM_H, (unsigned)n), dim3(256), smem, st, a));
+    return SCMX_OK;
+}
+static int run_latent_mma(const LatentRowsArgs<bf16_t>& a, int64_t n, cudaStream_t st) {
+    const int KS = (up8(a.R) + up8(a.r) + 15) / 16;
+    SCMX_REQUIRE(KS <= 72, SCMX_ELIMIT, "latent_rows: latent size %d and rotated part %d", a.R, a.r);
+    if (KS <= 8 && a.R <= 128) return run_latent_mma_n<1, 2>(a, n, st);
+    if (KS <= 40 && a.R <= 512) return run_latent_mma_n<5, 8>(a, n, st);
+    return run_latent_mma_n<9, 16>(a, n, st);
 }
 
 template <typename TI, typename TC, typename TQ>
@@ -639,13 +820,13 @@ extern "C" int scmx_latent_rows(const float* q, const void* cache, int64_t ldc, 
 #define FILL(T)                                                                                                           \
     LatentRowsArgs<T> a;                                                                                                   \
     a.q = q; a.cache = (const T*)cache; a.pos_dev = pos_dev; a.part = part; a.pos = pos; a.cap = cap; a.ldc = ldc;         \
-    a.window = window; a.H = H; a.R = R; a.r = r; a.nsplit = nsplit; a.ct = 0; a.scale = scale;                            \
-    if (H <= 16) return R <= 512 ? run_latent_rows<T, 4, 1>(a, n, (cudaStream_t)stream) : run_latent_rows<T, 4, 2>(a, n, (cudaStream_t)stream); \
-    return R <= 512 ? run_latent_rows<T, 8, 1>(a, n, (cudaStream_t)stream) : run_latent_rows<T, 8, 2>(a, n, (cudaStream_t)stream)
+    a.window = window; a.H = H; a.R = R; a.r = r; a.nsplit = nsplit; a.ct = 0; a.scale = scale;
     if (dt == 0) {
         FILL(bf16_t);
+        return run_latent_mma(a, n, (cudaStream_t)stream);
     }
     FILL(float);
+    return R <= 512 ? run_latent_rows<float, 8, 1>(a, n, (cudaStream_t)stream) : run_latent_rows<float, 8, 2>(a, n, (cudaStream_t)stream);
 #undef FILL
 }
 
@@ -654,7 +835,7 @@ extern "C" int scmx_latent_value(const float* part, const void* wuv, int64_t ldw
     SCMX_DT_OK("latent_value", w_dt);
     SCMX_DT_OK("latent_value", out_dt);
     LATENT_ROWS_OK("latent_value", n);
-    SCMX_REQUIRE(part && wuv && out && H > 0 && R > 0 && dv > 0 && ldw % 8 == 0 && ldw >= R && ldw <= 8192 && ((uintptr_t)wuv & 15) == 0 &&
+    SCMX_REQUIRE(part && wuv && out && H > 0 && R > 0 && dv > 0 && ldw % 8 == 0 && ldw >= R && ldw <= 4096 && ((uintptr_t)wuv & 15) == 0 &&
                  ldo >= (int64_t)H * dv && nsplit >= 1 && nsplit <= LR_SPLITS && window >= 0 && cap >= 1, SCMX_EINVAL, "latent_value: heads %d of %d, latent %d", H, dv, R);
     SCMX_REQUIRE(pos_dev != nullptr || (pos >= 0 && pos + n <= cap), SCMX_EINVAL, "latent_value: %lld rows at %lld in a cache of %lld", (long long)n,
                  (long long)pos, (long long)cap);
@@ -665,7 +846,7 @@ extern "C" int scmx_latent_value(const float* part, const void* wuv, int64_t ldw
         LatentValueArgs<TW, TO> a;                                                                                         \
         a.part = part; a.wuv = (const TW*)wuv; a.out = (TO*)out; a.pos_dev = pos_dev; a.ldw = ldw; a.ldo = ldo; a.pos = pos; \
         a.cap = cap; a.window = window; a.H = H; a.R = R; a.dv = dv; a.nsplit = nsplit;                                    \
-        SCMX_PDL_OK("latent_value_kernel", launch_pdl(latent_value_kernel<TW, TO>, grid, block, (size_t)ldw * 4, (cudaStream_t)stream, a)); \
+        SCMX_PDL_OK("latent_value_kernel", launch_pdl(latent_value_kernel<TW, TO>, grid, block, (size_t)ldw * 8, (cudaStream_t)stream, a)); \
         return SCMX_OK;                                                                                                    \
     } while (0)
     if (w_dt == 0 && out_dt == 0) GO(bf16_t, bf16_t);

@@ -248,9 +248,9 @@ def latent_rows(q, wuk, wuv, cs, cache, H, d, r, dv, window, scale, out_dtype, p
     pos, pd = cache.offset, _lib.ptr(pos_dev)
     _lib.mcall("scmx_latent_absorb", _lib.ptr(q), _ld(q), _dt(q), _lib.ptr(wuk.w), wuk.w.shape[1], wuk.dt, _lib.ptr(cs), cs.shape[0], T, H, d, R, r, pos, pd,
                _lib.ptr(qa), _lib.stream())
-    groups = -(-H // (4 if H <= 16 else 8))
+    groups = -(-H // 8)
     nsplit = max(1, min(64, n_sm // (groups * T)))
-    part = torch.empty((T, H, nsplit, R + 2), dtype=torch.float32, device=dev)
+    part = torch.empty((T, H, nsplit, (R + 3) // 4 * 4 + 4), dtype=torch.float32, device=dev)
     _lib.mcall("scmx_latent_rows", _lib.ptr(qa), _lib.ptr(cache.c), cache.c.shape[1], _dt(cache.c), T, pos, pd, cache.capacity, window, H, R, r, scale,
                nsplit, _lib.ptr(part), _lib.stream())
     o = empty_rows(T, H * dv, out_dtype, dev)
