@@ -208,24 +208,6 @@ struct DiffDecodeArgs {
     float scale, lambda, diff, eps;
 };
 
-// Eight stored values as loaded, converted on use.
-template <typename T> struct Raw8;
-template <> struct Raw8<bf16_t> {
-    uint4 w;
-    __device__ __forceinline__ void load(const bf16_t* p) { w = *reinterpret_cast<const uint4*>(p); }
-    __device__ __forceinline__ void get(float (&x)[8]) const {
-        x[0] = bf16_lo(w.x); x[1] = bf16_hi(w.x); x[2] = bf16_lo(w.y); x[3] = bf16_hi(w.y);
-        x[4] = bf16_lo(w.z); x[5] = bf16_hi(w.z); x[6] = bf16_lo(w.w); x[7] = bf16_hi(w.w);
-    }
-};
-template <> struct Raw8<float> {
-    float4 a, b;
-    __device__ __forceinline__ void load(const float* p) { a = reinterpret_cast<const float4*>(p)[0]; b = reinterpret_cast<const float4*>(p)[1]; }
-    __device__ __forceinline__ void get(float (&x)[8]) const {
-        x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w; x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w;
-    }
-};
-
 constexpr int DD_P = 64;          // positions per tile
 constexpr int DD_MIN_CHUNK = 64;  // positions per split at least
 

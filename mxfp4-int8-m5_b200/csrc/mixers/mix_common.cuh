@@ -28,6 +28,29 @@ __device__ __forceinline__ void ld8(const float* p, float (&v)[8]) {
     v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
     v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
 }
+// Eight stored values as loaded, converted on use.
+template <typename T> struct Raw8;
+template <> struct Raw8<bf16_t> {
+    uint4 w;
+    __device__ __forceinline__ void load(const bf16_t* p) { w = *reinterpret_cast<const uint4*>(p); }
+    __device__ __forceinline__ void store(bf16_t* p) const { *reinterpret_cast<uint4*>(p) = w; }
+    __device__ __forceinline__ void get(float (&x)[8]) const {
+        x[0] = bf16_lo(w.x); x[1] = bf16_hi(w.x); x[2] = bf16_lo(w.y); x[3] = bf16_hi(w.y);
+        x[4] = bf16_lo(w.z); x[5] = bf16_hi(w.z); x[6] = bf16_lo(w.w); x[7] = bf16_hi(w.w);
+    }
+};
+template <> struct Raw8<float> {
+    float4 a, b;
+    __device__ __forceinline__ void load(const float* p) { a = reinterpret_cast<const float4*>(p)[0]; b = reinterpret_cast<const float4*>(p)[1]; }
+    __device__ __forceinline__ void store(float* p) const {
+        reinterpret_cast<float4*>(p)[0] = a;
+        reinterpret_cast<float4*>(p)[1] = b;
+    }
+    __device__ __forceinline__ void get(float (&x)[8]) const {
+        x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w; x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w;
+    }
+};
+
 // Four consecutive values.
 __device__ __forceinline__ void st4(bf16_t* p, float a, float b, float c, float d) {
     *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(a, b), pack_bf16x2(c, d));

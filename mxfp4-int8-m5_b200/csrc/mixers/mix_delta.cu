@@ -139,18 +139,62 @@ struct DeltaStepArgs {
     float eps;
 };
 
-// Dot product of a stored row (multiple of 8 columns) with a vector in shared memory, one warp.
+// Products of stored rows (multiples of 8 columns) with a vector in shared memory, a group of lanes per row.  The first vector of the
+// first PASS rows per group is requested by `request`, which may run before the vector is known.
 template <typename T>
-__device__ __forceinline__ float warp_row_dot(const T* w, const float* x, int n, int lane) {
-    float s = 0.0f;
-    for (int e = 8 * lane; e < n; e += 256) {
-        float v[8];
-        ld8(w + e, v);
-#pragma unroll
-        for (int i = 0; i < 8; ++i) s = fmaf(v[i], x[e + i], s);
+struct RowDots {
+    static constexpr int PASS = 2;
+    Raw8<T> pre[PASS];
+    int lpr, sub, first, step;
+    __device__ __forceinline__ void setup(int n, int lane, int warp) {
+        lpr = 1;
+        while (lpr < 32 && 8 * lpr < n) lpr *= 2;
+        sub = lane & (lpr - 1);
+        step = 256 / lpr;
+        first = (32 * warp + lane) / lpr;
     }
-    return warp_sumf(s);
-}
+    __device__ __forceinline__ void request(const T* w, int n, int rows) {
+#pragma unroll
+        for (int k = 0; k < PASS; ++k)
+            if (first + k * step < rows && 8 * sub < n) pre[k].load(w + (int64_t)(first + k * step) * n + 8 * sub);
+    }
+    // done(row, product) for every row, on the lanes of its group; the warps of the CTA call it together
+    template <typename F>
+    __device__ __forceinline__ void run(const T* w, const float* x, int n, int rows, F done) {
+        auto dot = [&](const Raw8<T>& u, int e, float s) -> float {
+            float v[8];
+            u.get(v);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) s = fmaf(v[i], x[e + i], s);
+            return s;
+        };
+        auto finish = [&](int row, float s) {
+            for (int e = 8 * (sub + lpr); e < n; e += 8 * lpr)
+                if (row < rows) {
+                    Raw8<T> u;
+                    u.load(w + (int64_t)row * n + e);
+                    s = dot(u, e, s);
+                }
+            for (int o = lpr / 2; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+            if (row < rows) done(row, s);
+        };
+#pragma unroll
+        for (int k = 0; k < PASS; ++k) {
+            const int row = first + k * step;
+            finish(row, row < rows && 8 * sub < n ? dot(pre[k], 8 * sub, 0.0f) : 0.0f);
+        }
+        for (int r0 = PASS * step; r0 < rows; r0 += step) {
+            const int row = first + r0;
+            float s = 0.0f;
+            if (row < rows && 8 * sub < n) {
+                Raw8<T> u;
+                u.load(w + (int64_t)row * n + 8 * sub);
+                s = dot(u, 8 * sub, 0.0f);
+            }
+            finish(row, s);
+        }
+    }
+};
 
 template <typename T, bool CH>
 __global__ void __launch_bounds__(256) delta_step_kernel(const DeltaStepArgs a) {
@@ -165,6 +209,17 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const DeltaStepArgs a) 
     const int e0 = rank * a.cw, cw = min(a.cw, a.dv - e0);      // cw may be <= 0 on a trailing rank
     const int groups = cw > 0 ? 256 / cw : 0, grp = cw > 0 ? tid / cw : 0, col = cw > 0 ? tid - grp * cw : 0;
     const bool work = grp < groups;
+    // low-rank weights of this CTA's channels and values never change: requested before the previous kernel ends
+    const int per = (a.d + nc - 1) / nc, ch0 = min(a.d, rank * per), nch = min(per, a.d - ch0);
+    const T *wa = static_cast<const T*>(a.wa) + ((int64_t)h * a.d + ch0) * a.lwa, *wg = static_cast<const T*>(a.wg) + ((int64_t)h * a.dv + e0) * a.lwg;
+    RowDots<T> da, dg;
+    if (CH) {
+        da.setup(a.lwa, lane, warp);
+        dg.setup(a.lwg, lane, warp);
+        da.request(wa, a.lwa, nch);
+        dg.request(wg, a.lwg, cw);
+        cl.sync();                   // every CTA of the cluster runs: its shared memory may be written
+    }
     pdl_wait();
     constexpr int PRE = 16;          // the first rows of this thread's column are requested before anything else
     float* S = a.state + (int64_t)h * a.d * a.dv + e0 + col;
@@ -197,20 +252,15 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const DeltaStepArgs a) 
     }
     float gate = 0.0f;
     if (CH) {
-        cl.sync();                   // every CTA of the cluster runs: its shared memory may be written
-        const T *wa = static_cast<const T*>(a.wa) + (int64_t)h * a.d * a.lwa, *wg = static_cast<const T*>(a.wg) + ((int64_t)h * a.dv + e0) * a.lwg;
-        const int per = (a.d + nc - 1) / nc, c1 = min(a.d, (rank + 1) * per);
-#pragma unroll 4
-        for (int c = rank * per + warp; c < c1; c += 8) {
-            const float z = warp_row_dot(wa + (int64_t)c * a.lwa, sa, a.lwa, lane) + a.dtb[(int64_t)h * a.d + c];
-            const float g = expf(nA * softplus_f32(z));
-            if (lane < nc) *cl.map_shared_rank(sg + c, lane) = g;
-        }
-#pragma unroll 4
-        for (int c = warp; c < cw; c += 8) {
-            const float z = warp_row_dot(wg + (int64_t)c * a.lwg, sg1, a.lwg, lane);
-            if (lane == 0) sgate[c] = 1.0f / (1.0f + expf(-z));
-        }
+        __syncthreads();
+        da.run(wa, sa, a.lwa, nch, [&](int c, float z) {
+            if (da.sub >= nc) return;
+            const float g = expf(nA * softplus_f32(z + a.dtb[(int64_t)h * a.d + ch0 + c]));
+            for (int r = da.sub; r < nc; r += da.lpr) *cl.map_shared_rank(sg + ch0 + c, r) = g;
+        });
+        dg.run(wg, sg1, a.lwg, cw, [&](int c, float z) {
+            if (dg.sub == 0) sgate[c] = 1.0f / (1.0f + expf(-z));
+        });
         cl.sync();
         if (tid < cw) gate = sgate[tid];
     } else {

@@ -8,6 +8,9 @@
 //                      decay).  Ratios c_i / c_j are products of decays, so that nothing overflows however strong the decay is
 // delta_state_kernel   per head and 128 values, chunk after chunk: S^T lives in tensor memory (a lane per value), the products of a
 //                      chunk take S or U as the tensor-memory operand
+// delta_join_kernel    long portions with few heads run as several segments side by side: a first pass without outputs gives every
+//                      segment's end from a zero start and, from unit vectors in place of values, the matrix that a start is
+//                      multiplied with; the true starts follow from these; a second pass with them gives the outputs
 // Operands that enter the recurrence are stored as two bfloat16 terms (16 significant bits, three MMAs per product; raw keys,
 // queries and values are bfloat16 as projected and take one term); S itself is carried in float32.  Waits are bounded (status word
 // codes 61..64).
@@ -29,7 +32,18 @@ struct DeltaTcArgs {
     int32_t* status;
     uint64_t wait_ns;
     int nc, nvt;                             // chunks, item = chunk * H + head; tiles of 128 values
+    int nseg, len;                           // segments of `len` chunks (the last may be shorter)
+    float *ends, *mats, *starts;             // [nseg][H, d, dv], [nseg][H, d, d], [nseg][H, d, dv]; one segment: unused
 };
+
+// Segments: as many CTAs as SMs in either pass, four chunks each at least.
+constexpr int DT_SMS = 148;
+static int segments(int nc, int H, int nvt) {
+    int best = 1;
+    for (int s = 3; s <= 16; ++s)
+        if (nc / s >= 4 && H * nvt + (s - 2) * H * (nvt + 1) <= DT_SMS && s * H * nvt <= DT_SMS) best = s;
+    return best;
+}
 
 // Two or four values as two bfloat16 terms.
 __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
@@ -738,12 +752,15 @@ __device__ __forceinline__ void split32(const uint32_t (&v)[32], uint32_t (&pk)[
     for (int i = 0; i < 16; ++i) split2(__uint_as_float(v[2 * i]), __uint_as_float(v[2 * i + 1]), pk[i], pk[16 + i]);
 }
 
-template <int DB>
+// OUT: the pass with outputs (or the only one), from `starts`.  Otherwise the first pass over segments 0 .. nseg - 2: blockIdx.y =
+// value tile, or the unit vectors (nvt; not for segment 0, which starts from the carried state).
+template <int DB, bool OUT>
 __global__ void __launch_bounds__(DT_THREADS, 1)
     delta_state_kernel(const __grid_constant__ CUtensorMap tmWh, const __grid_constant__ CUtensorMap tmWl, const __grid_constant__ CUtensorMap tmQh,
                        const __grid_constant__ CUtensorMap tmQl, const __grid_constant__ CUtensorMap tmEh, const __grid_constant__ CUtensorMap tmEl,
                        const __grid_constant__ CUtensorMap tmBh, const __grid_constant__ CUtensorMap tmBl, const DeltaTcArgs a) {
     constexpr int D = 64 * DB;
+    if (!OUT && (int)blockIdx.y == a.nvt && (int)blockIdx.z + 1 >= a.nseg - 1) return;      // the unit vectors have no further segment
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);
     const uint32_t sbase = smem_u32(smem);
@@ -773,7 +790,9 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
     const uint32_t tmem = __shfl_sync(0xffffffffu, *tmem_slot, 0);
     pdl_wait();
     const DeltaArgs& p = a.p;
-    const int h = blockIdx.x, v0 = blockIdx.y * 128, nc = a.nc;
+    const bool unit = !OUT && (int)blockIdx.y == a.nvt;
+    const int h = blockIdx.x, v0 = unit ? 0 : blockIdx.y * 128, seg = blockIdx.z + (unit ? 1 : 0);
+    const int cb = seg * a.len, nc = min(a.len, a.nc - cb), dv = unit ? p.d : p.dv;      // chunks cb .. cb + nc - 1
     int fail = 0;
 
     if (warp == 0) {
@@ -790,12 +809,12 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
                 return true;
             };
             for (int c = 0; c < nc && fail == 0; ++c) {
-                const int item = c * p.H + h, row = item * DC;
+                const int item = (cb + c) * p.H + h, row = item * DC;
                 // slot c & 3 of the decays is free: it was read before the products of chunk c - 4, whose operands left the ring
                 bool first = true;
                 if (int w = mbar_wait(b_ve, (c & 1) ^ 1, abort_flag, a.wait_ns)) { fail = w == 1 ? 61 : -1; break; }
-                mbar_expect_tx(b_vf, 64 * 128 * 4);
-                bulk_load(sbase + DT_V_OFF, a.uv + ((int64_t)item * a.nvt + blockIdx.y) * DC * 128, 64 * 128 * 4, b_vf);
+                if (!unit) mbar_expect_tx(b_vf, 64 * 128 * 4);
+                if (!unit) bulk_load(sbase + DT_V_OFF, a.uv + ((int64_t)item * a.nvt + blockIdx.y) * DC * 128, 64 * 128 * 4, b_vf);
                 for (int b = 0; b < DB && fail == 0; ++b)
                     if (slot()) {
                         tma_load_2d(s, &tmWh, 128 * b, row, bar);
@@ -806,7 +825,7 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
                         }
                         first = false;
                     }
-                for (int b = 0; b < DB && fail == 0; ++b)
+                for (int b = 0; OUT && b < DB && fail == 0; ++b)
                     if (slot()) {
                         tma_load_2d(s, &tmQh, 128 * b, row, bar);
                         tma_load_2d(s + DC_BLK, &tmQl, 128 * b, row, bar);
@@ -816,7 +835,9 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
                         tma_load_2d(s, DB == 1 || b == 0 ? &tmEh : &tmEl, 0, row, bar);
                         tma_load_2d(s + DC_BLK, DB == 2 && b == 0 ? &tmEh : &tmEl, DB == 2 ? 128 : 0, row, bar);
                     }
-                if (fail || !slot()) break;
+                if (fail) break;
+                if (!OUT) continue;
+                if (!slot()) break;
                 tma_load_2d(s, &tmBh, 0, row, bar);
                 tma_load_2d(s + DC_BLK, &tmBl, 0, row, bar);
             }
@@ -865,9 +886,9 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
             if (!ok) break;
             umma_commit_on(on, b_u);
             const uint32_t o = tmem + DT_O + 64 * (c & 1);
-            if (!wait(b_oe + 8 * (c & 1), ((c >> 1) & 1) ^ 1, 63)) break;
+            if (OUT && !wait(b_oe + 8 * (c & 1), ((c >> 1) & 1) ^ 1, 63)) break;
 #pragma unroll
-            for (int b = 0; b < DB; ++b) {
+            for (int b = 0; OUT && b < DB; ++b) {
                 if (!(ok = next())) break;
                 split_product(o, tmem + DT_SP + 64 * b, b == 0);
                 done();
@@ -895,6 +916,7 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
             }
             if (!ok) break;
             umma_commit_on(on, b_s);
+            if (!OUT) continue;
             if (!(ok = next())) break;
             split_product(o, tmem + DT_UP, 0);
             done();
@@ -904,9 +926,10 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
     } else {
         const int wg = (warp - 2) >> 2, q = warp & 3, v = v0 + 32 * q + lane;
         const uint32_t lane_base = (uint32_t)(32 * q) << 16;
-        const bool in = v < p.dv, owner = wg < 2 * DB;       // owner: holds 32 channels of S
+        const bool in = v < dv, owner = wg < 2 * DB;       // owner: holds 32 channels of S
         const int ch = 32 * wg;
-        float* gS = p.state + ((int64_t)h * p.d + ch) * p.dv + v;
+        // this thread's row of a [heads, d, dv] state: channel ch, value v
+        auto state_row = [&](float* base, int segment) { return base + ((int64_t)segment * p.H + h) * p.d * dv + (int64_t)ch * dv + v; };
         auto wait = [&](uint32_t bar, uint32_t parity) -> bool {
             const int w = mbar_wait(bar, parity, abort_flag, a.wait_ns);
             if (__any_sync(0xffffffffu, w)) { fail = w == 1 ? 64 : -1; return false; }
@@ -915,11 +938,11 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
         };
         // T V of a chunk into U's place, this warpgroup's 32 tokens
         auto bring_values = [&](int c) -> bool {
-            if (!wait(b_vf, c & 1)) return false;
+            if (!unit && !wait(b_vf, c & 1)) return false;
             const float* src = reinterpret_cast<const float*>(smem + DT_V_OFF) + 32 * wg * 128 + 32 * q + lane;
             uint32_t u[32];
 #pragma unroll
-            for (int i = 0; i < 32; ++i) u[i] = in ? __float_as_uint(src[128 * i]) : 0u;
+            for (int i = 0; i < 32; ++i) u[i] = in && !unit ? __float_as_uint(src[128 * i]) : 0u;
             __syncwarp();
             if (lane == 0) mbar_arrive(b_ve);
             tmem_st32(tmem + DT_U + 32 * wg + lane_base, u);
@@ -935,13 +958,19 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
                     tmem_ld32(tmem + ch + lane_base, s);
                     tmem_ld_fence(s);
                 } else {
+                    const float* gS = a.nseg == 1 || (!OUT && seg == 0) ? state_row(p.state, 0) : OUT ? state_row(a.starts, seg) : nullptr;
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) s[i] = in && ch + i < p.d ? __float_as_uint(gS[(int64_t)i * p.dv]) : 0u;
+                    for (int i = 0; i < 32; ++i) {
+                        float x = unit && v == ch + i ? 1.0f : 0.0f;
+                        if (gS != nullptr && in && ch + i < p.d) x = gS[(int64_t)i * dv];
+                        s[i] = __float_as_uint(x);
+                    }
                 }
                 if (c == nc) {
+                    float* gE = !OUT ? state_row(unit ? a.mats : a.ends, seg) : seg == a.nseg - 1 ? state_row(p.state, 0) : nullptr;
 #pragma unroll
                     for (int i = 0; i < 32; ++i)
-                        if (in && ch + i < p.d) gS[(int64_t)i * p.dv] = __uint_as_float(s[i]);
+                        if (gE != nullptr && in && ch + i < p.d) gE[(int64_t)i * dv] = __uint_as_float(s[i]);
                 } else {
                     uint32_t pk[32];
                     split32(s, pk);
@@ -981,7 +1010,7 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
                 __syncwarp();
                 if (lane == 0) mbar_arrive(b_uw);
                 if (c + 1 < nc && !bring_values(c + 1)) break;
-            } else if (c > 0) {
+            } else if (OUT && c > 0) {
                 // outputs of the previous chunk, 32 tokens per warpgroup
                 const int b = (c - 1) & 1;
                 if (!wait(b_of + 8 * b, ((c - 1) >> 1) & 1)) break;
@@ -991,7 +1020,7 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
                 tc_fence_before();
                 __syncwarp();
                 if (lane == 0) mbar_arrive(b_oe + 8 * b);
-                const int64_t t0 = (int64_t)(c - 1) * DC + 32 * (wg - 2);
+                const int64_t t0 = (int64_t)(cb + c - 1) * DC + 32 * (wg - 2);
                 const int nt = (int)min((int64_t)32, p.n - t0);
                 float* out = p.o + (t0 * p.H + h) * p.dv + v;
                 const int64_t step = (int64_t)p.H * p.dv;
@@ -1021,16 +1050,87 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
     if (warp == 1) tmem_dealloc(tmem, 512);
 }
 
+
+// Starts of the segments: start 0 is the carried state, start 1 what segment 0 ends with, start s + 1 = M_s start_s + end_s.  Grid
+// (tiles of 32 values, heads); a warp owns 16 channels, operands in two terms.
+constexpr int DJ_PITCH = 40;
+template <int D>
+__global__ void __launch_bounds__(2 * D) delta_join_kernel(const DeltaTcArgs a) {
+    __shared__ float sS[D * DJ_PITCH];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t4 = lane & 3;
+    const DeltaArgs& p = a.p;
+    const int h = blockIdx.y, v0 = blockIdx.x * 32;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int64_t head = (int64_t)h * p.d * p.dv, plane = (int64_t)p.H * p.d * p.dv;
+    for (int i = tid; i < D * 32; i += 2 * D) {
+        const int c = i >> 5, v = i & 31;
+        sS[c * DJ_PITCH + v] = c < p.d && v0 + v < p.dv ? p.state[head + (int64_t)c * p.dv + v0 + v] : 0.0f;
+    }
+    __syncthreads();
+    for (int seg = 0; seg < a.nseg; ++seg) {
+        for (int i = tid; i < D * 32; i += 2 * D) {
+            const int c = i >> 5, v = i & 31;
+            if (c < p.d && v0 + v < p.dv) a.starts[seg * plane + head + (int64_t)c * p.dv + v0 + v] = sS[c * DJ_PITCH + v];
+        }
+        if (seg == a.nseg - 1) break;
+        const int r0 = 16 * warp + g;
+        float acc[4][4];
+#pragma unroll
+        for (int n = 0; n < 4; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int c = r0 + 8 * (e >> 1), v = v0 + 8 * n + 2 * t4 + (e & 1);
+                acc[n][e] = c < p.d && v < p.dv ? a.ends[seg * plane + head + (int64_t)c * p.dv + v] : 0.0f;
+            }
+        if (seg > 0) {
+            const float* m = a.mats + ((int64_t)seg * p.H + h) * p.d * p.d;
+            float x[D / 16][8];                  // this warp's rows of M: inner index as in the operand blocks
+#pragma unroll
+            for (int k = 0; k < D / 16; ++k)
+#pragma unroll
+                for (int e = 0; e < 8; ++e) {
+                    const int c = r0 + 8 * (e >> 2), j = 16 * k + t4 + 4 * (e & 3);
+                    x[k][e] = c < p.d && j < p.d ? m[(int64_t)c * p.d + j] : 0.0f;
+                }
+#pragma unroll
+            for (int k = 0; k < D / 16; ++k) {
+                uint32_t ah[4], al[4];
+                split2(x[k][0], x[k][1], ah[0], al[0]);
+                split2(x[k][4], x[k][5], ah[1], al[1]);
+                split2(x[k][2], x[k][3], ah[2], al[2]);
+                split2(x[k][6], x[k][7], ah[3], al[3]);
+#pragma unroll
+                for (int n = 0; n < 4; ++n) {
+                    uint32_t bh[2], bl[2];
+                    block_b<DJ_PITCH>(sS + 16 * k * DJ_PITCH + 8 * n, lane, bh, bl);
+                    mma_split(acc[n], ah, al, bh, bl);
+                }
+            }
+        }
+        __syncthreads();
+#pragma unroll
+        for (int n = 0; n < 4; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) sS[(r0 + 8 * (e >> 1)) * DJ_PITCH + 8 * n + 2 * t4 + (e & 1)] = acc[n][e];
+        __syncthreads();
+    }
+}
+
 bool delta_tc_supported(int64_t n, int H, int d, int dv, int64_t ldv) {
     return d % 8 == 0 && dv % 8 == 0 && d <= 128 && ldv % 8 == 0 && n < (1ll << 24) && (n + DC - 1) / DC * H < (1ll << 24);
 }
 
 static int64_t align256(int64_t b) { return (b + 255) / 256 * 256; }
 static int width(int d) { return d <= 64 ? 64 : 128; }
+static int64_t segment_bytes(int64_t n, int H, int d, int dv) {
+    const int nseg = segments((int)((n + DC - 1) / DC), H, (dv + 127) / 128);
+    return nseg == 1 ? 0 : 2 * align256((int64_t)nseg * H * d * dv * 4) + align256((int64_t)nseg * H * d * d * 4);
+}
 int64_t delta_tc_scratch(int64_t n, int H, int d, int dv) {
     const int64_t items = (n + DC - 1) / DC * H;
     return 6 * align256(items * DC * width(d) * 2) + 2 * align256(items * DC_BLK) + align256(items * ((dv + 127) / 128) * DC * 128 * 4) +
-           align256(items * width(d) * 4);
+           align256(items * width(d) * 4) + segment_bytes(n, H, d, dv);
 }
 
 static int run_prep_tc(void (*kernel)(DeltaTcArgs), int smem, int threads, bool (&configured)[64], const DeltaTcArgs& a, cudaStream_t st) {
@@ -1051,18 +1151,28 @@ static int run_prep(bool channel, const DeltaTcArgs& a, cudaStream_t st) {
                    : run_prep_tc(delta_prep_head_kernel<D>, DphSmem<D>::FLOATS * 4, DPH_THREADS, done[0], a, st);
 }
 
-template <int DB>
-static int run_state(const CUtensorMap (&m)[8], const DeltaTcArgs& a, cudaStream_t st) {
+template <int DB, bool OUT>
+static int run_state(const CUtensorMap (&m)[8], const DeltaTcArgs& a, dim3 grid, cudaStream_t st) {
     static bool configured[64] = {};
     const int dev = current_device();
     SCMX_REQUIRE(dev >= 0, SCMX_ECUDA, "no current CUDA device (ordinal 0..63)");
     if (!configured[dev]) {
-        SCMX_CUDA_OK(cudaFuncSetAttribute(delta_state_kernel<DB>, cudaFuncAttributeMaxDynamicSharedMemorySize, DT_SMEM));
+        SCMX_CUDA_OK(cudaFuncSetAttribute(delta_state_kernel<DB, OUT>, cudaFuncAttributeMaxDynamicSharedMemorySize, DT_SMEM));
         configured[dev] = true;
     }
-    SCMX_PDL_OK("delta_state_kernel", launch_pdl(delta_state_kernel<DB>, dim3(a.p.H, (a.p.dv + 127) / 128), dim3(DT_THREADS), (size_t)DT_SMEM, st, m[0], m[1],
-                                                 m[2], m[3], m[4], m[5], m[6], m[7], a));
+    SCMX_PDL_OK("delta_state_kernel", launch_pdl(delta_state_kernel<DB, OUT>, grid, dim3(DT_THREADS), (size_t)DT_SMEM, st, m[0], m[1], m[2], m[3], m[4], m[5],
+                                                 m[6], m[7], a));
     return SCMX_OK;
+}
+template <int DB>
+static int run_states(const CUtensorMap (&m)[8], const DeltaTcArgs& a, cudaStream_t st) {
+    if (a.nseg > 1) {
+        // segments 0 .. nseg - 2 of the values, 1 .. nseg - 2 of the unit vectors: the latter's blockIdx.z counts from segment 1
+        const int rc = run_state<DB, false>(m, a, dim3(a.p.H, a.nvt + 1, a.nseg - 1), st);
+        if (rc) return rc;
+        SCMX_PDL_OK("delta_join_kernel", launch_pdl(delta_join_kernel<64 * DB>, dim3((a.p.dv + 31) / 32, a.p.H), dim3(128 * DB), 0, st, a));
+    }
+    return run_state<DB, true>(m, a, dim3(a.p.H, a.nvt, a.nseg), st);
 }
 
 int delta_tc(const DeltaArgs& p, bool channel, void* scratch, int32_t* status, cudaStream_t st) {
@@ -1078,14 +1188,20 @@ int delta_tc(const DeltaArgs& p, bool channel, void* scratch, int32_t* status, c
     bf16_t** square[2] = {&a.bh, &a.bl};
     for (auto x : square) { *x = reinterpret_cast<bf16_t*>(s); s += align256(items * DC_BLK); }
     a.uv = reinterpret_cast<float*>(s); s += align256(items * a.nvt * DC * 128 * 4);
-    a.gend = reinterpret_cast<float*>(s);
+    a.gend = reinterpret_cast<float*>(s); s += align256(items * D * 4);
+    a.nseg = segments(a.nc, p.H, a.nvt);
+    a.len = (a.nc + a.nseg - 1) / a.nseg;
+    a.nseg = (a.nc + a.len - 1) / a.len;         // no empty segment
+    a.ends = reinterpret_cast<float*>(s); s += align256((int64_t)a.nseg * p.H * p.d * p.dv * 4);
+    a.starts = reinterpret_cast<float*>(s); s += align256((int64_t)a.nseg * p.H * p.d * p.dv * 4);
+    a.mats = reinterpret_cast<float*>(s);
     CUtensorMap m[8];
     int rc = 0;
     const bf16_t* src[8] = {a.wh, a.wl, a.qh, a.ql, a.eh, a.el, a.bh, a.bl};
     for (int i = 0; i < 8 && !rc; ++i) rc = make_map_u8(&m[i], src[i], items * DC, i < 6 ? 2 * D : 128, 128, DC, 128, 0);
     if (!rc) rc = D == 64 ? run_prep<64>(channel, a, st) : run_prep<128>(channel, a, st);
     if (rc) return rc;
-    return D == 64 ? run_state<1>(m, a, st) : run_state<2>(m, a, st);
+    return D == 64 ? run_states<1>(m, a, st) : run_states<2>(m, a, st);
 }
 
 }  // namespace scmx

@@ -255,25 +255,6 @@ struct LatentRowsArgs {
     float scale;
 };
 
-// Eight stored values as loaded, converted on use.
-template <typename T> struct Vec8Raw;
-template <> struct Vec8Raw<bf16_t> {
-    uint4 w;
-    __device__ __forceinline__ void load(const bf16_t* p) { w = *reinterpret_cast<const uint4*>(p); }
-    __device__ __forceinline__ void store(bf16_t* p) const { *reinterpret_cast<uint4*>(p) = w; }
-    __device__ __forceinline__ void get(float (&x)[8]) const {
-        x[0] = bf16_lo(w.x); x[1] = bf16_hi(w.x); x[2] = bf16_lo(w.y); x[3] = bf16_hi(w.y);
-        x[4] = bf16_lo(w.z); x[5] = bf16_hi(w.z); x[6] = bf16_lo(w.w); x[7] = bf16_hi(w.w);
-    }
-};
-template <> struct Vec8Raw<float> {
-    float4 a, b;
-    __device__ __forceinline__ void load(const float* p) { a = reinterpret_cast<const float4*>(p)[0]; b = reinterpret_cast<const float4*>(p)[1]; }
-    __device__ __forceinline__ void store(float* p) const { reinterpret_cast<float4*>(p)[0] = a; reinterpret_cast<float4*>(p)[1] = b; }
-    __device__ __forceinline__ void get(float (&x)[8]) const {
-        x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w; x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w;
-    }
-};
 // Two neighbouring values.
 __device__ __forceinline__ float2 ld2(const bf16_t* p) {
     const uint32_t u = *reinterpret_cast<const uint32_t*>(p);
@@ -321,7 +302,7 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(const LatentRowsArgs<T
 #pragma unroll
         for (int c = 0; c < NC; ++c) acc[h][c][0] = acc[h][c][1] = 0.0f;
     constexpr int KEEP = sizeof(T) == 2 ? 3 : 1;
-    Vec8Raw<T> raw[KEEP][4];
+    Raw8<T> raw[KEEP][4];
     auto row_of = [&](int64_t tb, int p) -> const T* {
         const int64_t t = tb + 4 * warp + p;
         return a.cache + (t < t1 ? t : t0) * a.ldc;
@@ -339,7 +320,7 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(const LatentRowsArgs<T
         float s[4 * HG];
 #pragma unroll
         for (int i = 0; i < 4 * HG; ++i) s[i] = 0.0f;
-        auto use = [&](int v, const Vec8Raw<T> (&w)[4]) {
+        auto use = [&](int v, const Raw8<T> (&w)[4]) {
             float x[4][8];
 #pragma unroll
             for (int p = 0; p < 4; ++p) {
@@ -361,7 +342,7 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(const LatentRowsArgs<T
         for (int k = 0; k < KEEP; ++k)
             if (lane + 32 * k < nv) use(lane + 32 * k, raw[k]);
         for (int v = lane + 32 * KEEP; v < nv; v += 32) {
-            Vec8Raw<T> w[4];
+            Raw8<T> w[4];
 #pragma unroll
             for (int p = 0; p < 4; ++p) w[p].load(row_of(tb, p) + 8 * v);
             use(v, w);
@@ -625,7 +606,7 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const LatentValueArgs
     // the first vectors of this warp's rows are requested before the previous kernel ends: weights never change
     constexpr int ROWS = LV_ROWS / 8, PRE = sizeof(TW) == 2 ? 2 : 1;
     const TW* w = a.wuv + ((int64_t)h * a.dv + e0 + warp) * a.ldw + 8 * lane;
-    Vec8Raw<TW> pre[ROWS][PRE];
+    Raw8<TW> pre[ROWS][PRE];
 #pragma unroll
     for (int j = 0; j < ROWS; ++j)
 #pragma unroll
@@ -676,7 +657,7 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const LatentValueArgs
         const int e = e0 + warp + 8 * j;
         if (e >= a.dv) continue;
         float s = 0.0f;
-        auto add = [&](const Vec8Raw<TW>& u, int i) {
+        auto add = [&](const Raw8<TW>& u, int i) {
             float v[8];
             u.get(v);
 #pragma unroll
@@ -686,7 +667,7 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const LatentValueArgs
         for (int k = 0; k < PRE; ++k)
             if (8 * lane + 256 * k < a.ldw) add(pre[j][k], 8 * lane + 256 * k);
         for (int i = 8 * lane + 256 * PRE; i < a.ldw; i += 256) {
-            Vec8Raw<TW> u;
+            Raw8<TW> u;
             u.load(w + 8 * j * a.ldw + (i - 8 * lane));
             add(u, i);
         }

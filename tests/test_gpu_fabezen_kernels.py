@@ -173,6 +173,18 @@ def test_delta_chunks_weak_and_strong_decays(X, channel, strength, spread):
     assert err(c.run([100, 300], 1), o) < 5e-5 and err(c.state, S) < 5e-5
 
 
+@pytest.mark.parametrize("H,G,d,dv", [(2, 1, 64, 40), (1, 1, 128, 200), (3, 3, 40, 128)])
+@pytest.mark.parametrize("channel", [False, True])
+@pytest.mark.parametrize("cuts", [[1100], [530, 770]])
+def test_delta_segments(X, H, G, d, dv, channel, cuts):
+    """Long portions with few heads run as segments side by side, with a state carried in."""
+    c = DeltaCase(X, sum(cuts), H, G, d, dv, channel, BF, seed=5, strength=-5.0)
+    start = rnd(49, H, d, dv, scale=0.3)
+    c.state.copy_(start)
+    o, S = c.oracle(npy(start))
+    assert err(c.run(cuts, 2), o) < 5e-4 and err(c.state, S) < 5e-4
+
+
 def test_delta_far_value_is_read_back(X):
     """A value written once under its own key and asked for 700 tokens later, almost without decay."""
     for channel in (False, True):
