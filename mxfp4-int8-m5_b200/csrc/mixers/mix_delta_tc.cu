@@ -1052,67 +1052,66 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
 
 
 // Starts of the segments: start 0 is the carried state, start 1 what segment 0 ends with, start s + 1 = M_s start_s + end_s.  Grid
-// (tiles of 32 values, heads); a warp owns 16 channels, operands in two terms.
-constexpr int DJ_PITCH = 40;
+// (tiles of 8 values, heads); a warp owns 16 channels, operands in two terms.
+constexpr int DJ_V = 8, DJ_PITCH = 10;       // rows 4 t4 + e of four lanes fall into distinct banks
 template <int D>
 __global__ void __launch_bounds__(2 * D) delta_join_kernel(const DeltaTcArgs a) {
     __shared__ float sS[D * DJ_PITCH];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t4 = lane & 3;
     const DeltaArgs& p = a.p;
-    const int h = blockIdx.y, v0 = blockIdx.x * 32;
+    const int h = blockIdx.y, v = blockIdx.x * DJ_V + 2 * t4, r0 = 16 * warp + g;      // this lane's results: rows r0, r0 + 8, values v, v + 1
     pdl_launch_dependents();
     pdl_wait();
     const int64_t head = (int64_t)h * p.d * p.dv, plane = (int64_t)p.H * p.d * p.dv;
-    for (int i = tid; i < D * 32; i += 2 * D) {
-        const int c = i >> 5, v = i & 31;
-        sS[c * DJ_PITCH + v] = c < p.d && v0 + v < p.dv ? p.state[head + (int64_t)c * p.dv + v0 + v] : 0.0f;
-    }
-    __syncthreads();
-    for (int seg = 0; seg < a.nseg; ++seg) {
-        for (int i = tid; i < D * 32; i += 2 * D) {
-            const int c = i >> 5, v = i & 31;
-            if (c < p.d && v0 + v < p.dv) a.starts[seg * plane + head + (int64_t)c * p.dv + v0 + v] = sS[c * DJ_PITCH + v];
-        }
-        if (seg == a.nseg - 1) break;
-        const int r0 = 16 * warp + g;
-        float acc[4][4];
+    const bool in[2] = {r0 < p.d && v < p.dv, r0 + 8 < p.d && v < p.dv};
+    const int64_t at[2] = {head + (int64_t)r0 * p.dv + v, head + (int64_t)(r0 + 8) * p.dv + v};
+    // this warp's rows of M and of the end from zero; inner index: a lane's four values of a 16-step are neighbours
+    float4 m[2][D / 16];
+    float2 end[2], cur[2];
+    auto request = [&](int seg) {
+        const float* src = a.mats + ((int64_t)seg * p.H + h) * p.d * p.d;
 #pragma unroll
-        for (int n = 0; n < 4; ++n)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int c = r0 + 8 * (e >> 1), v = v0 + 8 * n + 2 * t4 + (e & 1);
-                acc[n][e] = c < p.d && v < p.dv ? a.ends[seg * plane + head + (int64_t)c * p.dv + v] : 0.0f;
-            }
-        if (seg > 0) {
-            const float* m = a.mats + ((int64_t)seg * p.H + h) * p.d * p.d;
-            float x[D / 16][8];                  // this warp's rows of M: inner index as in the operand blocks
-#pragma unroll
-            for (int k = 0; k < D / 16; ++k)
-#pragma unroll
-                for (int e = 0; e < 8; ++e) {
-                    const int c = r0 + 8 * (e >> 2), j = 16 * k + t4 + 4 * (e & 3);
-                    x[k][e] = c < p.d && j < p.d ? m[(int64_t)c * p.d + j] : 0.0f;
-                }
+        for (int r = 0; r < 2; ++r) {
+            const int c = r0 + 8 * r;
 #pragma unroll
             for (int k = 0; k < D / 16; ++k) {
-                uint32_t ah[4], al[4];
-                split2(x[k][0], x[k][1], ah[0], al[0]);
-                split2(x[k][4], x[k][5], ah[1], al[1]);
-                split2(x[k][2], x[k][3], ah[2], al[2]);
-                split2(x[k][6], x[k][7], ah[3], al[3]);
+                const int j = 16 * k + 4 * t4;
+                m[r][k] = seg > 0 && c < p.d && j < p.d ? *reinterpret_cast<const float4*>(src + (int64_t)c * p.d + j) : make_float4(0, 0, 0, 0);
+            }
+            end[r] = in[r] ? *reinterpret_cast<const float2*>(a.ends + seg * plane + at[r]) : make_float2(0, 0);
+        }
+    };
 #pragma unroll
-                for (int n = 0; n < 4; ++n) {
-                    uint32_t bh[2], bl[2];
-                    block_b<DJ_PITCH>(sS + 16 * k * DJ_PITCH + 8 * n, lane, bh, bl);
-                    mma_split(acc[n], ah, al, bh, bl);
-                }
+    for (int r = 0; r < 2; ++r) cur[r] = in[r] ? *reinterpret_cast<const float2*>(p.state + at[r]) : make_float2(0, 0);
+    request(0);
+    for (int seg = 0; seg < a.nseg; ++seg) {
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            if (in[r]) *reinterpret_cast<float2*>(a.starts + seg * plane + at[r]) = cur[r];
+            *reinterpret_cast<float2*>(sS + (r0 + 8 * r) * DJ_PITCH + 2 * t4) = cur[r];
+        }
+        if (seg == a.nseg - 1) break;
+        __syncthreads();
+        float acc[3][4] = {};                    // high high, high remainder, remainder high: shorter chains
+        acc[0][0] = end[0].x; acc[0][1] = end[0].y;
+        acc[0][2] = end[1].x; acc[0][3] = end[1].y;
+        if (seg > 0) {
+#pragma unroll
+            for (int k = 0; k < D / 16; ++k) {
+                uint32_t ah[4], al[4], bh[2], bl[2];
+                split4(m[0][k], ah[0], ah[2], al[0], al[2]);
+                split4(m[1][k], ah[1], ah[3], al[1], al[3]);
+                const float* x = sS + (16 * k + 4 * t4) * DJ_PITCH + g;
+                split2(x[0], x[DJ_PITCH], bh[0], bl[0]);
+                split2(x[2 * DJ_PITCH], x[3 * DJ_PITCH], bh[1], bl[1]);
+                mma_16816(acc[0], ah, bh[0], bh[1]);
+                mma_16816(acc[1], ah, bl[0], bl[1]);
+                mma_16816(acc[2], al, bh[0], bh[1]);
             }
         }
-        __syncthreads();
-#pragma unroll
-        for (int n = 0; n < 4; ++n)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) sS[(r0 + 8 * (e >> 1)) * DJ_PITCH + 8 * n + 2 * t4 + (e & 1)] = acc[n][e];
+        if (seg + 1 < a.nseg - 1) request(seg + 1);
+        cur[0] = make_float2(acc[0][0] + (acc[1][0] + acc[2][0]), acc[0][1] + (acc[1][1] + acc[2][1]));
+        cur[1] = make_float2(acc[0][2] + (acc[1][2] + acc[2][2]), acc[0][3] + (acc[1][3] + acc[2][3]));
         __syncthreads();
     }
 }
@@ -1170,7 +1169,7 @@ static int run_states(const CUtensorMap (&m)[8], const DeltaTcArgs& a, cudaStrea
         // segments 0 .. nseg - 2 of the values, 1 .. nseg - 2 of the unit vectors: the latter's blockIdx.z counts from segment 1
         const int rc = run_state<DB, false>(m, a, dim3(a.p.H, a.nvt + 1, a.nseg - 1), st);
         if (rc) return rc;
-        SCMX_PDL_OK("delta_join_kernel", launch_pdl(delta_join_kernel<64 * DB>, dim3((a.p.dv + 31) / 32, a.p.H), dim3(128 * DB), 0, st, a));
+        SCMX_PDL_OK("delta_join_kernel", launch_pdl(delta_join_kernel<64 * DB>, dim3((a.p.dv + DJ_V - 1) / DJ_V, a.p.H), dim3(128 * DB), 0, st, a));
     }
     return run_state<DB, true>(m, a, dim3(a.p.H, a.nvt, a.nseg), st);
 }
