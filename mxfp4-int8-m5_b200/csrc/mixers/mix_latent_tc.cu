@@ -4,7 +4,7 @@
 // A CTA owns two tiles of 128 query rows of one head; they share the key and value tiles, and while the tensor core works on one
 // tile the other tile's softmax runs.  320 threads:
 //   warp 0      TMA producer: both query tiles once, then per tile of 128 keys the head's keys, the shared part and the values
-//   warp 1      one thread issues all MMAs: S_m = Q_m K^T (128 x 128, float32 in tensor memory), O_m += P_m V with P_m read from
+//   warp 1      all MMAs (the warp stays converged, one lane issues): S_m = Q_m K^T (128 x 128, float32 in tensor memory), O_m += P_m V with P_m read from
 //               tensor memory (it overwrites S_m)
 //   warps 2-9   two softmax warpgroups, one per query tile, a thread per row.  Weights are split into two bfloat16 terms (16
 //               significant bits); the running maximum is only raised when it has grown by more than 2^8
@@ -54,7 +54,7 @@ __global__ void __launch_bounds__(LA_THREADS, 1)
                    b_o = b_p + 16;
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + L::MISC_OFF);
     volatile int* abort_flag = reinterpret_cast<volatile int*>(smem + L::MISC_OFF + 4);
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int warp = __shfl_sync(0xffffffffu, (int)(threadIdx.x >> 5), 0), lane = threadIdx.x & 31;
 
     if (threadIdx.x == 0) {
         for (const CUtensorMap* m : {&tmQ, &tmQr, &tmK, &tmKr, &tmV}) prefetch_map(m);
@@ -74,7 +74,7 @@ __global__ void __launch_bounds__(LA_THREADS, 1)
     tc_fence_before();
     __syncthreads();
     tc_fence_after();
-    const uint32_t tmem = *tmem_slot;
+    const uint32_t tmem = __shfl_sync(0xffffffffu, *tmem_slot, 0);
     pdl_wait();
 
     const int npair = (a.n + 255) / 256;
@@ -110,57 +110,66 @@ __global__ void __launch_bounds__(LA_THREADS, 1)
             }
         }
     } else if (warp == 1) {
-        if (lane == 0) {
-            const uint32_t idesc_s = umma_idesc_bf16(128, 128);
-            const uint32_t idesc_o = umma_idesc_bf16(128, (a.dv + 15) & ~15) | IDESC_B_MN;
-            const int dsteps = (a.d + 15) / 16, rsteps = RB ? (a.r + 15) / 16 : 0;
-            auto scores = [&](int m, int ks) {
-                for (int k = 0; k < dsteps + rsteps; ++k) {
-                    const int kk = k < dsteps ? k : 4 * DU + k - dsteps;
-                    const uint32_t o = (kk >> 2) * LA_TILE;
-                    const uint64_t da = umma_desc(sbase + L::Q_OFF + m * KB * LA_TILE + o), db = umma_desc(sbase + L::K_OFF + ks * KB * LA_TILE + o);
-                    umma_bf16(tmem + 128 * m, da + 2 * (kk & 3), db + 2 * (kk & 3), idesc_s, k > 0);
-                }
-                umma_commit(b_s + 8 * m);
-            };
-            do {
-                if (int w = mbar_wait(b_q, 0, abort_flag, a.wait_ns)) { fail = w == 1 ? 53 : -1; break; }
-                if (int w = mbar_wait(b_kf, 0, abort_flag, a.wait_ns)) { fail = w == 1 ? 53 : -1; break; }
-                tc_fence_after();
-                for (int m = 0; m < 2; ++m)
-                    if (jlo >= lo[m] && jlo < hi[m]) scores(m, 0);
-                umma_commit(b_ke);
-                for (int j = jlo; j < jhi && fail == 0; ++j) {
-                    const int i = j - jlo, vs = i % VS, kn = (i + 1) % KS;
-                    for (int m = 0; m < 2; ++m) {
-                        const bool on = j >= lo[m] && j < hi[m];
-                        if (on)
-                            if (int w = mbar_wait(b_p + 8 * m, (j - lo[m]) & 1, abort_flag, a.wait_ns)) { fail = w == 1 ? 54 : -1; break; }
-                        if (m == 0)
-                            if (int w = mbar_wait(b_vf + 8 * vs, (i / VS) & 1, abort_flag, a.wait_ns)) { fail = w == 1 ? 53 : -1; break; }
-                        tc_fence_after();
-                        if (on) {
-                            const uint64_t dv = umma_desc_mn(sbase + L::V_OFF + vs * VB * LA_TILE, LA_TILE);
+        // the whole warp walks through the tiles; `on` is the lane that issues
+        const uint32_t on = elect_lane();
+        const uint32_t idesc_s = umma_idesc_bf16(128, 128);
+        const uint32_t idesc_o = umma_idesc_bf16(128, (a.dv + 15) & ~15) | IDESC_B_MN;
+        const int dsteps = (a.d + 15) / 16, rsteps = RB ? (a.r + 15) / 16 : 0;
+        auto wait = [&](uint32_t bar, uint32_t parity, int code) -> bool {
+            const int w = mbar_wait(bar, parity, abort_flag, a.wait_ns);
+            if (__any_sync(0xffffffffu, w)) { fail = w == 1 ? code : -1; return false; }
+            tc_fence_after();
+            return true;
+        };
+        auto scores = [&](int m, int ks) {
+            const uint32_t d = tmem + 128 * m;
+            uint32_t acc = 0;
 #pragma unroll
-                            for (int k = 0; k < 8; ++k) {       // 16 keys: high and remainder terms, 8 columns each
-                                const uint32_t pa = tmem + 128 * m + (k >> 1) * 32 + (k & 1) * 8;
-                                umma_bf16_ts(tmem + 256 + 128 * m, pa, dv + 128 * k, idesc_o, j > lo[m] || k > 0);
-                                umma_bf16_ts(tmem + 256 + 128 * m, pa + 16, dv + 128 * k, idesc_o, 1);
-                            }
-                            if (j + 1 == hi[m]) umma_commit(b_o + 8 * m);
-                        }
-                        if (j + 1 < jhi) {
-                            if (m == 0)
-                                if (int w = mbar_wait(b_kf + 8 * kn, ((i + 1) / KS) & 1, abort_flag, a.wait_ns)) { fail = w == 1 ? 53 : -1; break; }
-                            tc_fence_after();
-                            if (j + 1 >= lo[m] && j + 1 < hi[m]) scores(m, kn);
-                            if (m == 1) umma_commit(b_ke + 8 * kn);
-                        }
-                        if (m == 1) umma_commit(b_ve + 8 * vs);
+            for (int c = 0; c < KB; ++c) {
+                const uint64_t da = umma_desc(sbase + L::Q_OFF + (m * KB + c) * LA_TILE), db = umma_desc(sbase + L::K_OFF + (ks * KB + c) * LA_TILE);
+                const int steps = c < DU ? dsteps - 4 * c : rsteps;
+#pragma unroll
+                for (int k = 0; k < 4; ++k)
+                    if (k < steps) {
+                        umma_bf16_on(on, d, da + 2 * k, db + 2 * k, idesc_s, acc);
+                        acc = 1;
                     }
-                }
-            } while (false);
+            }
+            umma_commit_on(on, b_s + 8 * m);
+        };
+        bool ok = wait(b_q, 0, 53) && wait(b_kf, 0, 53);
+        if (ok) {
+#pragma unroll
+            for (int m = 0; m < 2; ++m)
+                if (jlo >= lo[m] && jlo < hi[m]) scores(m, 0);
+            umma_commit_on(on, b_ke);
         }
+        for (int j = jlo; j < jhi && ok; ++j) {
+            const int i = j - jlo, vs = i % VS, kn = (i + 1) % KS;
+#pragma unroll
+            for (int m = 0; m < 2; ++m) {
+                const bool now = j >= lo[m] && j < hi[m];
+                if (now && !(ok = wait(b_p + 8 * m, (j - lo[m]) & 1, 54))) break;
+                if (m == 0 && !(ok = wait(b_vf + 8 * vs, (i / VS) & 1, 53))) break;
+                if (now) {
+                    const uint64_t dv = umma_desc_mn(sbase + L::V_OFF + vs * VB * LA_TILE, LA_TILE);
+#pragma unroll
+                    for (int k = 0; k < 8; ++k) {       // 16 keys: high and remainder terms, 8 columns each
+                        const uint32_t pa = tmem + 128 * m + (k >> 1) * 32 + (k & 1) * 8;
+                        umma_bf16_ts_on(on, tmem + 256 + 128 * m, pa, dv + 128 * k, idesc_o, k > 0 ? 1u : (uint32_t)(j > lo[m]));
+                        umma_bf16_ts_on(on, tmem + 256 + 128 * m, pa + 16, dv + 128 * k, idesc_o, 1);
+                    }
+                    if (j + 1 == hi[m]) umma_commit_on(on, b_o + 8 * m);
+                }
+                if (j + 1 < jhi) {
+                    if (m == 0 && !(ok = wait(b_kf + 8 * kn, ((i + 1) / KS) & 1, 53))) break;
+                    if (j + 1 >= lo[m] && j + 1 < hi[m]) scores(m, kn);
+                    if (m == 1) umma_commit_on(on, b_ke + 8 * kn);
+                }
+                if (m == 1) umma_commit_on(on, b_ve + 8 * vs);
+            }
+        }
+        if (!on) fail = fail > 0 ? -1 : fail;      // one lane reports
     } else {
         const int m = (warp - 2) >> 2, q = warp & 3, row = 32 * q + lane;
         const uint32_t lane_base = (uint32_t)(32 * q) << 16, ts = tmem + 128 * m + lane_base, to = tmem + 256 + 128 * m + lane_base;
