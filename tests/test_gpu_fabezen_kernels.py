@@ -140,7 +140,7 @@ class DeltaCase:
         return O.delta_rule(q, k, npy(self.v).reshape(T, H, dv), g, O.sigmoid(npy(self.b)), S)
 
 
-@pytest.mark.parametrize("H,G,d,dv", [(2, 2, 16, 24), (4, 2, 64, 32), (3, 1, 5, 7), (2, 1, 128, 40), (1, 1, 200, 70), (6, 3, 24, 64)])
+@pytest.mark.parametrize("H,G,d,dv", [(2, 2, 16, 24), (4, 2, 48, 32), (3, 1, 5, 7), (2, 1, 128, 40), (1, 1, 200, 70), (6, 3, 24, 64)])
 @pytest.mark.parametrize("channel", [False, True])
 @pytest.mark.parametrize("dt", [BF, F32])
 def test_delta_token_by_token(X, H, G, d, dv, channel, dt):
@@ -201,7 +201,7 @@ def test_delta_far_value_is_read_back(X):
             assert np.abs(o[740]).max() > 1.0
 
 
-@pytest.mark.parametrize("H,G,d,dv,ra,rg", [(2, 1, 16, 24, 5, 9), (4, 4, 64, 64, 24, 24), (3, 3, 130, 100, 16, 40), (2, 2, 128, 300, 128, 64), (1, 1, 7, 5, 1, 1)])
+@pytest.mark.parametrize("H,G,d,dv,ra,rg", [(2, 1, 16, 24, 5, 9), (4, 4, 64, 72, 24, 40), (3, 3, 130, 100, 16, 40), (2, 2, 128, 300, 128, 64), (1, 1, 7, 5, 1, 1)])
 @pytest.mark.parametrize("channel", [False, True])
 @pytest.mark.parametrize("dt", [BF, F32])
 def test_delta_step(X, H, G, d, dv, ra, rg, channel, dt):
@@ -265,7 +265,7 @@ class LatentCase:
                                                   self.window or None) for i in range(H)], 1)
 
 
-@pytest.mark.parametrize("Q,R,r", [(12, 20, 6), (96, 96, 32), (7, 13, 0), (300, 512, 64)])
+@pytest.mark.parametrize("Q,R,r", [(12, 20, 6), (80, 104, 24), (7, 13, 0), (300, 512, 64), (1536, 512, 64)])
 @pytest.mark.parametrize("dt,tol", [(BF, 1e-2), (F32, 3e-6)])
 def test_latent_append(scmx, Q, R, r, dt, tol):
     c = LatentCase(scmx, 30, 1, 8, r, 8, R, 0, dt, Q=Q, capacity=33)
@@ -279,7 +279,7 @@ def test_latent_append(scmx, Q, R, r, dt, tol):
     assert float(c.cache.c[:, R:up].abs().sum()) == 0.0 and float(c.cache.c[:, up + r:].abs().sum()) == 0.0 and float(c.cache.c[30:].abs().sum()) == 0.0
 
 
-@pytest.mark.parametrize("H,d,r,dv,R", [(1, 8, 2, 8, 12), (4, 64, 32, 64, 96), (3, 10, 6, 14, 21), (6, 24, 0, 16, 40), (20, 16, 8, 24, 64), (2, 32, 16, 40, 700),
+@pytest.mark.parametrize("H,d,r,dv,R", [(1, 8, 2, 8, 12), (4, 72, 24, 56, 88), (3, 10, 6, 14, 21), (6, 24, 0, 16, 40), (20, 16, 8, 24, 64), (2, 32, 16, 40, 700),
                                         (18, 8, 2, 8, 600)])
 @pytest.mark.parametrize("window", [0, 1, 33, 70])
 @pytest.mark.parametrize("dt,tol", [(BF, 1.5e-2), (F32, 1e-5)])
@@ -291,7 +291,7 @@ def test_latent_rows(scmx, H, d, r, dv, R, window, dt, tol):
     assert err(torch.cat([c.attend(0, 1, False), c.attend(1, 3, False), c.attend(4, T - 5, False), c.attend(T - 1, 1, False)]), want) < tol
 
 
-@pytest.mark.parametrize("H,d,r,dv,R", [(2, 64, 32, 64, 96), (3, 128, 64, 128, 64), (1, 24, 8, 40, 16), (2, 40, 0, 24, 32), (2, 96, 16, 128, 48), (2, 128, 0, 72, 40)])
+@pytest.mark.parametrize("H,d,r,dv,R", [(2, 56, 40, 64, 80), (3, 128, 64, 128, 64), (1, 24, 8, 40, 16), (2, 40, 0, 24, 32), (2, 96, 16, 128, 48), (2, 128, 0, 72, 40)])
 @pytest.mark.parametrize("window", [0, 1, 40, 128, 129, 300])
 def test_latent_prompt(scmx, H, d, r, dv, R, window):
     T = 420
