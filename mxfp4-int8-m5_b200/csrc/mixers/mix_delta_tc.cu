@@ -1052,23 +1052,26 @@ __global__ void __launch_bounds__(DT_THREADS, 1)
 
 
 // Starts of the segments: start 0 is the carried state, start 1 what segment 0 ends with, start s + 1 = M_s start_s + end_s.  Grid
-// (tiles of 8 values, heads); a warp owns 16 channels, operands in two terms.
-constexpr int DJ_V = 8, DJ_PITCH = 10;       // rows 4 t4 + e of four lanes fall into distinct banks
-template <int D>
+// (tiles of 8 NT values, heads); a warp owns 16 channels, operands in two terms.
+template <int D, int NT>
 __global__ void __launch_bounds__(2 * D) delta_join_kernel(const DeltaTcArgs a) {
-    __shared__ float sS[D * DJ_PITCH];
+    constexpr int PITCH = 8 * NT + 2;            // rows 4 t4 + e of four lanes fall into distinct banks
+    __shared__ float sS[D * PITCH];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t4 = lane & 3;
     const DeltaArgs& p = a.p;
-    const int h = blockIdx.y, v = blockIdx.x * DJ_V + 2 * t4, r0 = 16 * warp + g;      // this lane's results: rows r0, r0 + 8, values v, v + 1
+    const int h = blockIdx.y, v = blockIdx.x * 8 * NT + 2 * t4, r0 = 16 * warp + g;      // results: rows r0, r0 + 8, values v + 8 n, v + 8 n + 1
     pdl_launch_dependents();
     pdl_wait();
     const int64_t head = (int64_t)h * p.d * p.dv, plane = (int64_t)p.H * p.d * p.dv;
-    const bool in[2] = {r0 < p.d && v < p.dv, r0 + 8 < p.d && v < p.dv};
+    auto in = [&](int r, int n) { return r0 + 8 * r < p.d && v + 8 * n < p.dv; };
     const int64_t at[2] = {head + (int64_t)r0 * p.dv + v, head + (int64_t)(r0 + 8) * p.dv + v};
     // this warp's rows of M and of the end from zero; inner index: a lane's four values of a 16-step are neighbours
-    float4 m[2][D / 16];
-    float2 end[2], cur[2];
-    auto request = [&](int seg) {
+    struct Operand {
+        float4 m[2][D / 16];
+        float2 end[2][NT];
+    } x, y;
+    float2 cur[2][NT];
+    auto request = [&](int seg, Operand& o) {
         const float* src = a.mats + ((int64_t)seg * p.H + h) * p.d * p.d;
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
@@ -1076,43 +1079,58 @@ __global__ void __launch_bounds__(2 * D) delta_join_kernel(const DeltaTcArgs a) 
 #pragma unroll
             for (int k = 0; k < D / 16; ++k) {
                 const int j = 16 * k + 4 * t4;
-                m[r][k] = seg > 0 && c < p.d && j < p.d ? *reinterpret_cast<const float4*>(src + (int64_t)c * p.d + j) : make_float4(0, 0, 0, 0);
+                o.m[r][k] = seg > 0 && c < p.d && j < p.d ? *reinterpret_cast<const float4*>(src + (int64_t)c * p.d + j) : make_float4(0, 0, 0, 0);
             }
-            end[r] = in[r] ? *reinterpret_cast<const float2*>(a.ends + seg * plane + at[r]) : make_float2(0, 0);
+#pragma unroll
+            for (int n = 0; n < NT; ++n)
+                o.end[r][n] = in(r, n) ? *reinterpret_cast<const float2*>(a.ends + seg * plane + at[r] + 8 * n) : make_float2(0, 0);
         }
     };
+    // writes the start of a segment and forms the next one, whose operand was requested a segment ago
+    auto step = [&](int seg, const Operand& o, Operand& next) -> bool {
 #pragma unroll
-    for (int r = 0; r < 2; ++r) cur[r] = in[r] ? *reinterpret_cast<const float2*>(p.state + at[r]) : make_float2(0, 0);
-    request(0);
-    for (int seg = 0; seg < a.nseg; ++seg) {
+        for (int r = 0; r < 2; ++r)
 #pragma unroll
-        for (int r = 0; r < 2; ++r) {
-            if (in[r]) *reinterpret_cast<float2*>(a.starts + seg * plane + at[r]) = cur[r];
-            *reinterpret_cast<float2*>(sS + (r0 + 8 * r) * DJ_PITCH + 2 * t4) = cur[r];
-        }
-        if (seg == a.nseg - 1) break;
+            for (int n = 0; n < NT; ++n) {
+                if (in(r, n)) *reinterpret_cast<float2*>(a.starts + seg * plane + at[r] + 8 * n) = cur[r][n];
+                *reinterpret_cast<float2*>(sS + (r0 + 8 * r) * PITCH + 8 * n + 2 * t4) = cur[r][n];
+            }
+        if (seg == a.nseg - 1) return false;
+        if (seg + 1 < a.nseg - 1) request(seg + 1, next);
         __syncthreads();
-        float acc[3][4] = {};                    // high high, high remainder, remainder high: shorter chains
-        acc[0][0] = end[0].x; acc[0][1] = end[0].y;
-        acc[0][2] = end[1].x; acc[0][3] = end[1].y;
+        float acc[NT][3][4] = {};                // high high, high remainder, remainder high: shorter chains
         if (seg > 0) {
 #pragma unroll
             for (int k = 0; k < D / 16; ++k) {
                 uint32_t ah[4], al[4], bh[2], bl[2];
-                split4(m[0][k], ah[0], ah[2], al[0], al[2]);
-                split4(m[1][k], ah[1], ah[3], al[1], al[3]);
-                const float* x = sS + (16 * k + 4 * t4) * DJ_PITCH + g;
-                split2(x[0], x[DJ_PITCH], bh[0], bl[0]);
-                split2(x[2 * DJ_PITCH], x[3 * DJ_PITCH], bh[1], bl[1]);
-                mma_16816(acc[0], ah, bh[0], bh[1]);
-                mma_16816(acc[1], ah, bl[0], bl[1]);
-                mma_16816(acc[2], al, bh[0], bh[1]);
+                split4(o.m[0][k], ah[0], ah[2], al[0], al[2]);
+                split4(o.m[1][k], ah[1], ah[3], al[1], al[3]);
+#pragma unroll
+                for (int n = 0; n < NT; ++n) {
+                    const float* s = sS + (16 * k + 4 * t4) * PITCH + 8 * n + g;
+                    split2(s[0], s[PITCH], bh[0], bl[0]);
+                    split2(s[2 * PITCH], s[3 * PITCH], bh[1], bl[1]);
+                    mma_16816(acc[n][0], ah, bh[0], bh[1]);
+                    mma_16816(acc[n][1], ah, bl[0], bl[1]);
+                    mma_16816(acc[n][2], al, bh[0], bh[1]);
+                }
             }
         }
-        if (seg + 1 < a.nseg - 1) request(seg + 1);
-        cur[0] = make_float2(acc[0][0] + (acc[1][0] + acc[2][0]), acc[0][1] + (acc[1][1] + acc[2][1]));
-        cur[1] = make_float2(acc[0][2] + (acc[1][2] + acc[2][2]), acc[0][3] + (acc[1][3] + acc[2][3]));
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+            for (int r = 0; r < 2; ++r)
+                cur[r][n] = make_float2(o.end[r][n].x + (acc[n][0][2 * r] + (acc[n][1][2 * r] + acc[n][2][2 * r])),
+                                        o.end[r][n].y + (acc[n][0][2 * r + 1] + (acc[n][1][2 * r + 1] + acc[n][2][2 * r + 1])));
         __syncthreads();
+        return true;
+    };
+#pragma unroll
+    for (int r = 0; r < 2; ++r)
+#pragma unroll
+        for (int n = 0; n < NT; ++n) cur[r][n] = in(r, n) ? *reinterpret_cast<const float2*>(p.state + at[r] + 8 * n) : make_float2(0, 0);
+    request(0, x);
+    for (int seg = 0; step(seg, x, y) && step(seg + 1, y, x); seg += 2) {
     }
 }
 
@@ -1169,7 +1187,11 @@ static int run_states(const CUtensorMap (&m)[8], const DeltaTcArgs& a, cudaStrea
         // segments 0 .. nseg - 2 of the values, 1 .. nseg - 2 of the unit vectors: the latter's blockIdx.z counts from segment 1
         const int rc = run_state<DB, false>(m, a, dim3(a.p.H, a.nvt + 1, a.nseg - 1), st);
         if (rc) return rc;
-        SCMX_PDL_OK("delta_join_kernel", launch_pdl(delta_join_kernel<64 * DB>, dim3((a.p.dv + DJ_V - 1) / DJ_V, a.p.H), dim3(128 * DB), 0, st, a));
+        const int nt = (a.p.dv + 7) / 8 * a.p.H <= DT_SMS ? 1 : (a.p.dv + 15) / 16 * a.p.H <= DT_SMS ? 2 : 4;      // one round of CTAs
+        const dim3 grid((a.p.dv + 8 * nt - 1) / (8 * nt), a.p.H), block(128 * DB);
+        SCMX_PDL_OK("delta_join_kernel", nt == 1   ? launch_pdl(delta_join_kernel<64 * DB, 1>, grid, block, 0, st, a)
+                                         : nt == 2 ? launch_pdl(delta_join_kernel<64 * DB, 2>, grid, block, 0, st, a)
+                                                   : launch_pdl(delta_join_kernel<64 * DB, 4>, grid, block, 0, st, a));
     }
     return run_state<DB, true>(m, a, dim3(a.p.H, a.nvt, a.nseg), st);
 }

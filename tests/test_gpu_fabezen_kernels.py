@@ -173,9 +173,9 @@ def test_delta_chunks_weak_and_strong_decays(X, channel, strength, spread):
     assert err(c.run([100, 300], 1), o) < 5e-5 and err(c.state, S) < 5e-5
 
 
-@pytest.mark.parametrize("H,G,d,dv", [(2, 1, 64, 40), (1, 1, 128, 200), (3, 3, 40, 128)])
+@pytest.mark.parametrize("H,G,d,dv", [(2, 1, 64, 40), (1, 1, 128, 200), (3, 3, 40, 128), (16, 8, 16, 128), (32, 16, 8, 120)])
 @pytest.mark.parametrize("channel", [False, True])
-@pytest.mark.parametrize("cuts", [[1100], [530, 770]])
+@pytest.mark.parametrize("cuts", [[1000], [530, 770]])
 def test_delta_segments(X, H, G, d, dv, channel, cuts):
     """Long portions with few heads run as segments side by side, with a state carried in."""
     c = DeltaCase(X, sum(cuts), H, G, d, dv, channel, BF, seed=5, strength=-5.0)
